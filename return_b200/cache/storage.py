@@ -10,11 +10,12 @@ contiguous.  A mixer whose cache is one vector a token (``LatentCacheNeed``: a l
 heads) gets a group of its own kind by (window, width) and one tensor ``[layers, num_pages, page_size, width]``.
 A mixer that asks for state of fixed size gets ``[max_reside + 1, *shape]``, one row per
 request slot and a last one that belongs to no request (the padding rows of a captured decode step
-point at it) (after rollout/cache.py:340-360).
+point at it) (after rollout/cache.py:340-360).  A run may also keep numbers of its own per request beside the cache
+that it owns or reads (the last inputs of a convolution or a blend): they are states of the same kind.
 """
 from __future__ import annotations
 
-from typing import Dict, List, Optional, Tuple
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
@@ -24,11 +25,12 @@ from .manager import CacheManager, GroupSpec
 
 class CacheStorage:
     def __init__(self, needs: List[object], page_size: int, num_pages: int, max_reside: int, env: BuildEnv,
-                 longest_append: Optional[int] = None):
+                 longest_append: Optional[int] = None, kept: Sequence[Optional[StateNeed]] = ()):
         """``num_pages``: pages of a group that keeps every key (the pool's capacity in tokens / page size).
         A group that keeps a window gets only what ``max_reside`` requests can hold of it at a time: the
         window plus the longest run of tokens one step may append (``longest_append``; None: unknown, the
-        group then gets ``num_pages`` too), in pages, plus one for the ragged ends."""
+        group then gets ``num_pages`` too), in pages, plus one for the ragged ends.  ``kept``: per run of the schedule,
+        what it keeps per request for itself, whichever cache it owns or reads (``LayerContext.kept``)."""
         self.env = env
         self.page_size = page_size
         self.max_reside = max_reside
@@ -74,6 +76,9 @@ class CacheStorage:
 
         for index, need in enumerate(needs):
             register((index,), need)
+        for index, need in enumerate(kept):
+            if need is not None:
+                self._state_needs[("kept", index)] = need
         if not self.group_specs:
             # a model without paged layers still counts tokens per request
             self.group_specs.append(GroupSpec("none", page_size, num_pages, None))
@@ -123,6 +128,10 @@ class CacheStorage:
 
     def layer_context(self, owner_index: int, batch, write: bool) -> LayerContext:
         return self._context((owner_index,), batch, write)
+
+    def kept(self, index: int) -> Optional[torch.Tensor]:
+        """What the run with this schedule index keeps per request for itself, [max_reside + 1, n], or None."""
+        return self.states.get(("kept", index))
 
     def _context(self, key: Tuple, batch, write: bool) -> LayerContext:
         ctx = LayerContext(batch=batch, write_cache=write)

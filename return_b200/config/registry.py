@@ -105,6 +105,12 @@ def _register_builtin() -> None:
         name="Duvadra", model_type="duvadra", config_cls=DuvadraConfig,
         decoder_spec=duvadra.decoder_spec, weight_sources=duvadra.weight_sources,
         ignorable_tensors=duvadra.ignorable_tensors, checkpoint_shapes=duvadra.checkpoint_shapes))
+    from ..models import losorax
+    from .losorax_config import LosoraxConfig
+    register_architecture(Architecture(
+        name="Losorax", model_type="losorax", config_cls=LosoraxConfig,
+        decoder_spec=losorax.decoder_spec, weight_sources=losorax.weight_sources,
+        ignorable_tensors=losorax.ignorable_tensors, checkpoint_shapes=losorax.checkpoint_shapes))
 
 
 _register_builtin()

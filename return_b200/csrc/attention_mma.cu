@@ -14,8 +14,10 @@
 // prompt was cut), and a sliding window bounds the keys from below.
 //
 // The kernels with MOD = true take a ScoreMod: keys bounded from below by the start of the query's own block of
-// `chunk` positions (instead of a window), scores capped softly (cap * tanh(s / cap)) and a penalty per head that
-// grows with the distance, slopes[h] * (i - j), taken off before the softmax.
+// `chunk` positions (instead of a window), scores capped softly (cap * tanh(s / cap)), a penalty per head that
+// grows with the distance, slopes[h] * (i - j), taken off before the softmax, and a bias per head and distance,
+// bias[h, min(i - j, bias_n - 1)], added to the score: a table in global memory that only key tiles within its reach
+// look up; behind it the last entry is a constant.
 //
 // K and V of one layer: [num_pages, Hkv, P, D] bfloat16.  Shared-memory tiles are [rows][D] with
 // the 16-byte chunks of a row XOR-swizzled by the row index, which keeps ldmatrix conflict-free.
@@ -100,11 +102,16 @@ struct ScoreMod {
     float softcap;             // 0: none
     const float* slopes;       // [Hq] or null
     int chunk;                 // 0: none
+    const float* bias;         // [Hq, bias_n] or null
+    int bias_n;
 };
-__device__ __forceinline__ float mod_score(float dot, const ScoreMod& sm, float slope, int dist) {
+// `brow`: the head's row of the bias table for a distance that may lie within it, or null: then `blast` (its last entry,
+// or zero without a table) is added.
+__device__ __forceinline__ float mod_score(float dot, const ScoreMod& sm, float slope, int dist, const float* brow, float blast) {
     float v = dot * sm.scale;
     if (sm.softcap > 0.f) v = sm.softcap * fast_tanh(v / sm.softcap);
     v = fmaf(-slope, (float)dist, v);
+    v += brow != nullptr ? __ldg(brow + min(max(dist, 0), sm.bias_n - 1)) : blast;
     return v * LOG2E;
 }
 
@@ -227,6 +234,8 @@ attn_prefill_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__
     const int lo_r0 = chunk > 0 ? (pos_r0 / chunk) * chunk : 0, lo_r1 = chunk > 0 ? (pos_r1 / chunk) * chunk : 0;
     const int lo_warp = chunk > 0 ? ((p0 + wrow) / chunk) * chunk : 0;     // the lowest bound among the warp's rows
     const float slope = (MOD && sm.slopes) ? sm.slopes[h] : 0.f;
+    const float* bias_row = (MOD && sm.bias) ? sm.bias + (size_t)h * sm.bias_n : nullptr;
+    const float bias_last = (MOD && sm.bias) ? bias_row[sm.bias_n - 1] : 0.f;
 
     for (int jt = jt_begin; jt <= jt_end; ++jt) {
         const int stage = (jt - jt_begin) & 1;
@@ -266,6 +275,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__
                 }
             }
             // scale, mask, running maximum
+            const float* brow = (MOD && p0 + wrow - (j_base + PF_N - 1) < sm.bias_n - 1) ? bias_row : nullptr;
             float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
             for (int nt = 0; nt < PF_N / 8; ++nt) {
@@ -274,7 +284,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__
                     const int j = j_base + nt * 8 + 2 * t4 + (e & 1);
                     const int pr = (e & 2) ? pos_r1 : pos_r0;
                     const bool vis = j <= pr && (window <= 0 || j > pr - window) && (!MOD || j >= ((e & 2) ? lo_r1 : lo_r0));
-                    const float v = !vis ? -INFINITY : MOD ? mod_score(s[nt][e], sm, slope, pr - j) : s[nt][e] * scale_log2;
+                    const float v = !vis ? -INFINITY : MOD ? mod_score(s[nt][e], sm, slope, pr - j, brow, bias_last) : s[nt][e] * scale_log2;
                     s[nt][e] = v;
                     if (e & 2) mx1 = fmaxf(mx1, v); else mx0 = fmaxf(mx0, v);
                 }
@@ -578,6 +588,11 @@ attn_decode_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__ 
     for (int i = 0; i < DTILES; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
 
+    // rows of the bias table of this thread's two query heads (a row that pads the tile takes the first head's)
+    const float* bias0 = (MOD && sm.bias) ? sm.bias + (size_t)(h0 + (g < rows_valid ? g : 0)) * sm.bias_n : nullptr;
+    const float* bias1 = (MOD && sm.bias) ? sm.bias + (size_t)(h0 + (g + 8 < rows_valid ? g + 8 : 0)) * sm.bias_n : nullptr;
+    const float last0 = (MOD && sm.bias) ? bias0[sm.bias_n - 1] : 0.f, last1 = (MOD && sm.bias) ? bias1[sm.bias_n - 1] : 0.f;
+
     int stage = 0, fill_stage = DC_STAGES - 1;
     for (int i = 0; i < n_my; ++i) {
         if (i + DC_STAGES - 1 < n_my) issue(i + DC_STAGES - 1, fill_stage);
@@ -605,12 +620,15 @@ attn_decode_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__ 
         if (MOD) {
             const float sl0 = (sm.slopes && g < rows_valid) ? sm.slopes[h0 + g] : 0.f;
             const float sl1 = (sm.slopes && g + 8 < rows_valid) ? sm.slopes[h0 + g + 8] : 0.f;
+            const bool near = hi - (j_base + DC_N - 1) < sm.bias_n - 1;           // the tile holds distances within the table
+            const float* br0 = near ? bias0 : nullptr;
+            const float* br1 = near ? bias1 : nullptr;
 #pragma unroll
             for (int nt = 0; nt < 2; ++nt) {
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int j = j_base + nt * 8 + 2 * t4 + (e & 1);
-                    const float v = (j >= lo && j <= hi) ? mod_score(s[nt][e] + s2[nt][e], sm, (e & 2) ? sl1 : sl0, hi - j) : -INFINITY;
+                    const float v = (j >= lo && j <= hi) ? mod_score(s[nt][e] + s2[nt][e], sm, (e & 2) ? sl1 : sl0, hi - j, (e & 2) ? br1 : br0, (e & 2) ? last1 : last0) : -INFINITY;
                     s[nt][e] = v;
                     if (e & 2) mx1 = fmaxf(mx1, v); else mx0 = fmaxf(mx0, v);
                 }
@@ -799,14 +817,15 @@ attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ 
 
 RB_EXPORT int rb_attn_head_dim() { return D; }
 
-// softcap 0, slopes null and chunk 0: the plain kernel; anything else: the MOD kernel (a window and a chunk exclude
+// softcap 0, slopes null, bias null and chunk 0: the plain kernel; anything else: the MOD kernel (a window and a chunk exclude
 // each other).
 RB_EXPORT int rb_attn_prefill_mod(const void* q, int ld, const void* kpool, const void* vpool, const int* tiles,
                                   int n_tiles, const int* cu_q, const int* seg_pos0, const int* block_table,
                                   int bt_stride, int page_size, void* out, int Hq, int Hkv, float scale,
                                   int window, const float* sink, int chunk, float softcap, const float* slopes,
-                                  cudaStream_t st) {
+                                  const float* bias, int bias_n, cudaStream_t st) {
     if (n_tiles <= 0) return 0;
+    if (bias != nullptr && bias_n < 1) return (int)cudaErrorInvalidValue;
     if (window > 0 && chunk > 0) return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)(PF_M + 4 * PF_N) * D * sizeof(bf16) + BT_CAP * sizeof(int);
     static PerDevice configured;
@@ -818,8 +837,8 @@ RB_EXPORT int rb_attn_prefill_mod(const void* q, int ld, const void* kpool, cons
     if (cfg != 0) return cfg;
     dim3 grid(n_tiles, Hq);
     ScoreMod sm;
-    sm.scale = scale; sm.softcap = softcap; sm.slopes = slopes; sm.chunk = chunk;
-    if (chunk > 0 || softcap > 0.f || slopes != nullptr)
+    sm.scale = scale; sm.softcap = softcap; sm.slopes = slopes; sm.chunk = chunk; sm.bias = bias; sm.bias_n = bias ? bias_n : 0;
+    if (chunk > 0 || softcap > 0.f || slopes != nullptr || bias != nullptr)
         return rb_launch_pdl(attn_prefill_kernel<true>, grid, dim3(128), smem, st, (const bf16*)q, ld, (const bf16*)kpool,
                              (const bf16*)vpool, tiles, cu_q, seg_pos0, block_table, bt_stride, page_size, (bf16*)out,
                              Hq, Hkv, scale * LOG2E, window, sink, sm);
@@ -833,7 +852,7 @@ RB_EXPORT int rb_attn_prefill(const void* q, int ld, const void* kpool, const vo
                               int bt_stride, int page_size, void* out, int Hq, int Hkv, float scale,
                               int window, const float* sink, cudaStream_t st) {
     return rb_attn_prefill_mod(q, ld, kpool, vpool, tiles, n_tiles, cu_q, seg_pos0, block_table, bt_stride, page_size, out,
-                               Hq, Hkv, scale, window, sink, 0, 0.f, nullptr, st);
+                               Hq, Hkv, scale, window, sink, 0, 0.f, nullptr, nullptr, 0, st);
 }
 
 // Floats of scratch that rb_attn_decode needs: part_o [n_dec, Hq, splits, D], part_ml [n_dec, Hq, splits, 2].
@@ -901,13 +920,13 @@ RB_EXPORT int rb_attn_decode_mod(const void* q, int ld, const void* kpool, const
                                  int n_dec, const int* cu_q, const int* seg_kv_len, const int* block_table,
                                  int bt_stride, int page_size, float* scratch, void* out, int Hq, int Hkv,
                                  float scale, int window, int num_splits, const float* sink, int chunk, float softcap,
-                                 const float* slopes, cudaStream_t st) {
-    if (window > 0 && chunk > 0) return (int)cudaErrorInvalidValue;
-    if (chunk <= 0 && softcap <= 0.f && slopes == nullptr)
+                                 const float* slopes, const float* bias, int bias_n, cudaStream_t st) {
+    if ((window > 0 && chunk > 0) || (bias != nullptr && bias_n < 1)) return (int)cudaErrorInvalidValue;
+    if (chunk <= 0 && softcap <= 0.f && slopes == nullptr && bias == nullptr)
         return launch_decode(q, ld, kpool, vpool, dec_segs, n_dec, cu_q, seg_kv_len, block_table, bt_stride, page_size,
                              scratch, out, Hq, Hkv, scale, window, num_splits, nullptr, sink, st);
     ScoreMod sm;
-    sm.scale = scale; sm.softcap = softcap; sm.slopes = slopes; sm.chunk = chunk;
+    sm.scale = scale; sm.softcap = softcap; sm.slopes = slopes; sm.chunk = chunk; sm.bias = bias; sm.bias_n = bias ? bias_n : 0;
     return launch_decode(q, ld, kpool, vpool, dec_segs, n_dec, cu_q, seg_kv_len, block_table, bt_stride, page_size,
                          scratch, out, Hq, Hkv, scale, window, num_splits, nullptr, sink, st, &sm);
 }

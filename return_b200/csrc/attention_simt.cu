@@ -14,8 +14,9 @@
 //
 // Options of the score, all off by default: `chunk` > 0 bounds the keys from below by the start of the query's own
 // block of `chunk` positions (blocks counted from position 0) instead of a window; `softcap` > 0 turns a scaled score
-// s into softcap * tanh(s / softcap); `slopes` [Hq] takes slopes[h] * (p - j) off the score of key j; `sink` [Hq] adds
-// exp(sink[h]) to the softmax's denominator (a term with no key and no value).
+// s into softcap * tanh(s / softcap); `slopes` [Hq] takes slopes[h] * (p - j) off the score of key j; `bias` [Hq, bias_n] adds
+// bias[h, min(p - j, bias_n - 1)] to it; `sink` [Hq] adds exp(sink[h]) to the softmax's denominator (a term with no key and
+// no value).
 #include "common.cuh"
 
 #define SIMT_MAX_D 256
@@ -27,7 +28,7 @@ attention_simt_kernel(const TA* __restrict__ q, int ld, const TA* __restrict__ k
                       const int* __restrict__ tok_seg, const int* __restrict__ block_table,
                       int bt_stride, int page_size, TA* __restrict__ out, int Hq, int Hkv, int D,
                       float scale, int window, int chunk, float softcap, const float* __restrict__ slopes,
-                      const float* __restrict__ sink) {
+                      const float* __restrict__ sink, const float* __restrict__ bias, int bias_n) {
     extern __shared__ float qs_all[];                    // 4 warps x D floats
     const int t = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -64,6 +65,7 @@ attention_simt_kernel(const TA* __restrict__ q, int ld, const TA* __restrict__ k
                 s = dot * scale;
                 if (softcap > 0.f) s = softcap * tanhf(s / softcap);
                 if (slopes) s -= slope * (float)(p - j);
+                if (bias) s += bias[(size_t)h * bias_n + min(p - j, bias_n - 1)];
             }
         }
         const float m_new = fmaxf(m, warp_max(s));
@@ -101,8 +103,9 @@ RB_EXPORT int rb_attention_simt_mod(const void* q, int ld, const void* kpool, co
                                 const int* pos, const int* tok_seg, const int* block_table,
                                 int bt_stride, int page_size, void* out, int act_dtype, int T,
                                 int Hq, int Hkv, int D, float scale, int window, int chunk, float softcap,
-                                const float* slopes, const float* sink, cudaStream_t st) {
+                                const float* slopes, const float* sink, const float* bias, int bias_n, cudaStream_t st) {
     if (T <= 0) return 0;
+    if (bias != nullptr && bias_n < 1) return (int)cudaErrorInvalidValue;
     if (window > 0 && chunk > 0) return (int)cudaErrorInvalidValue;
     if (D > SIMT_MAX_D || D <= 0 || Hkv <= 0 || Hq % Hkv) return (int)cudaErrorInvalidValue;
     dim3 grid(T, (Hq + 3) / 4);
@@ -110,11 +113,11 @@ RB_EXPORT int rb_attention_simt_mod(const void* q, int ld, const void* kpool, co
     if (act_dtype == RB_F32)
         attention_simt_kernel<float><<<grid, 128, smem, st>>>(
             (const float*)q, ld, (const float*)kpool, (const float*)vpool, pos, tok_seg, block_table,
-            bt_stride, page_size, (float*)out, Hq, Hkv, D, scale, window, chunk, softcap, slopes, sink);
+            bt_stride, page_size, (float*)out, Hq, Hkv, D, scale, window, chunk, softcap, slopes, sink, bias, bias_n);
     else
         attention_simt_kernel<bf16><<<grid, 128, smem, st>>>(
             (const bf16*)q, ld, (const bf16*)kpool, (const bf16*)vpool, pos, tok_seg, block_table,
-            bt_stride, page_size, (bf16*)out, Hq, Hkv, D, scale, window, chunk, softcap, slopes, sink);
+            bt_stride, page_size, (bf16*)out, Hq, Hkv, D, scale, window, chunk, softcap, slopes, sink, bias, bias_n);
     return rb_launch_status();
 }
 
@@ -123,5 +126,5 @@ RB_EXPORT int rb_attention_simt(const void* q, int ld, const void* kpool, const 
                                 int bt_stride, int page_size, void* out, int act_dtype, int T,
                                 int Hq, int Hkv, int D, float scale, int window, cudaStream_t st) {
     return rb_attention_simt_mod(q, ld, kpool, vpool, pos, tok_seg, block_table, bt_stride, page_size, out, act_dtype, T,
-                                 Hq, Hkv, D, scale, window, 0, 0.f, nullptr, nullptr, st);
+                                 Hq, Hkv, D, scale, window, 0, 0.f, nullptr, nullptr, nullptr, 0, st);
 }

@@ -36,8 +36,10 @@
 // rotated, tiles are aligned to absolute positions, a sliding window bounds the keys from below.
 //
 // The kernel with MOD = true takes a ScoreMod: keys bounded from below by the start of the query's own block of
-// `chunk` positions (instead of a window), scores capped softly (cap * tanh(s / cap)) and a penalty per head that grows
-// with the distance, slopes[h] * (i - j), taken off before the softmax.  A row's thread does that to its 64 scores
+// `chunk` positions (instead of a window), scores capped softly (cap * tanh(s / cap)), a penalty per head that grows
+// with the distance, slopes[h] * (i - j), taken off before the softmax, and a bias per head and distance added to the
+// score, bias[h, min(i - j, bias_n - 1)]: only key tiles within the table's reach look it up (neighbouring rows read
+// neighbouring entries), behind it the last entry is a constant.  A row's thread does that to its 64 scores
 // of a key tile right after it has read them from tensor memory; everything else is the plain kernel.
 // A step with too few such CTAs to fill the GPU (a short portion of a long prompt) splits the keys of every
 // block over gridDim.z CTAs; each leaves its unnormalised O with its reference maximum and sum in float32,
@@ -144,6 +146,8 @@ struct ScoreMod {
     float softcap;             // 0: none
     const float* slopes;       // [Hq] or null
     int chunk;                 // 0: none
+    const float* bias;         // [Hq, bias_n] or null
+    int bias_n;
 };
 
 template <bool MOD>
@@ -227,6 +231,8 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
         const float scale_eff = MOD ? 1.f : scale_log2;                        // the MOD rows hold finished exponents
         const float cap_l = MOD ? sm.softcap * LOG2E : 0.f, slope_l = slope * LOG2E;
         const float k_tanh = (MOD && sm.softcap > 0.f) ? sm.scale / sm.softcap * (2.0f * LOG2E) : 0.f;
+        const float* bias_row = (MOD && sm.bias) ? sm.bias + (size_t)h * sm.bias_n : nullptr;
+        const float bias_last_l = (MOD && sm.bias) ? bias_row[sm.bias_n - 1] * LOG2E : 0.f;
         unsigned char* myQ = sQ + qt * Q_BYTES;
         unsigned char* myPs = sP + qt * 2 * P_BYTES;           // this query tile's two P buffers
         {
@@ -260,7 +266,8 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
                 // the finished exponent of key j = j_base + i, in units of log2:
                 //   cap L tanh(s scale / cap) - slope L (pos - j)  =  cap L - 2 cap L / (e^(2 s scale / cap) + 1) + slope L i - slope L (pos - j_base)
                 // with L = log2(e): one product, 2^x, one sum, a reciprocal and two fused products a score
-                const float c0 = cap_l - slope_l * (float)(pos_r - j_base);
+                const bool near = sm.bias != nullptr && p0_t - (j_base + KN - 1) < sm.bias_n - 1;   // the tile holds distances within the table
+                const float c0 = cap_l - slope_l * (float)(pos_r - j_base) + (near ? 0.f : bias_last_l);
                 if (sm.softcap > 0.f) {
 #pragma unroll
                     for (int i = 0; i < 64; ++i) {
@@ -274,6 +281,12 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
 #pragma unroll
                     for (int i = 0; i < 64; ++i)
                         a[i] = __float_as_uint(fmaf(__uint_as_float(a[i]), sm.scale * LOG2E, fmaf(slope_l, (float)i, c0)));
+                }
+                if (near) {
+                    const int d0 = pos_r - j_base;
+#pragma unroll
+                    for (int i = 0; i < 64; ++i)
+                        a[i] = __float_as_uint(fmaf(__ldg(bias_row + min(max(d0 - i, 0), sm.bias_n - 1)), LOG2E, __uint_as_float(a[i])));
                 }
                 if (all_visible) {
 #pragma unroll
@@ -603,13 +616,15 @@ RB_EXPORT long long rb_attn_tc5_split_floats(int n_split, int total_rows, int Hq
 // tiles: [n_tiles, 2] = (segment, first row of a block of up to 256 query rows), the blocks with the
 // longest contexts first.  n_split > 1 splits the keys of every block over that many CTAs; ``scratch`` then
 // holds rb_attn_tc5_split_floats(...) floats and total_rows is the number of rows of q.
-// chunk, softcap, slopes: the score options (0, 0, null: the plain kernel); a window and a chunk exclude each other.
+// chunk, softcap, slopes, bias: the score options (0, 0, null, null: the plain kernel); a window and a chunk exclude each other.
 RB_EXPORT int rb_attn_prefill_tc5_mod(const void* q, int ld, const void* kpool, const void* vpool, const int* tiles,
                                       int n_tiles, const int* cu_q, const int* seg_pos0, const int* block_table,
                                       int bt_stride, int page_size, void* out, int Hq, int Hkv, float scale, int window,
                                       int n_split, void* scratch, int total_rows, int* status, const float* sink,
-                                      int chunk, float softcap, const float* slopes, cudaStream_t st) {
+                                      int chunk, float softcap, const float* slopes, const float* bias, int bias_n,
+                                      cudaStream_t st) {
     if (n_tiles <= 0) return 0;
+    if (bias != nullptr && bias_n < 1) return (int)cudaErrorInvalidValue;
     if (n_tiles > 65535 || n_split < 1 || n_split > 64 || (n_split > 1 && scratch == nullptr)) return (int)cudaErrorInvalidValue;
     if (window > 0 && chunk > 0) return (int)cudaErrorInvalidValue;
     static PerDevice configured;
@@ -623,8 +638,8 @@ RB_EXPORT int rb_attn_prefill_tc5_mod(const void* q, int ld, const void* kpool, 
     float* part_ml = part_o ? part_o + (size_t)n_split * total_rows * Hq * D : nullptr;
     dim3 grid(Hq, n_tiles, n_split);
     ScoreMod sm;
-    sm.scale = scale; sm.softcap = softcap; sm.slopes = slopes; sm.chunk = chunk;
-    if (chunk > 0 || softcap > 0.f || slopes != nullptr)
+    sm.scale = scale; sm.softcap = softcap; sm.slopes = slopes; sm.chunk = chunk; sm.bias = bias; sm.bias_n = bias ? bias_n : 0;
+    if (chunk > 0 || softcap > 0.f || slopes != nullptr || bias != nullptr)
         attn_prefill_tc5_kernel<true><<<grid, THREADS, SMEM_BYTES, st>>>(
             (const bf16*)q, ld, (const bf16*)kpool, (const bf16*)vpool, tiles, cu_q, seg_pos0, block_table, bt_stride,
             page_size, (bf16*)out, Hq, Hkv, scale * LOG2E, window, part_o, part_ml, total_rows, status, sink, sm);
@@ -645,5 +660,5 @@ RB_EXPORT int rb_attn_prefill_tc5(const void* q, int ld, const void* kpool, cons
                                   int n_split, void* scratch, int total_rows, int* status, const float* sink,
                                   cudaStream_t st) {
     return rb_attn_prefill_tc5_mod(q, ld, kpool, vpool, tiles, n_tiles, cu_q, seg_pos0, block_table, bt_stride, page_size, out,
-                                   Hq, Hkv, scale, window, n_split, scratch, total_rows, status, sink, 0, 0.f, nullptr, st);
+                                   Hq, Hkv, scale, window, n_split, scratch, total_rows, status, sink, 0, 0.f, nullptr, nullptr, 0, st);
 }

@@ -10,7 +10,8 @@
 // One warp a token.  s = softmax(z + bias) over all experts (float32; the bias per expert may be absent).  With groups > 1 the experts form `groups` equal
 // runs of neighbours, a group's score is its largest s, and only experts of the `keep` best groups can be chosen.
 // The `top` largest s among those are chosen (the lower index on a tie); weight = s / (sum of the chosen s + tiny),
-// which with tiny = 0 is the softmax over the chosen logits alone.
+// which with tiny = 0 is the softmax over the chosen logits alone; without `renorm` weight = s as it is.  Either times
+// out_scale.
 __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
@@ -23,7 +24,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ z, int ldz, const float* __restrict__ bias, int* __restrict__ expert_of,
                  float* __restrict__ weight, int T, int E, int top, int groups, int keep, float tiny, int score_fn,
-                 int group_top, float out_scale) {
+                 int group_top, float out_scale, int renorm) {
     extern __shared__ float route_smem[];                 // per warp: E scores, then `groups` group scores
     pdl_launch_dependents();
     pdl_wait();
@@ -94,13 +95,14 @@ moe_route_kernel(const float* __restrict__ z, int ldz, const float* __restrict__
         total += bv;
         __syncwarp();
     }
-    const float scale = out_scale / (total + tiny);
+    const float scale = renorm ? out_scale / (total + tiny) : out_scale;
     __syncwarp();
     for (int k = lane; k < top; k += 32) weight[(size_t)t * top + k] *= scale;
 }
 
 RB_EXPORT int rb_moe_route(const float* z, int ldz, const float* bias, int* expert_of, float* weight, int T, int E, int top,
-                           int groups, int keep, float tiny, int score_fn, int group_top, float out_scale, cudaStream_t st) {
+                           int groups, int keep, float tiny, int score_fn, int group_top, float out_scale, int renorm,
+                           cudaStream_t st) {
     if (T <= 0) return 0;
     if (score_fn < 0 || score_fn > 1 || group_top < 1 || group_top > 2) return (int)cudaErrorInvalidValue;
     if (groups < 1 || E % groups || top < 1 || top > E || keep < 1 || keep > groups || (long long)keep * (E / groups) < top)
@@ -108,7 +110,7 @@ RB_EXPORT int rb_moe_route(const float* z, int ldz, const float* bias, int* expe
     const size_t smem = (size_t)4 * (E + groups) * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     return rb_launch_pdl(moe_route_kernel, dim3((T + 3) / 4), dim3(128), smem, st, z, ldz, bias, expert_of, weight, T, E, top,
-                         groups, keep, tiny, score_fn, group_top, out_scale);
+                         groups, keep, tiny, score_fn, group_top, out_scale, renorm);
 }
 
 // ---------------------------------------------------------------- a pair's product, weights streamed
@@ -216,24 +218,29 @@ RB_EXPORT int rb_moe_pair_linear(const void* x, int ldx, int in_div, const void*
 // ---------------------------------------------------------------- the gated unit with a capped gate
 // in[r] = [gate (F numbers) | up (F numbers)];  g = min(gate, limit), u = clamp(up, -limit, limit);
 // out[r, f] = g * sigmoid(alpha * g) * (u + shift).  float32 arithmetic, one rounding at the store.  An infinite limit,
-// alpha = 1 and shift = 0 make it silu(gate) * up.
+// alpha = 1 and shift = 0 make it silu(gate) * up.  With `weight` the row's gate and up numbers are first multiplied by a
+// number of its pair (pair_at[r], or r): as the two products are linear, that is the expert run on its input times the
+// pair's weight.
 template <typename TA>
 __global__ void clamped_glu_kernel(const TA* __restrict__ in, int ldi, TA* __restrict__ out, int ldo, int F, float limit,
-                                   float alpha, float shift, long long total) {
+                                   float alpha, float shift, const float* __restrict__ weight, const int* __restrict__ pair_at,
+                                   long long total) {
     pdl_launch_dependents();
     pdl_wait();
     for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (long long)gridDim.x * blockDim.x) {
         const long long r = e / F;
         const int f = (int)(e % F);
-        const float g = fminf(to_f32(in[r * ldi + f]), limit);
-        const float u = fminf(fmaxf(to_f32(in[r * ldi + F + f]), -limit), limit);
+        const float c = weight ? weight[pair_at ? pair_at[r] : r] : 1.f;
+        const float g = fminf(c * to_f32(in[r * ldi + f]), limit);
+        const float u = fminf(fmaxf(c * to_f32(in[r * ldi + F + f]), -limit), limit);
         out[r * ldo + f] = from_f32<TA>(g / (1.0f + expf(-alpha * g)) * (u + shift));
     }
 }
 
 // bfloat16 with F a multiple of 8: eight outputs (two 16-byte loads, one store) a thread and step.
 __global__ void clamped_glu_bf16x8_kernel(const bf16* __restrict__ in, int ldi, bf16* __restrict__ out, int ldo, int F8,
-                                          float limit, float alpha, float shift, unsigned total) {
+                                          float limit, float alpha, float shift, const float* __restrict__ weight,
+                                          const int* __restrict__ pair_at, unsigned total) {
     pdl_launch_dependents();
     pdl_wait();
     for (unsigned e = blockIdx.x * blockDim.x + threadIdx.x; e < total; e += gridDim.x * blockDim.x) {
@@ -242,12 +249,13 @@ __global__ void clamped_glu_bf16x8_kernel(const bf16* __restrict__ in, int ldi, 
         const uint4 uv = *reinterpret_cast<const uint4*>(in + (size_t)r * ldi + F8 * 8 + f);
         const bf16* g8 = reinterpret_cast<const bf16*>(&gv);
         const bf16* u8 = reinterpret_cast<const bf16*>(&uv);
+        const float c = weight ? weight[pair_at ? pair_at[r] : r] : 1.f;
         uint4 ov;
         bf16* o8 = reinterpret_cast<bf16*>(&ov);
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
-            const float g = fminf(__bfloat162float(g8[k]), limit);
-            const float u = fminf(fmaxf(__bfloat162float(u8[k]), -limit), limit);
+            const float g = fminf(c * __bfloat162float(g8[k]), limit);
+            const float u = fminf(fmaxf(c * __bfloat162float(u8[k]), -limit), limit);
             o8[k] = __float2bfloat16_rn(g / (1.0f + expf(-alpha * g)) * (u + shift));
         }
         *reinterpret_cast<uint4*>(out + (size_t)r * ldo + f) = ov;
@@ -255,7 +263,7 @@ __global__ void clamped_glu_bf16x8_kernel(const bf16* __restrict__ in, int ldi, 
 }
 
 RB_EXPORT int rb_clamped_glu(const void* in, int ldi, void* out, int ldo, int act_dtype, int rows, int F, float limit,
-                             float alpha, float shift, cudaStream_t st) {
+                             float alpha, float shift, const float* weight, const int* pair_at, cudaStream_t st) {
     const long long total = (long long)rows * F;
     if (total <= 0) return 0;
     if (act_dtype == RB_BF16 && F % 8 == 0 && ldi % 8 == 0 && ldo % 8 == 0 && ((uintptr_t)in % 16) == 0 &&
@@ -263,19 +271,19 @@ RB_EXPORT int rb_clamped_glu(const void* in, int ldi, void* out, int ldo, int ac
         const unsigned items = (unsigned)(total / 8);
         const int nblocks = (int)min((unsigned)(148 * 16), (items + 255) / 256);
         return rb_launch_pdl(clamped_glu_bf16x8_kernel, dim3(nblocks), dim3(256), 0, st, (const bf16*)in, ldi, (bf16*)out, ldo,
-                             F / 8, limit, alpha, shift, items);
+                             F / 8, limit, alpha, shift, weight, pair_at, items);
     }
     const int blocks = (int)min((long long)4096, (total + 255) / 256);
     if (act_dtype == RB_F32)
         return rb_launch_pdl(clamped_glu_kernel<float>, dim3(blocks), dim3(256), 0, st, (const float*)in, ldi, (float*)out, ldo, F,
-                             limit, alpha, shift, total);
+                             limit, alpha, shift, weight, pair_at, total);
     return rb_launch_pdl(clamped_glu_kernel<bf16>, dim3(blocks), dim3(256), 0, st, (const bf16*)in, ldi, (bf16*)out, ldo, F, limit,
-                         alpha, shift, total);
+                         alpha, shift, weight, pair_at, total);
 }
 
 // ---------------------------------------------------------------- the weighted sum of a token's experts
 // out[t, :] = sum_k weight[t, k] * y[row_of ? row_of[t * top + k] : t * top + k, :]  (+ shared[t, :]), k ascending, float32
-// sums.  row_of: where a pair's row lies when the pairs were put in the order of their experts.
+// sums.  row_of: where a pair's row lies when the pairs were put in the order of their experts.  weight null: a plain sum.
 template <typename TA>
 __global__ void moe_combine_kernel(const TA* __restrict__ y, const int* __restrict__ row_of, const float* __restrict__ weight,
                                    const TA* __restrict__ shared, TA* __restrict__ out, int H, int top) {
@@ -287,7 +295,7 @@ __global__ void moe_combine_kernel(const TA* __restrict__ y, const int* __restri
         for (int k = 0; k < top; ++k) {
             const int pair = t * top + k;
             const size_t row = row_of ? (size_t)row_of[pair] : (size_t)pair;
-            acc = fmaf(weight[pair], to_f32(y[row * H + i]), acc);
+            acc = fmaf(weight ? weight[pair] : 1.f, to_f32(y[row * H + i]), acc);
         }
         if (shared != nullptr) acc += to_f32(shared[(size_t)t * H + i]);
         out[(size_t)t * H + i] = from_f32<TA>(acc);

@@ -6,6 +6,8 @@
 //     fixed decay:     S <- a S + k v^T                                   o = S^T q
 //     delta rule:      S <- g * S (row i by g_i);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //     delta rule, one decay a head: the same with a scalar g per token and head
+//     general delta:   S <- g * S (row i by g_i) - c (k^T S) + k v^T, both terms of the old S;  o = S^T q: the removal has a
+//                      vector c of its own (per token, head and key row) instead of running along the key
 //     matrix memory:   m' = max(f + m, i);  a = exp(f + m - m'),  b = exp(i - m');
 //                      S <- a S + b k v^T;  n <- a n + b k;  o = S^T q / (max(|n . q|, exp(-m')) + 1e-6)
 //     bonus rule:      o = (S + diag(u) k v^T)^T q;  S <- g * S (row i by g_i) + k v^T: the token's own pair is read with
@@ -37,15 +39,17 @@
 #define MODE_BONUS 3
 #define MODE_SSM 4
 #define MODE_DELTA_HEAD 5
+#define MODE_GENERAL_DELTA 6
 
 struct ScanArgs {
     const void* q; const void* k; const void* v;        // (t, head, i) at base + t * ld + head * dim + i
     int q_ld, k_ld, v_ld;
     int q_f32, k_f32, v_f32;                            // 1: float32, 0: bfloat16
-    const float* gate_a;      // decay: [H] decays; memory: [T, 2H] gate pre-activations (input, forget); delta and bonus:
-                              // [T, H*D] row decays; state space: [T, H] decays
+    const float* gate_a;      // decay: [H] decays; memory: [T, 2H] gate pre-activations (input, forget); delta, general delta
+                              // and bonus: [T, H*D] row decays; state space: [T, H] decays
     const float* gate_b;      // memory: [2H] gate biases; delta: [T, H] beta; state space: [T, H] steps
                               // delta with one decay a head: gate_a [T, H] decays, gate_b [T, H] beta
+                              // general delta: gate_b [T, H*D] removal vectors
     const float* extra;       // bonus: [H, D] weights of the token's own pair; state space: [H] skip weights
     float cap, q_scale;
     float* state;             // [slots, state_stride]
@@ -82,12 +86,14 @@ linear_scan_kernel(const ScanArgs a) {
     // NR values as 16-byte pieces, and the eight runs that one such request covers fall on different banks
     constexpr int RS = NR + 4, DS = R * RS;
     constexpr int PER = SCAN_TC * DP / SCAN_THREADS;   // q (and k) elements of a chunk that a thread brings in
-    constexpr bool ROW_DECAY = MODE == MODE_DELTA || MODE == MODE_BONUS;     // a decay per token, head and key row
+    constexpr bool ROW_REMOVAL = MODE == MODE_GENERAL_DELTA;                 // a removal vector per token and head
+    constexpr bool ROW_DECAY = MODE == MODE_DELTA || MODE == MODE_BONUS || ROW_REMOVAL;      // a decay per token, head and key row
     static_assert(SCAN_TC * SCAN_COLS <= SCAN_THREADS && (SCAN_TC * DP) % SCAN_THREADS == 0, "staging by all threads");
     pdl_wait();
     __shared__ __align__(16) float sq[SCAN_TC][DS];
     __shared__ __align__(16) float sk[SCAN_TC][DS];
     __shared__ __align__(16) float sg[ROW_DECAY ? SCAN_TC : 1][DS];
+    __shared__ __align__(16) float sc[ROW_REMOVAL ? SCAN_TC : 1][ROW_REMOVAL ? DS : 4];
     __shared__ float sv[SCAN_TC][SCAN_COLS];
     __shared__ float sa[SCAN_TC], sb[SCAN_TC];
     const int seg = blockIdx.z, h = blockIdx.y, j0 = blockIdx.x * SCAN_COLS;
@@ -133,7 +139,7 @@ linear_scan_kernel(const ScanArgs a) {
     // product right behind a load would make the warp wait for it there, before the arithmetic it is meant to hide
     // behind.  Converting, scaling and the gates' transcendental functions happen on the way to shared memory.
     uint32_t rq[PER], rk[PER], rv = 0u;
-    float rg[ROW_DECAY ? PER : 1], ra = 0.f, rb = 0.f;
+    float rg[ROW_DECAY ? PER : 1], rc[ROW_REMOVAL ? PER : 1], ra = 0.f, rb = 0.f;
     auto raw = [](const void* p, int f32, size_t i) -> uint32_t {
         return f32 ? ((const uint32_t*)p)[i] : (uint32_t)((const unsigned short*)p)[i];
     };
@@ -148,6 +154,7 @@ linear_scan_kernel(const ScanArgs a) {
             rq[u] = live ? raw(a.q, a.q_f32, t * a.q_ld + (size_t)kvh * D + i) : 0u;
             rk[u] = live ? raw(a.k, a.k_f32, t * a.k_ld + (size_t)kvh * D + i) : 0u;
             if (ROW_DECAY) rg[u] = live ? a.gate_a[(t * H + h) * D + i] : 1.f;
+            if (ROW_REMOVAL) rc[u] = live ? a.gate_b[(t * H + h) * D + i] : 0.f;
         }
         if (tid < SCAN_TC * SCAN_COLS) {
             const int tt = tid / SCAN_COLS, c = tid - tt * SCAN_COLS;
@@ -174,6 +181,7 @@ linear_scan_kernel(const ScanArgs a) {
             sq[tt][at] = cooked(rq[u], a.q_f32) * a.q_scale;
             sk[tt][at] = cooked(rk[u], a.k_f32);
             if (ROW_DECAY) sg[tt][at] = rg[u];
+            if (ROW_REMOVAL) sc[tt][at] = rc[u];
         }
         if (tid < SCAN_TC * SCAN_COLS) sv[tid / SCAN_COLS][tid % SCAN_COLS] = cooked(rv, a.v_f32);
         if (tid < SCAN_TC) {
@@ -239,6 +247,30 @@ linear_scan_kernel(const ScanArgs a) {
             for (int ii = 0; ii < NR; ++ii) {
                 S[ii] = fmaf(fa, S[ii], kr[ii] * vdt);
                 o4[ii & 3] = fmaf(S[ii], qr[ii], o4[ii & 3]);
+            }
+        } else if (MODE == MODE_GENERAL_DELTA) {
+            // what the old state holds for the key; the decay and the new pair do not wait for the sum over the lanes
+            float k4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int i4 = 0; i4 < NR; i4 += 4) {
+                const float4 g4 = *(const float4*)&sg[tt][r * RS + i4];
+                const float gr[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    k4[i] = fmaf(S[i4 + i], kr[i4 + i], k4[i]);
+                    S[i4 + i] = fmaf(gr[i], S[i4 + i], kr[i4 + i] * vj);
+                }
+            }
+            const float kv = lanes_sum<R>((k4[0] + k4[1]) + (k4[2] + k4[3]));
+#pragma unroll
+            for (int i4 = 0; i4 < NR; i4 += 4) {
+                const float4 c4 = *(const float4*)&sc[tt][r * RS + i4];
+                const float cr[4] = {c4.x, c4.y, c4.z, c4.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    S[i4 + i] = fmaf(-cr[i], kv, S[i4 + i]);
+                    o4[i] = fmaf(S[i4 + i], qr[i4 + i], o4[i]);
+                }
             }
         } else {
             if (MODE == MODE_DELTA_HEAD) {
@@ -335,8 +367,8 @@ static int launch_scan(const ScanArgs& a, int segments, cudaStream_t st) {
     return rb_launch_pdl(linear_scan_kernel<MODE, 32, R>, grid, dim3(SCAN_THREADS), 0, st, a);
 }
 
-// mode: 0 fixed decay, 1 matrix memory, 2 delta rule, 3 bonus rule, 4 state space.  The arguments are those of
-// ScanArgs, in its order.
+// mode: 0 fixed decay, 1 matrix memory, 2 delta rule, 3 bonus rule, 4 state space, 5 delta rule with one decay a head,
+// 6 general delta.  The arguments are those of ScanArgs, in its order.
 RB_EXPORT int rb_linear_scan(int mode, const void* q, const void* k, const void* v, int q_ld, int k_ld, int v_ld,
                              int q_f32, int k_f32, int v_f32, const float* gate_a, const float* gate_b,
                              const float* extra, float cap,
@@ -355,6 +387,7 @@ RB_EXPORT int rb_linear_scan(int mode, const void* q, const void* k, const void*
     if (mode == MODE_BONUS) return extra ? launch_scan<MODE_BONUS>(a, segments, st) : (int)cudaErrorInvalidValue;
     if (mode == MODE_SSM) return extra && gate_b ? launch_scan<MODE_SSM>(a, segments, st) : (int)cudaErrorInvalidValue;
     if (mode == MODE_DELTA_HEAD) return gate_b ? launch_scan<MODE_DELTA_HEAD>(a, segments, st) : (int)cudaErrorInvalidValue;
+    if (mode == MODE_GENERAL_DELTA) return gate_b ? launch_scan<MODE_GENERAL_DELTA>(a, segments, st) : (int)cudaErrorInvalidValue;
     return (int)cudaErrorInvalidValue;
 }
 
@@ -666,6 +699,57 @@ RB_EXPORT int rb_delta_prep(const void* x, int ld, const void* taps, int taps_dt
         rb_launch_pdl(delta_prep_kernel<bf16>, dim3(grid), dim3(128), 0, st, (const bf16*)x, ld, taps, taps_dtype, K, state, state_stride, conv_off,
             tok_seg, cu_q, seg_slot, q32, k32, v32, a, A_log, dt_bias, vec_dtype, b, H, G, D, V, q_scale, DA);
     return rb_launch_status();
+}
+
+// ---------------------------------------------------------------- what the general delta rule needs of a token
+// Per (token, head), one warp, in float32:
+//   decay[t, h, i] = exp(-scale * sigmoid(decay[t, h, i] + w0[h, i]))              (in place over the projection's output)
+//   removal[t, h, i] = sigmoid(a[t, h, i] + a_bias[h, i]) * k[t, h, i] / (sum_i k^2 + unit_eps)
+// With u = k / sqrt(sum k^2 + unit_eps) the scan's removal (rate * u)(u^T S) is removal (k^T S).  k and a are runs of
+// columns of the projection rows.
+template <typename TA>
+__global__ void __launch_bounds__(128)
+general_delta_prep_kernel(const TA* __restrict__ proj, int ld, int k_off, int a_off, const void* __restrict__ a_bias,
+                          const void* __restrict__ w0, int vec_dtype, float scale, float unit_eps, float* __restrict__ decay,
+                          float* __restrict__ removal, int rows, int H, int D) {
+    pdl_wait();
+    const int row = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+    if (row >= rows) return;
+    const int t = row / H, h = row - t * H;
+    const TA* k = proj + (size_t)t * ld + k_off + (size_t)h * D;
+    const TA* a = proj + (size_t)t * ld + a_off + (size_t)h * D;
+    float* dc = decay + (size_t)row * D;
+    float* rm = removal + (size_t)row * D;
+    float kv[8], ss = 0.f;                                // up to 256 key rows
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+        const int i = lane + 32 * u;
+        kv[u] = i < D ? to_f32(k[i]) : 0.f;
+        ss = fmaf(kv[u], kv[u], ss);
+    }
+    ss = warp_sum(ss);
+    const float inv = 1.0f / (ss + unit_eps);
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+        const int i = lane + 32 * u;
+        if (i >= D) break;
+        const size_t e = (size_t)h * D + i;
+        dc[i] = expf(-scale * sigmoid_f(dc[i] + load_as_f32(w0, vec_dtype, e)));
+        rm[i] = sigmoid_f(to_f32(a[i]) + load_as_f32(a_bias, vec_dtype, e)) * kv[u] * inv;
+    }
+}
+
+RB_EXPORT int rb_general_delta_prep(const void* proj, int ld, int k_off, int a_off, const void* a_bias, const void* w0,
+                                    int vec_dtype, float scale, float unit_eps, float* decay, float* removal, int act_dtype,
+                                    int T, int H, int D, cudaStream_t st) {
+    if (T <= 0) return 0;
+    if (D < 1 || D > 256) return (int)cudaErrorInvalidValue;
+    const int rows = T * H;
+    if (act_dtype == RB_F32)
+        return rb_launch_pdl(general_delta_prep_kernel<float>, dim3((rows + 3) / 4), dim3(128), 0, st, (const float*)proj, ld, k_off,
+                             a_off, a_bias, w0, vec_dtype, scale, unit_eps, decay, removal, rows, H, D);
+    return rb_launch_pdl(general_delta_prep_kernel<bf16>, dim3((rows + 3) / 4), dim3(128), 0, st, (const bf16*)proj, ld, k_off,
+                         a_off, a_bias, w0, vec_dtype, scale, unit_eps, decay, removal, rows, H, D);
 }
 
 // The conv state after a step: the last K - 1 inputs of each channel, oldest first.  A segment shorter than K - 1

@@ -46,7 +46,7 @@ class ModelRunner:
         self.max_positions = max_positions
         self.storage = CacheStorage(model.cache_needs(), engine_config.page_size, engine_config.num_pages,
                                     engine_config.max_reside, self.env,
-                                    longest_append=min(engine_config.prefill_chunk, max_positions))
+                                    longest_append=min(engine_config.prefill_chunk, max_positions), kept=model.kept_needs())
         self.manager: CacheManager = self.storage.make_manager()
         self.storage.allocate()
         self.staging = BatchStaging(self.env.device)

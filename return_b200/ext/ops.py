@@ -100,7 +100,7 @@ def core() -> ctypes.CDLL:
         lib.rb_gemm_skinny_ctas.restype = c_int
         lib.rb_qk_norm_rope_write.argtypes = [P, I, P, P, I, F, F, P, P, I, P, P, P, I, I, P, P, I, I, I, I, I, I, P]
         lib.rb_attention_simt.argtypes = [P, I, P, P, P, P, P, I, I, P, I, I, I, I, I, F, I, P]
-        lib.rb_attention_simt_mod.argtypes = [P, I, P, P, P, P, P, I, I, P, I, I, I, I, I, F, I, I, F, P, P, P]
+        lib.rb_attention_simt_mod.argtypes = [P, I, P, P, P, P, P, I, I, P, I, I, I, I, I, F, I, I, F, P, P, P, I, P]
         lib.rb_attn_prep.argtypes = [P, I, I, I, I, P, P, P, I, P, P, I, F, P, P, I, P, P, P, I, I, P, P, P, I, I, I, I, I, I, I, I, P]
         lib.rb_attn_gate.argtypes = [P, P, I, I, I, I, I, I, I, I, P]
         lib.rb_embedding_pair.argtypes = [P, P, I, P, P, P, P, P, P, P, I, I, I, F, I, L, L, P]
@@ -127,6 +127,8 @@ def build_all():
     paths = [build.library_path("return_core", _CORE_SOURCES, {"RB_PDL_MODE": PDL_MODE})]
     paths.append(build.library_path("return_tc5", _TC5_SOURCES, _tc5_defines()))
     paths.append(build.library_path("return_recurrent", _RECURRENT_SOURCES, {"RB_PDL_MODE": PDL_MODE}))
+    paths.append(build.library_path("return_attn_conv", _ATTN_CONV_SOURCES, {"RB_PDL_MODE": PDL_MODE}))
+    paths.append(build.library_path("return_tanh_norm", _TANH_NORM_SOURCES, {"RB_PDL_MODE": PDL_MODE}))
     paths.append(build.library_path("return_latent", _LATENT_SOURCES, {"RB_PDL_MODE": PDL_MODE}))
     paths.append(build.library_path("return_moe", _MOE_SOURCES, {"RB_PDL_MODE": PDL_MODE}))
     paths.append(build.library_path("return_moe_tc5", _MOE_TC5_SOURCES, {"RB_PDL_MODE": PDL_MODE}))
@@ -632,8 +634,8 @@ def attention_lib(head_dim: int) -> ctypes.CDLL:
         lib.rb_attn_decode.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, P, I, I, F, I, I, P, P]
         lib.rb_attn_decode_fused.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, P, I, I, F, I, I, P, P, I, F, F, P, P, I, I, P]
         lib.rb_attn_decode_fused.restype = c_int
-        lib.rb_attn_prefill_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, I, I, F, I, P, I, F, P, P]
-        lib.rb_attn_decode_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, P, I, I, F, I, I, P, I, F, P, P]
+        lib.rb_attn_prefill_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, I, I, F, I, P, I, F, P, P, I, P]
+        lib.rb_attn_decode_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, P, I, I, F, I, I, P, I, F, P, P, I, P]
         lib.rb_attn_prefill_mod.restype = lib.rb_attn_decode_mod.restype = c_int
         lib.rb_attn_decode_scratch_floats.argtypes = [I, I, I]
         lib.rb_attn_decode_scratch_floats.restype = ctypes.c_longlong
@@ -676,7 +678,7 @@ def attention_tc5_lib(head_dim: int) -> ctypes.CDLL:
         lib = build.load(f"return_attn_tc5_d{head_dim}", ["attention_tc5.cu"], _attn_tc5_defines(head_dim))
         P, I, F = c_void_p, c_int, c_float
         lib.rb_attn_prefill_tc5.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, I, I, F, I, I, P, I, P, P, P]
-        lib.rb_attn_prefill_tc5_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, I, I, F, I, I, P, I, P, P, I, F, P, P]
+        lib.rb_attn_prefill_tc5_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, I, I, F, I, I, P, I, P, P, I, F, P, P, I, P]
         lib.rb_attn_prefill_tc5_mod.restype = c_int
         lib.rb_attn_tc5_split_floats.argtypes = [I, I, I]
         lib.rb_attn_tc5_split_floats.restype = ctypes.c_longlong
@@ -692,14 +694,22 @@ def _sink_ptr(sink, num_heads):
     return _ptr(sink)
 
 
+def _bias_args(bias, num_heads):
+    """The pointer and row length of a bias table by head and distance, or (None, 0)."""
+    if bias is None:
+        return None, 0
+    assert bias.dtype == torch.float32 and bias.dim() == 2 and bias.shape[0] == num_heads and bias.shape[1] >= 1 and bias.is_contiguous()
+    return _ptr(bias), bias.shape[1]
+
+
 def attention_prefill_tc5(qkv, k_pool, v_pool, tiles, cu_q, seg_pos0, block_table, page_size, out, num_heads,
                           num_kv_heads, head_dim, scale, window=0, num_splits=1, held=None, sink=None,
-                          chunk=0, softcap=0.0, slopes=None) -> None:
+                          chunk=0, softcap=0.0, slopes=None, bias=None) -> None:
     """tcgen05 attention for the listed (segment, first row) blocks of up to TC5_TILE_ROWS query rows
     (the blocks with the longest contexts should come first: they take longest).  ``num_splits`` > 1 splits
     every block's keys over that many CTAs and merges them in a second launch; ``held``: the step's map of
-    work buffers, so that the layers share the buffer of the partial results.  ``chunk``, ``softcap``, ``slopes``: the
-    score options of ``paged_attention``."""
+    work buffers, so that the layers share the buffer of the partial results.  ``chunk``, ``softcap``, ``slopes``, ``bias``:
+    the score options of ``paged_attention``."""
     assert qkv.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.is_contiguous()
     assert tiles.dtype == torch.int32 and tiles.is_contiguous()
     lib = attention_tc5_lib(head_dim)
@@ -718,7 +728,7 @@ def attention_prefill_tc5(qkv, k_pool, v_pool, tiles, cu_q, seg_pos0, block_tabl
                                        block_table.stride(0), page_size, _ptr(out), num_heads, num_kv_heads, scale,
                                        int(window or 0), num_splits, _ptr(scratch), T, _ptr(tc5_status(qkv.device)),
                                        _sink_ptr(sink, num_heads), int(chunk or 0), float(softcap or 0.0),
-                                       _sink_ptr(slopes, num_heads), _stream()), "attention_prefill_tc5", 2 if num_splits > 1 else 1)
+                                       _sink_ptr(slopes, num_heads), *_bias_args(bias, num_heads), _stream()), "attention_prefill_tc5", 2 if num_splits > 1 else 1)
 
 
 PREFILL_SPLIT_MIN_KEYS = 512       # a CTA of a split block keeps at least this many keys
@@ -765,17 +775,18 @@ def decode_splits(n_ctas_base: int, max_kv_len: int, ctas_per_sm: int = 2) -> in
 
 
 def attention_prefill_mma(qkv, k_pool, v_pool, tiles, cu_q, seg_pos0, block_table, page_size, out, num_heads,
-                          num_kv_heads, head_dim, scale, window=0, sink=None, chunk=0, softcap=0.0, slopes=None) -> None:
+                          num_kv_heads, head_dim, scale, window=0, sink=None, chunk=0, softcap=0.0, slopes=None,
+                          bias=None) -> None:
     """Tensor-core attention for the listed (segment, first row) tiles of up to 64 query rows.  ``chunk``, ``softcap``,
-    ``slopes``: the score options of ``paged_attention``."""
+    ``slopes``, ``bias``: the score options of ``paged_attention``."""
     assert qkv.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.is_contiguous()
     assert tiles.dtype == torch.int32 and tiles.is_contiguous()
     lib = attention_lib(head_dim)
     _check(lib.rb_attn_prefill_mod(_ptr(qkv), qkv.stride(0), _ptr(k_pool), _ptr(v_pool), _ptr(tiles), tiles.shape[0],
                                    _ptr(cu_q), _ptr(seg_pos0), _ptr(block_table), block_table.stride(0), page_size,
                                    _ptr(out), num_heads, num_kv_heads, scale, int(window or 0), _sink_ptr(sink, num_heads),
-                                   int(chunk or 0), float(softcap or 0.0), _sink_ptr(slopes, num_heads), _stream()),
-           "attention_prefill")
+                                   int(chunk or 0), float(softcap or 0.0), _sink_ptr(slopes, num_heads), *_bias_args(bias, num_heads),
+                                   _stream()), "attention_prefill")
 
 
 def _split_scratch(lib, n, num_heads, num_splits, device, held=None):
@@ -793,9 +804,9 @@ def _split_scratch(lib, n, num_heads, num_splits, device, held=None):
 
 def attention_decode_mma(qkv, k_pool, v_pool, decode_segs, cu_q, seg_kv_len, block_table, page_size, out,
                          num_heads, num_kv_heads, head_dim, scale, window=0, num_splits=1, held=None, sink=None,
-                         chunk=0, softcap=0.0, slopes=None) -> None:
+                         chunk=0, softcap=0.0, slopes=None, bias=None) -> None:
     """Tensor-core attention for segments of one token, the keys split ``num_splits`` ways.  ``chunk``, ``softcap``,
-    ``slopes``: the score options of ``paged_attention``."""
+    ``slopes``, ``bias``: the score options of ``paged_attention``."""
     assert qkv.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.is_contiguous()
     lib = attention_lib(head_dim)
     n = decode_segs.shape[0]
@@ -804,7 +815,7 @@ def attention_decode_mma(qkv, k_pool, v_pool, decode_segs, cu_q, seg_kv_len, blo
                                   _ptr(cu_q), _ptr(seg_kv_len), _ptr(block_table), block_table.stride(0), page_size,
                                   _ptr(scratch), _ptr(out), num_heads, num_kv_heads, scale, int(window or 0),
                                   num_splits, _sink_ptr(sink, num_heads), int(chunk or 0), float(softcap or 0.0),
-                                  _sink_ptr(slopes, num_heads), _stream()), "attention_decode", 2 if num_splits > 1 else 1)
+                                  _sink_ptr(slopes, num_heads), *_bias_args(bias, num_heads), _stream()), "attention_decode", 2 if num_splits > 1 else 1)
 
 
 def _decode_split_count(batch, num_heads, num_kv_heads, window) -> int:
@@ -883,7 +894,7 @@ def attention_decode_fused(qkv, q_weight, k_weight, eps, offset, cos, sin, rot_d
 
 
 def paged_attention(qkv, k_pool, v_pool, batch, block_table, page_size, out, num_heads, num_kv_heads,
-                    head_dim, scale, window=None, sink=None, chunk=None, softcap=None, slopes=None) -> None:
+                    head_dim, scale, window=None, sink=None, chunk=None, softcap=None, slopes=None, bias=None) -> None:
     """Attention of every token of the step over its request's cached keys (its own included).
 
     float32: the CUDA-core kernel, whose result does not depend on how the work was cut.
@@ -893,7 +904,7 @@ def paged_attention(qkv, k_pool, v_pool, batch, block_table, page_size, out, num
     Options of the score: ``window`` (the last n keys) or ``chunk`` (the keys of the query's own block of n positions,
     blocks counted from position 0), never both; ``sink`` (float32 [heads]: exp(sink) joins the softmax's denominator);
     ``softcap`` (a scaled score s becomes cap * tanh(s / cap)); ``slopes`` (float32 [heads]: slopes[h] * (i - j) is taken
-    off the score of key j for query i)."""
+    off the score of key j for query i); ``bias`` (float32 [heads, n]: bias[h, min(i - j, n - 1)] is added to it)."""
     if window and chunk:
         raise KernelError("a window and a chunk exclude each other")
     if qkv.dtype == torch.float32:
@@ -903,7 +914,7 @@ def paged_attention(qkv, k_pool, v_pool, batch, block_table, page_size, out, num
             _ptr(qkv), qkv.stride(0), _ptr(k_pool), _ptr(v_pool), _ptr(batch.pos), _ptr(batch.tok_seg), _ptr(block_table),
             block_table.stride(0), page_size, _ptr(out), dtype_code(qkv.dtype), T, num_heads, num_kv_heads, head_dim, scale,
             int(window or 0), int(chunk or 0), float(softcap or 0.0), _sink_ptr(slopes, num_heads),
-            _sink_ptr(sink, num_heads), _stream()), "attention_simt")
+            _sink_ptr(sink, num_heads), *_bias_args(bias, num_heads), _stream()), "attention_simt")
         return
     host = batch.host
     bound = window or chunk                       # either bounds the keys a query can see
@@ -912,17 +923,17 @@ def paged_attention(qkv, k_pool, v_pool, batch, block_table, page_size, out, num
             attention_prefill_tc5(qkv, k_pool, v_pool, batch.tiles[TILES_TC5], batch.cu_q, batch.seg_pos0, block_table,
                                   page_size, out, num_heads, num_kv_heads, head_dim, scale, window or 0,
                                   _prefill_split_count(batch, num_heads, bound), getattr(batch, "scratch", None), sink,
-                                  chunk, softcap, slopes)
+                                  chunk, softcap, slopes, bias)
         else:
             attention_prefill_mma(qkv, k_pool, v_pool, batch.tiles[TILES_MMA], batch.cu_q, batch.seg_pos0, block_table,
                                   page_size, out, num_heads, num_kv_heads, head_dim, scale, window or 0, sink,
-                                  chunk, softcap, slopes)
+                                  chunk, softcap, slopes, bias)
     n_dec = host.decode_segs.shape[0]
     if n_dec:
         attention_decode_mma(qkv, k_pool, v_pool, batch.decode_segs, batch.cu_q, batch.seg_kv_len, block_table,
                              page_size, out, num_heads, num_kv_heads, head_dim, scale, window or 0,
                              _decode_split_count(batch, num_heads, num_kv_heads, bound), getattr(batch, "scratch", None), sink,
-                             chunk, softcap, slopes)
+                             chunk, softcap, slopes, bias)
 
 
 def attention_prepare(proj, q_off: int, k_off: int, v_off: int, biases, norms, eps: float, tables, batch, kv, q_out,
@@ -958,11 +969,107 @@ def attention_gate(o, gate, g_off: int, per_head: bool, num_heads: int, vdim: in
                                num_heads, vdim, head_dim, _stream()), "attention_gate")
 
 
+# ------------------------------------------------------------------------------- attention behind a convolution
+
+_attn_conv = None
+_ATTN_CONV_SOURCES = ["attention_conv.cu"]
+
+
+def attention_conv_lib() -> ctypes.CDLL:
+    """The kernel between the projections and the attention of heads that pass a short convolution (csrc/attention_conv.cu);
+    compiled when a model that has such an attention is first run."""
+    global _attn_conv
+    if _attn_conv is None:
+        lib = build.load("return_attn_conv", _ATTN_CONV_SOURCES, {"RB_PDL_MODE": PDL_MODE})
+        P, I, F, L = c_void_p, c_int, c_float, ctypes.c_longlong
+        lib.rb_attn_conv_prep.argtypes = [P, I, P, I, I, P, L, I, P, P, P, P, P, I, I, P, P, P, I, I, I, I, I, I, I, I, I, I, F, F, I, P]
+        lib.rb_attn_conv_prep.restype = c_int
+        _attn_conv = lib
+    return _attn_conv
+
+
+def attention_conv_prepare(proj, taps, kept, kept_off: int, batch, kv, q_out, num_heads: int, num_kv_heads: int, dim: int,
+                           vdim: int, head_dim: int, norm_eps: Optional[float] = None, temperature=None, own_kv: bool = True,
+                           write_kv: bool = True) -> None:
+    """From projection rows [q | k | v] (only q without ``own_kv``) to what the paged attention reads: every channel through
+    its causal filter ``taps`` [channels, K] (last column: the token itself), q and k heads over their root mean square
+    (``norm_eps``; None: not normed), q heads times 1 + coef ln(floor((p + 1) / every) + 1) (``temperature`` = (coef, every)),
+    q heads padded to ``head_dim`` into q_out, k and v heads into their pages.  ``kept`` (float32 [slots, n]): a request's
+    last K - 1 rows of inputs from column kept_off, read and renewed."""
+    T = proj.shape[0]
+    K = taps.shape[1]
+    channels = num_heads * dim + (num_kv_heads * (dim + vdim) if own_kv else 0)
+    assert proj.stride(1) == 1 and proj.shape[1] >= channels and taps.shape[0] == channels and taps.is_contiguous()
+    assert q_out.is_contiguous() and q_out.dtype == proj.dtype and q_out.shape == (T, num_heads * head_dim)
+    assert kv.k.dtype == kv.v.dtype == proj.dtype and kv.k.shape[-1] == head_dim
+    if K > 1:
+        assert kept.dtype == torch.float32 and kept.is_contiguous() and kept.shape[1] >= kept_off + (K - 1) * channels
+    coef, every = temperature if temperature is not None else (0.0, 0)
+    _check(attention_conv_lib().rb_attn_conv_prep(
+        _ptr(proj), proj.stride(0), _ptr(taps), dtype_code(taps.dtype), K, _ptr(kept) if K > 1 else None,
+        kept.stride(0) if K > 1 else 0, kept_off, _ptr(batch.pos), _ptr(batch.tok_seg), _ptr(batch.cu_q), _ptr(batch.seg_slot),
+        _ptr(kv.block_table), kv.block_table.stride(0), kv.page_size, _ptr(kv.k), _ptr(kv.v), _ptr(q_out),
+        dtype_code(proj.dtype), T, num_heads, num_kv_heads, dim, vdim, head_dim, 1 if own_kv else 0, 1 if write_kv else 0,
+        0 if norm_eps is None else 1, float(norm_eps or 0.0), float(coef), int(every), _stream()), "attention_conv_prepare")
+
+
+# ------------------------------------------------------------------------------- squashes in the place of norms
+
+_tanh_norm = None
+_TANH_NORM_SOURCES = ["tanh_norm.cu"]
+
+
+def tanh_norm_lib() -> ctypes.CDLL:
+    """The joint of layers whose norms are elementwise squashes (csrc/tanh_norm.cu); compiled when a model that has them is
+    first run."""
+    global _tanh_norm
+    if _tanh_norm is None:
+        lib = build.load("return_tanh_norm", _TANH_NORM_SOURCES, {"RB_PDL_MODE": PDL_MODE})
+        P, I, L = c_void_p, c_int, ctypes.c_longlong
+        lib.rb_tanh_joint.argtypes = [P, P, P, I, P, P, P, P, P, P, P, P, L, I, P, P, P, P, P, I, I, I, P]
+        lib.rb_tanh_joint.restype = c_int
+        _tanh_norm = lib
+    return _tanh_norm
+
+
+def tanh_joint(x_in, x_out, y, post, nxt, out, shift=None, batch=None, rows=None) -> None:
+    """x = x_in + post(y), left in ``x_out`` (None: not stored); out = next(x), with ``shift`` blended with the row before:
+    h + (h_before - h) * mu.  x_in, x_out float32 [T, H]; y [T, H] float32 or bfloat16, or None: nothing is added; ``post``
+    and ``nxt``: (alpha [1], w [H], b [H]) in float32 of tanh(alpha x) * w + b, or None (y as it is; no ``out``).  ``shift`` =
+    (mu float32 [H], kept float32 [slots, n], column of the request's last h in its row), with ``batch`` (the step's
+    tables); x_out is then another buffer than x_in if something is added.  ``rows`` (int32): only these rows of x_in."""
+    T, H = x_in.shape
+    n = T if rows is None else rows.numel()
+    assert x_in.dtype == torch.float32 and x_in.is_contiguous()
+    assert x_out is None or (x_out.dtype == torch.float32 and x_out.is_contiguous() and x_out.shape == x_in.shape and rows is None)
+    assert y is None or (y.shape == x_in.shape and y.is_contiguous())
+    for triple in (post, nxt):
+        assert triple is None or all(v.dtype == torch.float32 and v.is_contiguous() for v in triple)
+        assert triple is None or (triple[0].numel() == 1 and triple[1].numel() == triple[2].numel() == H)
+    if nxt is not None:
+        assert out.is_contiguous() and out.shape == (n, H)
+    elif x_out is None or y is None:
+        return
+    mu = kept = None
+    off = stride = 0
+    if shift is not None:
+        mu, kept, off = shift
+        stride = kept.stride(0)
+        assert mu.dtype == kept.dtype == torch.float32 and mu.numel() == H and kept.is_contiguous() and off + H <= kept.shape[1]
+    none3 = (None, None, None)
+    _check(tanh_norm_lib().rb_tanh_joint(
+        _ptr(x_in), _ptr(x_out) if y is not None else None, _ptr(y), _is_f32(y) if y is not None else 1,
+        *(_ptr(v) for v in (post or none3)), *(_ptr(v) for v in (nxt or none3)), _ptr(mu), _ptr(kept), stride, off,
+        _ptr(batch.tok_seg) if mu is not None else None, _ptr(batch.cu_q) if mu is not None else None,
+        _ptr(batch.seg_slot) if mu is not None else None, _ptr(rows), _ptr(out) if nxt is not None else None,
+        dtype_code(out.dtype) if nxt is not None else F32, n, H, _stream()), "tanh_joint")
+
+
 # ------------------------------------------------------------------------------- mixers with a matrix state
 
 _recurrent = None
 _RECURRENT_SOURCES = ["recurrent.cu"]
-SCAN_DECAY, SCAN_MEMORY, SCAN_DELTA, SCAN_BONUS, SCAN_SSM, SCAN_DELTA_HEAD = 0, 1, 2, 3, 4, 5
+SCAN_DECAY, SCAN_MEMORY, SCAN_DELTA, SCAN_BONUS, SCAN_SSM, SCAN_DELTA_HEAD, SCAN_GENERAL_DELTA = 0, 1, 2, 3, 4, 5, 6
 SCAN_MAX_KEY_DIM = 256
 
 
@@ -991,6 +1098,8 @@ def recurrent_lib() -> ctypes.CDLL:
         lib.rb_gated_recurrence.argtypes = [P, P, I, P, P, P, I, F, P, I, P, P, L, I, P, P, P, I, I, I, I, P, P]
         lib.rb_gated_pieces_combine.argtypes = [P, P, P, L, I, P, P, I, I, P]
         lib.rb_gated_conv.restype = lib.rb_gated_recurrence.restype = lib.rb_gated_pieces_combine.restype = c_int
+        lib.rb_general_delta_prep.argtypes = [P, I, I, I, P, P, I, F, F, P, P, I, I, I, I, P]
+        lib.rb_general_delta_prep.restype = c_int
         lib.rb_conv_state_update.argtypes = [P, I, I, P, L, I, P, P, I, I, I, P]
         lib.rb_head_norm_gate.argtypes = [P, P, I, P, I, I, I, F, P, I, I, I, I, P]
         lib.rb_add_dual_norm.argtypes = [P, P, I, F, P, I, F, P, P, P, I, F, F, P, P, I, I, I, P]
@@ -1020,7 +1129,8 @@ def linear_scan(mode: int, q, k, v, gate_a, gate_b, state, offsets, batch, out, 
     matrix, the normaliser and the running maximum start inside a row (the last two for ``SCAN_MEMORY`` only).
     ``gate_a`` / ``gate_b`` by mode: SCAN_DECAY: [heads] decays / None; SCAN_MEMORY: [T, 2 heads] gate
     pre-activations (input, forget) / [2 heads] biases; SCAN_DELTA: [T, heads, dim] row decays / [T, heads] beta;
-    SCAN_DELTA_HEAD: [T, heads] decays / [T, heads] beta;
+    SCAN_DELTA_HEAD: [T, heads] decays / [T, heads] beta; SCAN_GENERAL_DELTA (S <- g * S - c (k^T S) + k v^T, o = S^T q):
+    [T, heads, dim] row decays / [T, heads, dim] removal vectors c;
     SCAN_BONUS (o = (S + diag(u) k v^T)^T q, then S <- g * S + k v^T): [T, heads, dim] row decays / None, ``extra`` = u
     [heads, dim]; SCAN_SSM (S <- a S + dt k v^T, o = S^T q + d v): [T, heads] decays / [T, heads] steps, ``extra`` = d
     [heads].
@@ -1123,6 +1233,21 @@ def delta_prep(x, taps, state, conv_off: int, batch, q32, k32, v32, a, A_log, dt
         _ptr(batch.tok_seg), _ptr(batch.cu_q), _ptr(batch.seg_slot), _ptr(q32), _ptr(k32), _ptr(v32), _ptr(a),
         _ptr(A_log), _ptr(dt_bias), dtype_code(A_log.dtype), _ptr(b), dtype_code(x.dtype), T, heads, kv_heads, dim, vdim,
         q_scale, 1 if head_decay else 0, _stream()), "delta_prep")
+
+
+def general_delta_prep(proj, k_off: int, a_off: int, a_bias, w0, scale: float, unit_eps: float, decay, removal, heads: int,
+                       dim: int) -> None:
+    """What the general delta rule's scan needs per token, head and key row: decay = exp(-scale * sigmoid(decay + w0)) in place
+    (float32 [T, heads * dim]) and removal = sigmoid(a + a_bias) * k / (sum of the head's k^2 + unit_eps), with k and a the
+    columns of ``proj`` from k_off and a_off."""
+    T = proj.shape[0]
+    n = heads * dim
+    assert proj.stride(1) == 1 and a_bias.dtype == w0.dtype and a_bias.numel() == w0.numel() == n
+    for t in (decay, removal):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n)
+    _check(recurrent_lib().rb_general_delta_prep(_ptr(proj), proj.stride(0), k_off, a_off, _ptr(a_bias), _ptr(w0),
+                                                 dtype_code(w0.dtype), scale, unit_eps, _ptr(decay), _ptr(removal),
+                                                 dtype_code(proj.dtype), T, heads, dim, _stream()), "general_delta_prep")
 
 
 def gated_conv(x, x_bias, taps, conv_bias, state, conv_off: int, batch, out) -> None:
@@ -1446,9 +1571,9 @@ def moe_lib() -> ctypes.CDLL:
     if _moe is None:
         lib = build.load("return_moe", _MOE_SOURCES, {"RB_PDL_MODE": PDL_MODE})
         P, I, F = c_void_p, c_int, c_float
-        lib.rb_moe_route.argtypes = [P, I, P, P, P, I, I, I, I, I, F, I, I, F, P]
+        lib.rb_moe_route.argtypes = [P, I, P, P, P, I, I, I, I, I, F, I, I, F, I, P]
         lib.rb_moe_pair_linear.argtypes = [P, I, I, P, P, P, I, I, I, I, I, P]
-        lib.rb_clamped_glu.argtypes = [P, I, P, I, I, I, I, F, F, F, P]
+        lib.rb_clamped_glu.argtypes = [P, I, P, I, I, I, I, F, F, F, P, P, P]
         lib.rb_moe_combine.argtypes = [P, P, P, P, P, I, I, I, I, P]
         lib.rb_moe_sort.argtypes = [P, I, I, P, P, P, P]
         lib.rb_moe_grouped_gemm.argtypes = [P, I, P, I, P, P, I, P, I, I, I, I, P]
@@ -1461,13 +1586,13 @@ def moe_lib() -> ctypes.CDLL:
 
 
 def moe_route(logits, expert_of, weight, top: int, groups: int = 1, keep: int = 1, tiny: float = 1e-20, bias=None,
-              score: str = "softmax", group_top: int = 1, scale: float = 1.0) -> None:
+              score: str = "softmax", group_top: int = 1, scale: float = 1.0, renorm: bool = True) -> None:
     """The router's choice per token from float32 logits [T, E] (plus ``bias``, float32 [E], if given): softmax over all
     experts; with ``groups`` > 1 only the
     experts of the ``keep`` groups (equal runs of neighbours) with the largest best score can be chosen; the ``top``
     largest scores among them, in falling order, into expert_of (int32 [T, top]) with weight = score / (sum + tiny).
     ``score`` "sigmoid": every expert's score is the logistic of its own logit.  ``group_top`` 2: a group scores as the sum
-    of its two best.  ``scale``: a factor on the weights."""
+    of its two best.  ``scale``: a factor on the weights.  ``renorm`` False: weight = score, not divided by the sum."""
     T, E = logits.shape
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
     assert expert_of.dtype == torch.int32 and expert_of.shape == (T, top) and expert_of.is_contiguous()
@@ -1475,7 +1600,7 @@ def moe_route(logits, expert_of, weight, top: int, groups: int = 1, keep: int = 
     if bias is not None:
         assert bias.dtype == torch.float32 and bias.numel() == E and bias.is_contiguous()
     _check(moe_lib().rb_moe_route(_ptr(logits), logits.stride(0), _ptr(bias), _ptr(expert_of), _ptr(weight), T, E, top, groups,
-                                  keep, tiny, {"softmax": 0, "sigmoid": 1}[score], group_top, scale, _stream()), "moe_route")
+                                  keep, tiny, {"softmax": 0, "sigmoid": 1}[score], group_top, scale, 1 if renorm else 0, _stream()), "moe_route")
 
 
 def moe_pair_linear(x, in_div: int, w, expert_of, out) -> None:
@@ -1488,19 +1613,26 @@ def moe_pair_linear(x, in_div: int, w, expert_of, out) -> None:
                                         dtype_code(x.dtype), pairs, N, K, _stream()), "moe_pair_linear")
 
 
-def clamped_glu(gate_up, out, limit: float, alpha: float, shift: float = 1.0) -> None:
+def clamped_glu(gate_up, out, limit: float, alpha: float, shift: float = 1.0, weight=None, pair_at=None) -> None:
     """gate_up [rows, 2F] = [gate | up]: out = g * sigmoid(alpha g) * (u + shift) with g = min(gate, limit) and
-    u = clamp(up, -limit, limit).  An infinite limit, alpha = 1 and shift = 0 give silu(gate) * up."""
+    u = clamp(up, -limit, limit).  An infinite limit, alpha = 1 and shift = 0 give silu(gate) * up.  ``weight`` (float32):
+    row r's gate and up are multiplied by weight[pair_at[r]] (weight[r] without ``pair_at``) first."""
     rows, F2 = gate_up.shape
+    assert weight is None or (weight.dtype == torch.float32 and weight.numel() == rows and weight.is_contiguous())
+    assert pair_at is None or (pair_at.dtype == torch.int32 and pair_at.numel() == rows)
     assert out.shape == (rows, F2 // 2) and out.dtype == gate_up.dtype and gate_up.stride(1) == 1 and out.stride(1) == 1
     _check(moe_lib().rb_clamped_glu(_ptr(gate_up), gate_up.stride(0), _ptr(out), out.stride(0), dtype_code(out.dtype), rows,
-                                    F2 // 2, float(limit), float(alpha), float(shift), _stream()), "clamped_glu")
+                                    F2 // 2, float(limit), float(alpha), float(shift), _ptr(weight), _ptr(pair_at), _stream()),
+           "clamped_glu")
 
 
-def moe_combine(y, weight, shared, out, row_of=None) -> None:
-    """out[t] = sum_k weight[t, k] * y[row of pair t * top + k] (+ shared[t]); sums in float32 in the order of k."""
-    T, top = weight.shape
-    H = out.shape[1]
+def moe_combine(y, weight, shared, out, row_of=None, top=None) -> None:
+    """out[t] = sum_k weight[t, k] * y[row of pair t * top + k] (+ shared[t]); sums in float32 in the order of k.  ``weight``
+    None (with ``top``): a plain sum."""
+    T, H = out.shape
+    if weight is not None:
+        assert weight.shape[0] == T and weight.dtype == torch.float32 and weight.is_contiguous()
+        top = weight.shape[1]
     assert y.shape == (T * top, H) and y.is_contiguous() and out.is_contiguous() and out.dtype == y.dtype
     if shared is not None:
         assert shared.shape == out.shape and shared.is_contiguous() and shared.dtype == y.dtype
@@ -1574,8 +1706,9 @@ MOE_TC5_MIN_PAIRS = 1024
 
 
 def moe_experts(x, gate_up, down, expert_of, weight, shared, out, limit: float, alpha: float, ctx=None,
-                shift: float = 1.0) -> None:
-    """out[t] = sum_k weight[t, k] * expert_{expert_of[t, k]}(x[t]) (+ shared[t]); gate_up [E, 2F, H], down [E, H, F];
+                shift: float = 1.0, weigh_input: bool = False) -> None:
+    """out[t] = sum_k weight[t, k] * expert_{expert_of[t, k]}(x[t]) (+ shared[t]), or with ``weigh_input`` the sum of
+    expert(weight[t, k] * x[t]); gate_up [E, 2F, H], down [E, H, F];
     an expert is down(g sigmoid(alpha g) (u + shift)) with the gate capped at ``limit`` and the up part clamped to it."""
     E, F2, H = gate_up.shape
     T, top = expert_of.shape
@@ -1586,6 +1719,7 @@ def moe_experts(x, gate_up, down, expert_of, weight, shared, out, limit: float, 
             return ctx.buffer(name, shape, dtype or x.dtype, x.device)
         return torch.empty(shape, dtype=dtype or x.dtype, device=x.device)
 
+    w_in, w_out = (weight, None) if weigh_input else (None, weight)
     gu = buf("moe.pair_gate_up", (pairs, F2))
     act = buf("moe.pair_act", (pairs, F2 // 2))
     y = buf("moe.pair_y", (pairs, H))
@@ -1599,18 +1733,18 @@ def moe_experts(x, gate_up, down, expert_of, weight, shared, out, limit: float, 
             rows = buf("moe.pair_rows", (pairs, H))
             moe_gather_rows(x, pair_at, top, rows)
             moe_tc5_gemm(rows, gate_up, offsets, gu)
-            clamped_glu(gu, act, limit, alpha, shift)
+            clamped_glu(gu, act, limit, alpha, shift, w_in, pair_at)
             moe_tc5_gemm(act, down, offsets, y)
         else:
             moe_grouped_gemm(x, pair_at, top, gate_up, offsets, gu)
-            clamped_glu(gu, act, limit, alpha, shift)
+            clamped_glu(gu, act, limit, alpha, shift, w_in, pair_at)
             moe_grouped_gemm(act, None, 1, down, offsets, y)
-        moe_combine(y, weight, shared, out, row_of=place_of)
+        moe_combine(y, w_out, shared, out, row_of=place_of, top=top)
         return
     moe_pair_linear(x, top, gate_up, expert_of, gu)
-    clamped_glu(gu, act, limit, alpha, shift)
+    clamped_glu(gu, act, limit, alpha, shift, w_in)
     moe_pair_linear(act, 1, down, expert_of, y)
-    moe_combine(y, weight, shared, out)
+    moe_combine(y, w_out, shared, out, top=top)
 
 
 # ------------------------------------------------------------------------------- sampling

@@ -105,6 +105,10 @@ class DecoderModel:
             out.append(StateNeed((1,), torch.int32))
         return out
 
+    def kept_needs(self) -> List[Optional[StateNeed]]:
+        """Per schedule entry: what the run keeps per request for itself, whichever cache it owns or reads."""
+        return [self.blocks[e.layer].kept_need() for e in self.spec.schedule]
+
     @staticmethod
     def _fold(stream, deltas):
         """A block may leave several outputs still to be added to the stream (one per branch); whoever cannot take
@@ -136,6 +140,7 @@ class DecoderModel:
             owner = index if entry.cache_of is None else entry.cache_of
             ctx = storage.layer_context(owner, batch, write=entry.cache_of is None)
             ctx.position = index
+            ctx.kept, ctx.next_kept = storage.kept(index), storage.kept(index + 1)
             ctx.next_block = self.blocks[schedule[index + 1].layer] if index + 1 < len(schedule) else None
             block = self.blocks[entry.layer]
             if isinstance(delta, tuple) and not getattr(block, "takes_delta_pair", False):

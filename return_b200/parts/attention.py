@@ -8,6 +8,8 @@ attention over the block table, output projection
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..ext import ops
@@ -127,13 +129,29 @@ class PagedAttention(Mixer):
         return o
 
 
+def distance_rows(rows: int, reach: float):
+    """The row of a distance table of ``rows`` rows for every distance 0, 1, 2, ... up to the first that has the last row
+    (all farther ones have it too): row n below half = rows // 2, then rows for ever longer spans,
+    half + floor(ln(n / half) / ln(reach / half) * (rows - half)).  Worked out in float64."""
+    half = rows // 2
+    out, n = [], 0
+    while not out or out[-1] != rows - 1:
+        out.append(n if n < half else
+                   min(rows - 1, half + math.floor(math.log(n / half) / math.log(reach / half) * (rows - half))))
+        n += 1
+    return out
+
+
 @MIXERS.register("gated_attention")
 class GatedAttention(Mixer):
     """``GatedAttentionSpec``: one product gives a row [q | k | v | gate] (k and v only if the layer owns its cache; v
     only if it has a value projection); one kernel prepares the row (biases, the norm over a whole projection, the
     rotation of neighbouring pairs, heads padded to the cache's head size, keys and values into their pages); the
     engine's paged attention kernels run with the layer's score options; the gate is applied and the heads are
-    projected out.  A layer that reads another run's cache prepares its queries only."""
+    projected out.  A layer that reads another run's cache prepares its queries only.  Heads that are prepared one by
+    one (a convolution over time, a norm per head, a query temperature) have a row kernel of their own
+    (csrc/attention_conv.cu); the run keeps the last rows of its projections per request (``kept_floats``), also when the
+    keys and values it attends to are another run's."""
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
@@ -156,12 +174,26 @@ class GatedAttention(Mixer):
             raise ValueError("the row kernel rotates neighbouring pairs: the position encoding must be 'rope_interleaved'")
         if self.position is not None and s.position.rotary_dim > s.key_dim:
             raise ValueError("the rotary width is at most the key size")
+        self.by_head = bool(s.conv_taps or s.head_norm_eps is not None or s.temperature is not None)
+        if self.by_head and (s.bias or s.whole_norm_eps is not None or s.position is not None or s.values_are_keys):
+            raise ValueError("heads that are prepared one by one (conv_taps, head_norm_eps, temperature) take no biases, norm over a "
+                             "whole projection, rotation, or keys as values")
+        if s.conv_taps is not None and not (1 <= s.conv_taps <= 33):
+            raise ValueError("conv_taps: 1 to 33")
+        if s.temperature is not None and int(s.temperature[1]) < 1:
+            raise ValueError("temperature: a positive run length")
+        if s.distance_bias is not None and (s.distance_bias[0] < 2 or not s.distance_bias[1] > s.distance_bias[0] // 2):
+            raise ValueError("distance_bias: at least two rows, and a reach beyond half of them")
+        if s.sink and s.fixed_sink is not None:
+            raise ValueError("a learned sink and a fixed one exclude each other")
         self.nq = s.num_heads * s.key_dim
         self.nk = s.num_kv_heads * s.key_dim if s.own_cache else 0
         self.nv = s.num_kv_heads * s.value_dim if (s.own_cache and not s.values_are_keys) else 0
         self.ng = 0 if s.gate is None else s.num_heads if s.gate == "head" else s.num_heads * s.value_dim
         self._slopes = None
         self._sink = None
+        self._taps = None
+        self._bias = None
 
     # ------------------------------------------------------------------ parameters and cache
     def params(self):
@@ -176,6 +208,10 @@ class GatedAttention(Mixer):
                 p["k_norm"] = ParamSpec((self.nk,), role="vector", init="ones_normal")
         if s.sink:
             p["sink"] = ParamSpec((s.num_heads,), role="vector", init="normal:0.5")
+        if s.conv_taps:
+            p["conv"] = ParamSpec((self.nq + self.nk + self.nv, s.conv_taps), role="vector", init="normal:0.5")
+        if s.distance_bias is not None:
+            p["rel"] = ParamSpec((s.distance_bias[0], s.num_heads), role="vector", init="normal:1.0")
         return p
 
     def bind(self, tensors):
@@ -186,6 +222,18 @@ class GatedAttention(Mixer):
         if s.slope_exponent is not None:
             h = torch.arange(1, s.num_heads + 1, dtype=torch.float64)
             self._slopes = torch.exp2(-float(s.slope_exponent) * h / s.num_heads).float().to(self.env.device)
+        if s.fixed_sink is not None:
+            self._sink = torch.full((s.num_heads,), float(s.fixed_sink), dtype=torch.float32, device=self.env.device)
+        if self.by_head:                    # without a convolution: a filter of the token itself
+            self._taps = self.p_conv.contiguous() if s.conv_taps else torch.ones(
+                (self.nq + self.nk + self.nv, 1), dtype=torch.float32, device=self.env.device)
+        if s.distance_bias is not None:     # the table by distance instead of by row, [heads, distances]
+            rows = torch.tensor(distance_rows(*s.distance_bias), dtype=torch.int64, device=self.p_rel.device)
+            self._bias = self.p_rel.float()[rows].t().contiguous()
+
+    def kept_floats(self):
+        s = self.spec
+        return (self.nq + self.nk + self.nv) * (s.conv_taps - 1) if s.conv_taps else 0
 
     def cache_need(self):
         s = self.spec
@@ -220,6 +268,23 @@ class GatedAttention(Mixer):
         proj = ctx.buffer("gated_attention.proj", (T, self.nq + self.nk + self.nv + self.ng), dt, dev)
         ops.linear(x, self.p_in, proj)
         write = bool(ctx.write_cache and s.own_cache)
+        q = ctx.buffer("gated_attention.q", (T, s.num_heads * self.D), dt, dev)
+        if self.by_head:
+            ops.attention_conv_prepare(proj, self._taps, ctx.kept, 0, b, kv, q, s.num_heads, s.num_kv_heads, s.key_dim, s.value_dim,
+                                       self.D, s.head_norm_eps, s.temperature, own_kv=s.own_cache, write_kv=write)
+        else:
+            self._prepare_rows(proj, b, kv, q, write)
+        o = ctx.buffer("gated_attention.o", (T, s.num_heads * self.D), dt, dev)
+        ops.paged_attention(q, kv.k, kv.v, b, kv.block_table, kv.page_size, o, s.num_heads, s.num_kv_heads, self.D,
+                            s.scale, s.window, self._sink, s.chunk, s.softcap, self._slopes, self._bias)
+        if s.gate is not None:
+            ops.attention_gate(o, proj, self.nq + self.nk + self.nv, s.gate == "head", s.num_heads, s.value_dim, self.D)
+        y = ctx.buffer("gated_attention.y", (T, s.hidden_size), torch.float32, dev)
+        ops.linear(o, self.p_o, y)
+        return y
+
+    def _prepare_rows(self, proj, b, kv, q, write: bool):
+        s = self.spec
         biases = None
         if s.bias:
             bq, bk = self.p_bias[:self.nq], self.p_bias[self.nq:self.nq + self.nk]
@@ -227,16 +292,7 @@ class GatedAttention(Mixer):
         norms = None
         if s.whole_norm_eps is not None:
             norms = (self.p_q_norm, self.p_k_norm if write else None)
-        q = ctx.buffer("gated_attention.q", (T, s.num_heads * self.D), dt, dev)
         ops.attention_prepare(proj, 0, self.nq, -1 if (s.values_are_keys or not s.own_cache) else self.nq + self.nk,
                               biases, norms, float(s.whole_norm_eps or 0.0),
                               self.position.tables() if self.position is not None else None, b, kv, q,
                               s.num_heads, s.num_kv_heads, s.key_dim, s.value_dim, self.D, write_kv=write)
-        o = ctx.buffer("gated_attention.o", (T, s.num_heads * self.D), dt, dev)
-        ops.paged_attention(q, kv.k, kv.v, b, kv.block_table, kv.page_size, o, s.num_heads, s.num_kv_heads, self.D,
-                            s.scale, s.window, self._sink, s.chunk, s.softcap, self._slopes)
-        if s.gate is not None:
-            ops.attention_gate(o, proj, self.nq + self.nk + self.nv, s.gate == "head", s.num_heads, s.value_dim, self.D)
-        y = ctx.buffer("gated_attention.y", (T, s.hidden_size), torch.float32, dev)
-        ops.linear(o, self.p_o, y)
-        return y

@@ -95,6 +95,9 @@ class LayerContext:
     kv: Optional[KVView] = None
     state: Optional[torch.Tensor] = None      # [num_slots, *StateNeed.shape]; row = batch.seg_slot
     write_cache: bool = True
+    kept: Optional[torch.Tensor] = None       # float32 [num_slots, n] if the block asked for it (Block.kept_need): what this
+                                              # run keeps per request for itself, whichever cache it owns or reads
+    next_kept: Optional[torch.Tensor] = None  # the same of the run that comes after this one
     position: int = -1                        # index of this run in the model's schedule
     next_block: Any = None                    # the block that runs after this one in this step, or None (a block may
                                               # prepare what its successor's first norm needs)
@@ -172,6 +175,11 @@ class Mixer(Part):
     def cache_need(self):
         return None
 
+    def kept_floats(self) -> int:
+        """How many float32 numbers a run of the mixer keeps per request beside the cache it owns or reads.  It finds them
+        in the first columns of ``ctx.kept``; a new request's are zero."""
+        return 0
+
     def forward(self, x, ctx: LayerContext):
         raise NotImplementedError
 
@@ -184,6 +192,11 @@ class FeedForward(Part):
 class Block(Part):
     def cache_need(self):
         return None
+
+    def kept_need(self):
+        """The ``StateNeed`` of what a run keeps per request for itself (``LayerContext.kept``), or None."""
+        n = self.mixer.kept_floats() if getattr(self, "mixer", None) is not None else 0
+        return StateNeed((n,), torch.float32) if n else None
 
     def first_norm(self):
         """(weight, eps, offset, size) if the block's first act is an RMSNorm of the residual stream, else None."""

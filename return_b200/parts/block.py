@@ -10,7 +10,7 @@ from __future__ import annotations
 import torch
 
 from ..ext import ops
-from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, ParamSpec
+from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, ParamSpec, StateNeed
 
 
 @BLOCKS.register("prenorm")
@@ -246,7 +246,13 @@ class SandwichBlock(Block):
     One kernel sits at every joint: it norms the sublayer's output, adds it to the float32 stream and norms the stream
     for the sublayer that runs next (csrc/elementwise.cu, ``postnorm_add_norm``), also across the border to the next
     block when that block begins with an RMSNorm of the stream (``first_norm``): the normed rows are then left for it
-    under ``sandwich.prenormed`` in the step's scratch.  The block owes the stream nothing when it returns."""
+    under ``sandwich.prenormed`` in the step's scratch.  The block owes the stream nothing when it returns.
+
+    With ``TanhNormSpec`` norms the joint's kernel is another one (csrc/tanh_norm.cu), which also blends the rows that a
+    mixer reads with their predecessors (``token_shift``) and reads and renews what a request kept of its last step.  It
+    needs the stream before and after the add side by side, so the stream goes from one buffer to a second one at the
+    joint inside the layer and back at the joint behind it.  ``layer_scale`` costs nothing: the vector is folded into the
+    weight (and bias) of the norm behind the sublayer."""
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
@@ -258,25 +264,53 @@ class SandwichBlock(Block):
             self._children.update({"feed_forward": self.feed_forward,
                                    "feed_forward_norm": NORMS.build(spec.feed_forward_norm, env),
                                    "feed_forward_post_norm": NORMS.build(spec.feed_forward_post_norm, env)})
-        for name, part in self._children.items():
-            if name.endswith("norm") and getattr(part.spec, "kind", None) != "rmsnorm":
-                raise ValueError("the norms of a sandwich block are RMSNorms")
+        kinds = {getattr(part.spec, "kind", None) for name, part in self._children.items() if name.endswith("norm")}
+        if kinds not in ({"rmsnorm"}, {"tanh_norm"}):
+            raise ValueError("the norms of a sandwich block are all RMSNorms or all squashes ('tanh_norm')")
+        self._tanh = kinds == {"tanh_norm"}
+        self._sublayers = ("mixer",) + (("feed_forward",) if self.feed_forward is not None else ())
+        self._shift_off = (self.mixer.kept_floats() + 3) // 4 * 4       # where a request's last normed row lies in what it keeps
+        self.shift = None
 
     @property
     def graph_safe(self):
         return all(part.graph_safe for part in self._children.values())
 
     def params(self):
-        return {f"{child}.{name}": p for child, part in self._children.items()
-                for name, p in part.params().items()}
+        p = {f"{child}.{name}": ps for child, part in self._children.items() for name, ps in part.params().items()}
+        n = self.spec.mixer_norm.size
+        if self.spec.layer_scale:
+            p.update({f"{sub}_scale": ParamSpec((n,), role="vector", init="ones_normal") for sub in self._sublayers})
+        if self.spec.token_shift:
+            p["shift"] = ParamSpec((n,), role="vector", init="uniform01")
+        return p
 
     def bind(self, tensors):
         for child, part in self._children.items():
             prefix = child + "."
             part.bind({k[len(prefix):]: v for k, v in tensors.items() if k.startswith(prefix)})
+        # what the joints take of the norms behind the sublayers, with the layer's scales folded in
+        self._post = {}
+        for sub in self._sublayers:
+            norm = self._children[sub + "_post_norm"]
+            scale = tensors[sub + "_scale"].float() if self.spec.layer_scale else None
+            if self._tanh:
+                self._post[sub] = norm.triple(scale)
+            elif scale is not None:
+                self._post[sub] = ((norm.spec.offset + norm.p_weight.float()) * scale, norm.spec.eps, 0.0)
+            else:
+                self._post[sub] = self._triple(norm)
+        if self.spec.token_shift:
+            self.shift = tensors["shift"].float().contiguous()
 
     def cache_need(self):
         return self.mixer.cache_need()
+
+    def kept_need(self):
+        if not self.spec.token_shift:
+            return super().kept_need()
+        n = self.spec.mixer_norm.size
+        return StateNeed((self._shift_off + (n + 3) // 4 * 4,), torch.float32)
 
     def batch_tilings(self):
         out = {}
@@ -298,7 +332,46 @@ class SandwichBlock(Block):
     def _triple(norm):
         return norm.p_weight, norm.spec.eps, norm.spec.offset
 
+    def _shift_args(self, kept):
+        if not self.spec.token_shift:
+            return None
+        if kept is None:
+            raise ValueError("a layer that blends its rows with their predecessors needs what its requests kept")
+        return self.shift, kept, self._shift_off
+
+    def _forward_tanh(self, stream, delta, ctx):
+        T, H = stream.shape
+        dt, dev = self.env.act_dtype, stream.device
+        c = self._children
+        held = getattr(ctx.batch, "scratch", None)
+        pre = held.pop("sandwich.prenormed", None) if held is not None else None
+        if delta is None and pre is not None and pre["position"] == ctx.position:
+            a = pre["rows"]
+        else:
+            if delta is not None:
+                ops.tanh_joint(stream, stream, delta, None, None, None)             # what the block before still owes
+            a = ctx.buffer("sandwich.normed_a", (T, H), dt, dev)
+            ops.tanh_joint(stream, None, None, None, c["mixer_norm"].triple(), a, shift=self._shift_args(ctx.kept), batch=ctx.batch)
+        y, post, x = self.mixer.forward(a, ctx), self._post["mixer"], stream
+        if self.feed_forward is not None:
+            b = ctx.buffer("sandwich.normed_b", (T, H), dt, dev)
+            x = ctx.buffer("sandwich.stream_mid", (T, H), torch.float32, dev)
+            ops.tanh_joint(stream, x, y, post, c["feed_forward_norm"].triple(), b)
+            y, post = self.feed_forward.forward(b, ctx), self._post["feed_forward"]
+        nxt = ctx.next_block
+        ahead = held is not None and isinstance(nxt, SandwichBlock) and nxt._tanh and nxt.spec.mixer_norm.size == H
+        if ahead and (x is not stream or not nxt.spec.token_shift):
+            rows = ctx.buffer("sandwich.normed_a", (T, H), dt, dev)                  # this block's own normed input is used up by now
+            ops.tanh_joint(x, stream, y, post, nxt._children["mixer_norm"].triple(), rows, shift=nxt._shift_args(ctx.next_kept),
+                           batch=ctx.batch)
+            held["sandwich.prenormed"] = {"rows": rows, "position": ctx.position + 1}
+        else:
+            ops.tanh_joint(x, stream, y, post, None, None)
+        return None
+
     def forward(self, stream, delta, ctx):
+        if self._tanh:
+            return self._forward_tanh(stream, delta, ctx)
         T, H = stream.shape
         dt, dev = self.env.act_dtype, stream.device
         c = self._children
@@ -309,19 +382,25 @@ class SandwichBlock(Block):
         else:
             a = ctx.buffer("sandwich.normed_a", (T, H), dt, dev)
             c["mixer_norm"].add_forward(stream, delta, a)       # stream += delta; a = norm(stream)
+        if self.spec.token_shift:
+            mu, kept, off = self._shift_args(ctx.kept)
+            shifted = ctx.buffer("sandwich.shifted", (1, T, H), dt, dev)
+            ops.token_shift_mix(a, mu.view(1, H), kept, off, ctx.batch, shifted)
+            ops.conv_state_update(a, 2, kept, off, ctx.batch, H)                # after every token has read the old one
+            a = shifted[0]
         mixed = self.mixer.forward(a, ctx)
-        last = mixed, c["mixer_post_norm"]
+        last = mixed, self._post["mixer"]
         if self.feed_forward is not None:
             b = ctx.buffer("sandwich.normed_b", (T, H), dt, dev)
-            ops.postnorm_add_norm(stream, mixed, self._triple(c["mixer_post_norm"]), self._triple(c["feed_forward_norm"]), b)
-            last = self.feed_forward.forward(b, ctx), c["feed_forward_post_norm"]
+            ops.postnorm_add_norm(stream, mixed, last[1], self._triple(c["feed_forward_norm"]), b)
+            last = self.feed_forward.forward(b, ctx), self._post["feed_forward"]
         nxt = ctx.next_block.first_norm() if ctx.next_block is not None and hasattr(ctx.next_block, "first_norm") else None
         if nxt is not None and nxt[3] == H and held is not None and isinstance(ctx.next_block, SandwichBlock):
             rows = ctx.buffer("sandwich.normed_a", (T, H), dt, dev)      # this block's own normed input is used up by now
-            ops.postnorm_add_norm(stream, last[0], self._triple(last[1]), (nxt[0], nxt[1], nxt[2]), rows)
+            ops.postnorm_add_norm(stream, last[0], last[1], (nxt[0], nxt[1], nxt[2]), rows)
             held["sandwich.prenormed"] = {"rows": rows, "position": ctx.position + 1}
         else:
-            ops.postnorm_add_norm(stream, last[0], self._triple(last[1]))
+            ops.postnorm_add_norm(stream, last[0], last[1])
         return None
 
 

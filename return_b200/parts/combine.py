@@ -18,6 +18,9 @@ class MixerSum(Mixer):
         if not (len(spec.names) == len(spec.mixers) == len(spec.scales) == 2):
             raise ValueError("a sum of mixers has two children, each with a name and a scale")
         self.children = {name: MIXERS.build(m, env) for name, m in zip(spec.names, spec.mixers)}
+        keeping = [name for name, child in self.children.items() if child.kept_floats()]
+        if keeping:
+            raise ValueError(f"children of a sum of mixers keep nothing of their own beside a cache or state: {keeping} do")
 
     @property
     def graph_safe(self):

@@ -2,9 +2,9 @@
 
 ``clamped_glu``: y = down( g * sigmoid(alpha g) * (u + 1) ), g = min(gate(x), limit), u = clamp(up(x), -limit, limit).
 ``moe``: a router (float32 logits, optionally with a bias per expert, softmax over all experts, optionally only the
-experts of the best groups, the top few chosen, their scores renormalised) picks experts per token; the experts'
-outputs are summed with those weights, in the order of falling score, and a shared feed-forward may run for every token
-beside them.  The experts are capped gated units or plain ones (silu(gate) * up), which are the same kernel with no
+experts of the best groups, the top few chosen, their scores renormalised or taken as they are) picks experts per token;
+the experts' outputs are summed with those weights (or each expert reads its input times its weight), in the order of
+falling score, and a shared feed-forward may run for every token beside them.  The experts are capped gated units or plain ones (silu(gate) * up), which are the same kernel with no
 cap, alpha = 1 and nothing added to the up part.
 
 The experts' weights are stacked: ``experts.gate_up`` [E * 2F, hidden] (per expert its gate rows, then its up rows)
@@ -92,9 +92,10 @@ class MixtureOfExperts(FeedForward):
         expert_of = work_buffer(ctx, "moe.expert_of", (T, s.top), torch.int32, dev)
         weight = work_buffer(ctx, "moe.weight", (T, s.top), torch.float32, dev)
         ops.moe_route(logits, expert_of, weight, s.top, s.groups, s.keep_groups, s.renorm_tiny, bias=self.router_bias,
-                      score=s.score, group_top=s.group_top, scale=s.weight_scale)
+                      score=s.score, group_top=s.group_top, scale=s.weight_scale, renorm=s.renormalize)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
         y = work_buffer(ctx, "moe.y", (T, s.hidden_size), dt, dev)
         limit, alpha, shift = self.unit
-        ops.moe_experts(x, self.gate_up, self.down, expert_of, weight, shared, y, limit, alpha, ctx, shift=shift)
+        ops.moe_experts(x, self.gate_up, self.down, expert_of, weight, shared, y, limit, alpha, ctx, shift=shift,
+                        weigh_input=s.weigh_input)
         return y

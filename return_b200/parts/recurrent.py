@@ -451,6 +451,59 @@ class GatedDelta(_StateMixer):
         return self._project_out(mixed, ctx)
 
 
+@MIXERS.register("general_delta")
+class GeneralDelta(_StateMixer):
+    """``GeneralDeltaSpec``: one product gives [r | k | v | gate | rate | low rank]; the decay's second product follows; a
+    small kernel makes decays and removal vectors; the scan, per-head norm, gate and output projection are those of the
+    other state mixers.  The request's state row holds S."""
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        s = spec
+        self.H, self.D, self.V = s.num_heads, s.key_dim, s.key_dim
+        if self.D > ops.SCAN_MAX_KEY_DIM:
+            raise ValueError(f"key_dim={self.D}: the scan kernel holds up to {ops.SCAN_MAX_KEY_DIM} key rows a head")
+        if s.decay_rank <= 0:
+            raise ValueError("decay_rank must be positive")
+        self.s_floats = self.H * _pad8(self.D) * self.V
+
+    def params(self):
+        s = self.spec
+        HD = self.H * self.D
+        return {"in": ParamSpec((5 * HD + s.decay_rank, s.hidden_size)),                    # r, k, v, gate, rate, low rank of the decay
+                "decay_up": ParamSpec((HD, s.decay_rank), init="normal:0.2"),
+                "decay_bias": ParamSpec((HD,), role="vector", init="normal:0.5"),
+                "rate_bias": ParamSpec((HD,), role="vector", init="normal:0.5"),
+                "norm": ParamSpec((HD,), role="vector", init="ones_normal"),
+                "o": ParamSpec((s.hidden_size, HD))}
+
+    def bind(self, tensors):
+        super().bind(tensors)
+        self._w0, self._rate_bias = self.p_decay_bias.float().contiguous(), self.p_rate_bias.float().contiguous()
+
+    def cache_need(self):
+        return StateNeed((self.s_floats,), torch.float32)
+
+    def forward(self, x, ctx):
+        s, b = self.spec, ctx.batch
+        T, dev, dt = x.shape[0], x.device, x.dtype
+        HD = self.H * self.D
+        proj = ctx.buffer("general_delta.in", (T, 5 * HD + s.decay_rank), dt, dev)
+        ops.linear(x, self.p_in, proj)
+        low = ctx.buffer("general_delta.low", (T, s.decay_rank), dt, dev)
+        ops.activation(proj[:, 5 * HD:], low, "tanh")
+        decay = ctx.buffer("general_delta.decay", (T, HD), torch.float32, dev)
+        ops.linear(low, self.p_decay_up, decay)
+        removal = ctx.buffer("general_delta.removal", (T, HD), torch.float32, dev)
+        ops.general_delta_prep(proj, HD, 4 * HD, self._rate_bias, self._w0, s.decay_scale, s.unit_eps, decay, removal, self.H, self.D)
+        o = ctx.buffer("general_delta.o", (T, HD), torch.float32, dev)
+        ops.linear_scan(ops.SCAN_GENERAL_DELTA, proj, proj[:, HD:], proj[:, 2 * HD:], decay, removal, ctx.state, (0, 0, 0), b, o,
+                        self.H, self.H, self.D, self.V)
+        mixed = ctx.buffer("general_delta.mixed", (T, HD), dt, dev)
+        ops.head_norm_gate(o, proj[:, 3 * HD:], self.p_norm, 2, 1, s.eps, mixed, self.H, self.V)
+        return self._project_out(mixed, ctx)
+
+
 @MIXERS.register("gated_linear_recurrence")
 class GatedLinearRecurrence(Mixer):
     """``GatedLinearRecurrenceSpec``: one product gives [y | x]; a kernel convolves x over time (reading the request's

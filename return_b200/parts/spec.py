@@ -25,6 +25,14 @@ class NormSpec:
 
 
 @dataclass(frozen=True)
+class TanhNormSpec:
+    """An elementwise squash in the place of a norm: y = tanh(alpha * x) * w + b with one number alpha and vectors w and b
+    over the last ``size`` elements.  No mean, no variance."""
+    size: int
+    kind: str = "tanh_norm"
+
+
+@dataclass(frozen=True)
 class RopeSpec:
     """Half-split rotary encoding of the first ``rotary_dim`` elements of a head."""
     rotary_dim: int
@@ -134,7 +142,14 @@ class GatedAttentionSpec:
     number per head whose exponential joins the softmax's denominator); ``gate`` "head" (a head's output times the
     logistic of one projected number) or "element" (one per value element).  ``own_cache`` False: the layer has no key
     and value projections and reads the cache that another run of the schedule wrote.  ``cache_window``: how many of the
-    latest keys the cache must keep for this layer and every layer that reads its cache (None: all)."""
+    latest keys the cache must keep for this layer and every layer that reads its cache (None: all).
+    Heads prepared one by one instead of as a whole row (these exclude ``bias``, ``whole_norm_eps``, ``position`` and
+    ``values_are_keys``): ``conv_taps`` n (every channel of the q, k and v projections passes a causal filter over the last
+    n tokens; the run keeps a request's last n - 1 projected rows); ``head_norm_eps`` (each q and k head over its root mean
+    square, no weight); ``temperature`` (coef, every): q at position p times 1 + coef ln(floor((p + 1) / every) + 1).
+    ``distance_bias`` (rows, reach): a learned table [rows, heads] is added to the scores by the distance n = i - j: row n
+    below half = rows // 2, else min(rows - 1, half + floor(ln(n / half) / ln(reach / half) * (rows - half))).
+    ``fixed_sink``: a number whose exponential joins every head's denominator (0: one is added to it)."""
     hidden_size: int
     num_heads: int
     num_kv_heads: int
@@ -153,6 +168,11 @@ class GatedAttentionSpec:
     gate: Optional[str] = None
     own_cache: bool = True
     cache_window: Optional[int] = None
+    conv_taps: Optional[int] = None
+    head_norm_eps: Optional[float] = None
+    temperature: Optional[Tuple[float, int]] = None
+    distance_bias: Optional[Tuple[int, float]] = None
+    fixed_sink: Optional[float] = None
     kind: str = "gated_attention"
 
 
@@ -207,6 +227,24 @@ class GatedDeltaSpec:
     eps: float
     unit_eps: float = 1e-6
     kind: str = "gated_delta"
+
+
+@dataclass(frozen=True)
+class GeneralDeltaSpec:
+    """Delta rule whose removal does not run along the key alone and whose decay is per head and key row.  q, k, v and an
+    output gate are plain projections (``num_heads`` heads of ``key_dim``, values of the same size); the decay is
+    w = exp(-``decay_scale`` sigmoid(W2 tanh(W1 x) + w0)) through a low rank ``decay_rank``; the removal rate is
+    r = sigmoid(W_a x + b).  With u = k / sqrt(sum k^2 + ``unit_eps``): S <- diag(w) S - (r * u)(u^T S) + k v^T, both terms of
+    the old S; o = S^T q.  Each head's o is divided by its root mean square, weighted over all heads, gated by sigmoid of
+    the gate projection, and projected out."""
+    hidden_size: int
+    num_heads: int
+    key_dim: int
+    decay_rank: int
+    eps: float
+    decay_scale: float
+    unit_eps: float = 1e-6
+    kind: str = "general_delta"
 
 
 @dataclass(frozen=True)
@@ -334,7 +372,9 @@ class MoESpec:
     the logits.  ``expert`` is a ``ClampedGLUSpec`` or a ``SwiGLUSpec`` with rows not woven.  ``shared``: a feed-forward
     that runs for every token and is added, or None.  ``score`` "sigmoid": every expert's score is the logistic of its own
     logit instead of a softmax over all.  ``group_top`` 2: a group is ranked by the sum of its two largest scores instead of
-    its largest.  ``weight_scale``: a factor on the weights after they were divided by their sum."""
+    its largest.  ``weight_scale``: a factor on the weights after they were divided by their sum.  ``renormalize`` False: the
+    chosen scores are the weights as they are.  ``weigh_input`` True: a weight multiplies its expert's input instead of its
+    output."""
     hidden_size: int
     num_experts: int
     top: int
@@ -348,18 +388,25 @@ class MoESpec:
     score: str = "softmax"
     group_top: int = 1
     weight_scale: float = 1.0
+    renormalize: bool = True
+    weigh_input: bool = False
 
 
 @dataclass(frozen=True)
 class SandwichBlockSpec:
     """x += post_a(mixer(pre_a(x))); x += post_b(feed_forward(pre_b(x))): a norm before and after each sublayer.
-    ``feed_forward`` None: the layer has none (and no norms for it)."""
+    ``feed_forward`` None: the layer has none (and no norms for it).  The norms are all RMSNorms or all ``TanhNormSpec``.
+    ``layer_scale``: a learned vector per sublayer multiplies its normed output element by element.  ``token_shift``: with
+    a learned vector mu the mixer reads a_t + (a_(t-1) - a_t) * mu in the place of its normed input a_t (a_(-1) = 0); the
+    run keeps a request's last a."""
     mixer: Any
     feed_forward: Any
     mixer_norm: Any
     mixer_post_norm: Any
     feed_forward_norm: Any = None
     feed_forward_post_norm: Any = None
+    layer_scale: bool = False
+    token_shift: bool = False
     kind: str = "sandwich"
 
 

@@ -246,6 +246,10 @@ def random_parameters(params: Dict[str, "ParamSpec"], sources: Dict[str, Source]
                 dst[row:row + t.shape[0]].copy_(t)
                 row += t.shape[0]
                 continue
+            if not shp:                            # a single number
+                dst[row:row + 1].copy_(random_tensor(seed, n, shp, init, dt, device))
+                row += 1
+                continue
             if 0 < len(shp) < dst.dim():           # vectors stacked into a matrix: each is one row
                 dst[row].copy_(random_tensor(seed, n, shp, init, dt, device))
                 row += 1
