@@ -430,8 +430,7 @@ def run_workload(name: str, layers: int = 0, new: int = 0) -> Dict[str, object]:
 def kernel_scan(mode=0, batch=1, tokens=2048, heads=16, kv_heads=0, dim=128, vdim=128, iters=10, warmup=3) -> Dict[str, object]:
     """The recurrence kernel of the mixers with a matrix state alone: ``batch`` segments of ``tokens`` tokens each
     (tokens = 1: a decode step).  mode 0: fixed decay, 1: matrix memory, 2: delta rule, 3: row decays with a bonus, 4: state
-    space.  Reports the time of a launch,
-    the float32 operations per second, and the bandwidth on the states (each read and written once)."""
+    space, 6: general delta rule.  Reports the time of a launch, the float32 operations per second, and the bandwidth on the states (each read and written once)."""
     from types import SimpleNamespace
     from .ext import ops
     dev = torch.device("cuda:0")
@@ -457,7 +456,10 @@ def kernel_scan(mode=0, batch=1, tokens=2048, heads=16, kv_heads=0, dim=128, vdi
     else:
         ga, gb = torch.sigmoid(rnd(T, heads * dim) + 3.0).contiguous(), torch.sigmoid(rnd(T, heads)).contiguous()
     extra = None
-    if mode == ops.SCAN_BONUS:
+    if mode == 6:
+        gb = (torch.sigmoid(rnd(T, heads * dim)) * k).contiguous()
+        qb, kb, vb = (x.bfloat16() for x in (q, k, v))
+    elif mode == ops.SCAN_BONUS:
         gb, extra = None, rnd(heads * dim)
     elif mode == ops.SCAN_SSM:
         extra = rnd(heads)
@@ -465,8 +467,11 @@ def kernel_scan(mode=0, batch=1, tokens=2048, heads=16, kv_heads=0, dim=128, vdi
     fns = [(lambda st=st: ops.linear_scan(mode, q, k, v, ga, gb, st, (0, n_off, m_off), b, out, heads, G, dim, vdim,
                                           q_scale=dim ** -0.5 if mode < ops.SCAN_BONUS else 1.0, cap=15.0, extra=extra))
            for st in states]
+    if mode == 6:
+        assert G == heads and dim == vdim, "the general delta rule has as many key heads as value heads, of one size"
+        fns = [(lambda st=st: ops.general_delta_scan(qb, kb, vb, ga, gb, st, 0, b, out, heads, dim)) for st in states]
     ms = _time_kernels(fns, iters, warmup)
-    flops = T * heads * dim * vdim * (6.0 if mode == ops.SCAN_DELTA else 4.0)
+    flops = T * heads * dim * vdim * (6.0 if mode in (ops.SCAN_DELTA, 6) else 4.0)
     return {"kernel": "linear_scan", "mode": mode, "batch": batch, "tokens": tokens, "heads": heads, "dim": dim, "vdim": vdim,
             "ms": round(ms, 4), "ns_per_token": round(ms * 1e6 / tokens, 1), "tflops_f32": round(flops / ms / 1e9, 3),
             "state_gbs": round(2.0 * batch * s_floats * 4 / ms / 1e6, 1)}
@@ -893,3 +898,101 @@ def compare_duvadra(size: str, tokens: int, batch: int, steps: int, warmup: int,
         del r["prefill_kernels"], r["decode_kernels"]
     return {"size": size, "width": W, "ff": ff, "heads": H, "kv_heads": G, "layers": L, "tokens": tokens, "batch": batch,
             "window": window, "block": 8192, "duvadra": new, "nozizen": old, "kernels": kernels}
+
+
+def losorax_raw_config(width: int, ff: int, heads: int, kv_heads: int, layers: int, vocab: int, bias_rows: int = 32,
+                       bias_max: int = 1024) -> dict:
+    """A Losorax configuration whose mixers carry as many heads of 128 as the attention of a Qwen3 model of this width: of
+    every four layers the first is an attention with keys of its own, the second one on the first's keys and values, the
+    third a general delta rule (states of 128 x 128, a decay of rank 64), the fourth an attention again; four taps, a bias
+    table of 32 rows that reaches 1,024 positions; the first and fourth feed-forwards are gated units, the others 32
+    experts of a quarter of the dense size each, four of them a token."""
+    dense = {"kind": "dense", "ff": ff}
+    experts = {"kind": "moe", "router": {"experts": 32, "top": 4}, "expert": {"ff": ff // 4}}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "conv": 4, "bias_rows": bias_rows,
+           "bias_max": bias_max, "q_temp": {"coef": 0.2, "every": 512}}
+    delta = {"heads": heads, "dim": 128, "decay_rank": 64}
+    out = []
+    for i in range(layers):
+        k = i % 4
+        if k == 2:
+            out.append({"type": "general_delta", "mixer": delta, "mlp": experts})
+        else:
+            out.append({"type": "attention", "mixer": dict(att, kv_from=i - 1) if k == 1 else att, "mlp": experts if k == 1 else dense})
+    return {"architecture": "Losorax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": out}
+
+
+def compare_losorax(size: str, tokens: int, batch: int, steps: int, warmup: int, hbm_gbs: float, bf16_tflops: float):
+    """The Losorax design beside the Duvadra decoder (the nearest the engine has: attention with score options on shared
+    keys, a delta rule on the scan kernel, gated units beside experts with logistic scores) at equal width, feed-forward,
+    layer count and heads: throughput of both, and how far the kernels of each mechanism are from their rooflines beside
+    the like kernels of the other model.  Rooflines: the scan over decoded tokens against the copy bandwidth (every state
+    read and written once), over a prompt against the tensor peak (6 T heads dim vdim operations, although the scans run
+    in float32 on the CUDA cores); attention over decoded tokens against the copy bandwidth (the keys and values a query
+    sees read once), over a prompt against the tensor peak (the causal half; both on the kernels with the score options);
+    what prepares the attentions' rows (the projections read, the padded queries and the pages written), what joins two
+    sublayers (the float32 stream read and written, the sublayer's output read, the normed rows written) and what
+    surrounds the scan against the copy bandwidth; the experts' products of a prompt against the tensor peak and of
+    decoded tokens against the copy bandwidth (each reached expert read once)."""
+    from .config.duvadra_config import DuvadraConfig
+    from .config.losorax_config import LosoraxConfig
+    sz = DESIGN_SIZES[size]
+    W, ff, H, G, L, V = sz["width"], sz["ff"], sz["heads"], sz["kv_heads"], sz["layers"], sz["vocab"]
+    raw, old_raw = losorax_raw_config(W, ff, H, G, L, V), duvadra_raw_config(W, ff, H, G, L, V)
+    new = measure_design(LosoraxConfig(raw), tokens, batch, steps, warmup)
+    old = measure_design(DuvadraConfig(old_raw), tokens, batch, steps, warmup)
+    D, F, top, E, window = 128, ff // 4, 4, 32, 1024
+    kinds = [layer["type"] for layer in raw["layers"]]
+    n_att, n_delta = kinds.count("attention"), kinds.count("general_delta")
+    n_own = sum(1 for layer in raw["layers"] if layer["type"] == "attention" and "kv_from" not in layer["mixer"])
+    n_moe = sum(1 for layer in raw["layers"] if layer["mlp"]["kind"] == "moe")
+    o_kinds = [layer["type"] for layer in old_raw["layers"]]
+    o_blocks, o_windows, o_delta = o_kinds.count("attention"), o_kinds.count("parallel") + o_kinds.count("parallel_2"), o_kinds.count("parallel")
+    o_moe = sum(1 for layer in old_raw["layers"] if layer["mlp"]["kind"] == "moe")
+    distinct = E * (1.0 - (1.0 - 1.0 / E) ** (batch * top))
+    frac = lambda work, ms, peak: round(work / (ms * 1e-3) / peak, 4) if ms > 0 else None
+    k_new, k_old, d_new, d_old = new["prefill_kernels"], old["prefill_kernels"], new["decode_kernels"], old["decode_kernels"]
+    att_dec = ("attn_decode", "attn_combine")
+    att_pf = ("attn_prefill_kernel", "attn_prefill_tc5_kernel<true>")
+    moe_pf, moe_dec = ("moe_grouped_gemm", "moe_tc5"), ("moe_pair_linear", "moe_grouped_gemm")
+    moe_small = ("clamped_glu", "moe_combine", "moe_route", "moe_sort", "moe_gather")
+    hbm, peak = hbm_gbs * 1e9, bf16_tflops * 1e12
+    row = lambda times, names, work, roof, key: {"ms": round(_kernel_ms(times, *names), 4), key: frac(work, _kernel_ms(times, *names), roof)}
+    # bytes a token: every attention reads its projection row and writes its query row, an owner also keys and values
+    prep_new = 2.0 * D * (n_att * 2 * H + n_own * 4 * G)
+    # the block attentions (half of them own keys), the windowed ones (their k serves as v in one kind of the two)
+    prep_old = 2.0 * D * ((o_blocks + o_windows) * 2 * H + (o_blocks / 2 + o_delta) * 4 * G + (o_windows - o_delta) * 3 * G)
+    kernels = {
+        "decode_scan_losorax": row(d_new, ("general_delta_scan",), 2.0 * 4 * D * D * H * n_delta * batch, hbm, "of_hbm"),
+        "decode_scan_duvadra": row(d_old, ("linear_scan",), 2.0 * 4 * D * D * H * o_delta * batch, hbm, "of_hbm"),
+        "prefill_scan_losorax": row(k_new, ("general_delta_scan",), 6.0 * tokens * D * D * H * n_delta, peak, "of_bf16_peak"),
+        "prefill_scan_duvadra": row(k_old, ("linear_scan",), 6.0 * tokens * D * D * H * o_delta, peak, "of_bf16_peak"),
+        "decode_attention_losorax": row(d_new, att_dec, 2.0 * 2 * G * D * batch * tokens * n_att, hbm, "of_hbm"),
+        "decode_attention_duvadra": row(d_old, att_dec, 2.0 * 2 * G * D * batch * (tokens * o_blocks + min(tokens, window) * o_windows), hbm, "of_hbm"),
+        "prefill_attention_losorax": row(k_new, att_pf, 4.0 * tokens * tokens / 2 * H * D * n_att, peak, "of_bf16_peak"),
+        "prefill_attention_blocks_duvadra": row(k_old, att_pf, 4.0 * tokens * tokens / 2 * H * D * o_blocks, peak, "of_bf16_peak"),
+        "prefill_rows_losorax": row(k_new, ("attn_conv_prep",), prep_new * tokens, hbm, "of_hbm"),
+        "prefill_rows_duvadra": row(k_old, ("attn_prep",), prep_old * tokens, hbm, "of_hbm"),
+        # the float32 stream read and written, the sublayer's output read (float32 from the mixers, bfloat16 from the
+        # feed-forwards), the normed rows written, twice a layer
+        "prefill_joint_losorax": row(k_new, ("tanh_joint",), L * tokens * W * (2.0 * 2 * 4 + 4 + 2 + 2 * 2), hbm, "of_hbm"),
+        "prefill_add_norm_duvadra": row(k_old, ("add_dual_norm",), L * tokens * W * (2.0 * 2 * 4 + 4 + 2 + 2 * 2), hbm, "of_hbm"),
+        # beside the scan: k and a read, decays read and written, removal vectors written; the read-out and the gate read,
+        # the gated rows written (the other model: q, k, v read and written in float32 behind their convolution)
+        "prefill_scan_sides_losorax": row(k_new, ("general_delta_prep", "head_norm_gate"), n_delta * tokens * H * D * (2.0 * 2 + 3 * 4 + 4 + 2 + 2), hbm, "of_hbm"),
+        "prefill_scan_sides_duvadra": row(k_old, ("delta_prep", "head_norm_gate"), o_delta * tokens * D * ((2.0 * G + H) * 6 + H * 8), hbm, "of_hbm"),
+        "prefill_experts_losorax": row(k_new, moe_pf, n_moe * 2.0 * tokens * top * 3 * F * W, peak, "of_bf16_peak"),
+        "prefill_experts_duvadra": row(k_old, moe_pf, o_moe * 2.0 * tokens * top * 3 * F * W, peak, "of_bf16_peak"),
+        "decode_experts_losorax": row(d_new, moe_dec, n_moe * 2.0 * distinct * 3 * F * W, hbm, "of_hbm"),
+        "decode_experts_duvadra": row(d_old, moe_dec, o_moe * 2.0 * distinct * 3 * F * W, hbm, "of_hbm"),
+    }
+    for name, names in (("rows", ("attn_conv_prep", "attn_prep", "attn_gate")), ("joints", ("tanh_joint", "add_dual_norm")),
+                        ("scan_sides", ("delta_prep", "head_norm_gate", "conv_state_update", "activation_kernel")), ("expert_helpers", moe_small)):
+        for model, pf, dec in (("losorax", k_new, d_new), ("duvadra", k_old, d_old)):
+            kernels[f"decode_{name}_{model}"] = {"ms": round(_kernel_ms(dec, *names), 4)}
+            if name == "expert_helpers":
+                kernels[f"prefill_{name}_{model}"] = {"ms": round(_kernel_ms(pf, *names), 4)}
+    for r in (new, old):
+        del r["prefill_kernels"], r["decode_kernels"]
+    return {"size": size, "width": W, "ff": ff, "heads": H, "kv_heads": G, "layers": L, "tokens": tokens, "batch": batch,
+            "bias_rows": 32, "bias_max": 1024, "losorax": new, "duvadra": old, "kernels": kernels}

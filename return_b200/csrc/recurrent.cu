@@ -6,8 +6,6 @@
 //     fixed decay:     S <- a S + k v^T                                   o = S^T q
 //     delta rule:      S <- g * S (row i by g_i);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //     delta rule, one decay a head: the same with a scalar g per token and head
-//     general delta:   S <- g * S (row i by g_i) - c (k^T S) + k v^T, both terms of the old S;  o = S^T q: the removal has a
-//                      vector c of its own (per token, head and key row) instead of running along the key
 //     matrix memory:   m' = max(f + m, i);  a = exp(f + m - m'),  b = exp(i - m');
 //                      S <- a S + b k v^T;  n <- a n + b k;  o = S^T q / (max(|n . q|, exp(-m')) + 1e-6)
 //     bonus rule:      o = (S + diag(u) k v^T)^T q;  S <- g * S (row i by g_i) + k v^T: the token's own pair is read with
@@ -39,17 +37,15 @@
 #define MODE_BONUS 3
 #define MODE_SSM 4
 #define MODE_DELTA_HEAD 5
-#define MODE_GENERAL_DELTA 6
 
 struct ScanArgs {
     const void* q; const void* k; const void* v;        // (t, head, i) at base + t * ld + head * dim + i
     int q_ld, k_ld, v_ld;
     int q_f32, k_f32, v_f32;                            // 1: float32, 0: bfloat16
-    const float* gate_a;      // decay: [H] decays; memory: [T, 2H] gate pre-activations (input, forget); delta, general delta
-                              // and bonus: [T, H*D] row decays; state space: [T, H] decays
+    const float* gate_a;      // decay: [H] decays; memory: [T, 2H] gate pre-activations (input, forget); delta and bonus:
+                              // [T, H*D] row decays; state space: [T, H] decays
     const float* gate_b;      // memory: [2H] gate biases; delta: [T, H] beta; state space: [T, H] steps
                               // delta with one decay a head: gate_a [T, H] decays, gate_b [T, H] beta
-                              // general delta: gate_b [T, H*D] removal vectors
     const float* extra;       // bonus: [H, D] weights of the token's own pair; state space: [H] skip weights
     float cap, q_scale;
     float* state;             // [slots, state_stride]
@@ -86,14 +82,12 @@ linear_scan_kernel(const ScanArgs a) {
     // NR values as 16-byte pieces, and the eight runs that one such request covers fall on different banks
     constexpr int RS = NR + 4, DS = R * RS;
     constexpr int PER = SCAN_TC * DP / SCAN_THREADS;   // q (and k) elements of a chunk that a thread brings in
-    constexpr bool ROW_REMOVAL = MODE == MODE_GENERAL_DELTA;                 // a removal vector per token and head
-    constexpr bool ROW_DECAY = MODE == MODE_DELTA || MODE == MODE_BONUS || ROW_REMOVAL;      // a decay per token, head and key row
+    constexpr bool ROW_DECAY = MODE == MODE_DELTA || MODE == MODE_BONUS;     // a decay per token, head and key row
     static_assert(SCAN_TC * SCAN_COLS <= SCAN_THREADS && (SCAN_TC * DP) % SCAN_THREADS == 0, "staging by all threads");
     pdl_wait();
     __shared__ __align__(16) float sq[SCAN_TC][DS];
     __shared__ __align__(16) float sk[SCAN_TC][DS];
     __shared__ __align__(16) float sg[ROW_DECAY ? SCAN_TC : 1][DS];
-    __shared__ __align__(16) float sc[ROW_REMOVAL ? SCAN_TC : 1][ROW_REMOVAL ? DS : 4];
     __shared__ float sv[SCAN_TC][SCAN_COLS];
     __shared__ float sa[SCAN_TC], sb[SCAN_TC];
     const int seg = blockIdx.z, h = blockIdx.y, j0 = blockIdx.x * SCAN_COLS;
@@ -139,7 +133,7 @@ linear_scan_kernel(const ScanArgs a) {
     // product right behind a load would make the warp wait for it there, before the arithmetic it is meant to hide
     // behind.  Converting, scaling and the gates' transcendental functions happen on the way to shared memory.
     uint32_t rq[PER], rk[PER], rv = 0u;
-    float rg[ROW_DECAY ? PER : 1], rc[ROW_REMOVAL ? PER : 1], ra = 0.f, rb = 0.f;
+    float rg[ROW_DECAY ? PER : 1], ra = 0.f, rb = 0.f;
     auto raw = [](const void* p, int f32, size_t i) -> uint32_t {
         return f32 ? ((const uint32_t*)p)[i] : (uint32_t)((const unsigned short*)p)[i];
     };
@@ -154,7 +148,6 @@ linear_scan_kernel(const ScanArgs a) {
             rq[u] = live ? raw(a.q, a.q_f32, t * a.q_ld + (size_t)kvh * D + i) : 0u;
             rk[u] = live ? raw(a.k, a.k_f32, t * a.k_ld + (size_t)kvh * D + i) : 0u;
             if (ROW_DECAY) rg[u] = live ? a.gate_a[(t * H + h) * D + i] : 1.f;
-            if (ROW_REMOVAL) rc[u] = live ? a.gate_b[(t * H + h) * D + i] : 0.f;
         }
         if (tid < SCAN_TC * SCAN_COLS) {
             const int tt = tid / SCAN_COLS, c = tid - tt * SCAN_COLS;
@@ -181,7 +174,6 @@ linear_scan_kernel(const ScanArgs a) {
             sq[tt][at] = cooked(rq[u], a.q_f32) * a.q_scale;
             sk[tt][at] = cooked(rk[u], a.k_f32);
             if (ROW_DECAY) sg[tt][at] = rg[u];
-            if (ROW_REMOVAL) sc[tt][at] = rc[u];
         }
         if (tid < SCAN_TC * SCAN_COLS) sv[tid / SCAN_COLS][tid % SCAN_COLS] = cooked(rv, a.v_f32);
         if (tid < SCAN_TC) {
@@ -247,30 +239,6 @@ linear_scan_kernel(const ScanArgs a) {
             for (int ii = 0; ii < NR; ++ii) {
                 S[ii] = fmaf(fa, S[ii], kr[ii] * vdt);
                 o4[ii & 3] = fmaf(S[ii], qr[ii], o4[ii & 3]);
-            }
-        } else if (MODE == MODE_GENERAL_DELTA) {
-            // what the old state holds for the key; the decay and the new pair do not wait for the sum over the lanes
-            float k4[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-            for (int i4 = 0; i4 < NR; i4 += 4) {
-                const float4 g4 = *(const float4*)&sg[tt][r * RS + i4];
-                const float gr[4] = {g4.x, g4.y, g4.z, g4.w};
-#pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    k4[i] = fmaf(S[i4 + i], kr[i4 + i], k4[i]);
-                    S[i4 + i] = fmaf(gr[i], S[i4 + i], kr[i4 + i] * vj);
-                }
-            }
-            const float kv = lanes_sum<R>((k4[0] + k4[1]) + (k4[2] + k4[3]));
-#pragma unroll
-            for (int i4 = 0; i4 < NR; i4 += 4) {
-                const float4 c4 = *(const float4*)&sc[tt][r * RS + i4];
-                const float cr[4] = {c4.x, c4.y, c4.z, c4.w};
-#pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    S[i4 + i] = fmaf(-cr[i], kv, S[i4 + i]);
-                    o4[i] = fmaf(S[i4 + i], qr[i4 + i], o4[i]);
-                }
             }
         } else {
             if (MODE == MODE_DELTA_HEAD) {
@@ -367,8 +335,8 @@ static int launch_scan(const ScanArgs& a, int segments, cudaStream_t st) {
     return rb_launch_pdl(linear_scan_kernel<MODE, 32, R>, grid, dim3(SCAN_THREADS), 0, st, a);
 }
 
-// mode: 0 fixed decay, 1 matrix memory, 2 delta rule, 3 bonus rule, 4 state space, 5 delta rule with one decay a head,
-// 6 general delta.  The arguments are those of ScanArgs, in its order.
+// mode: 0 fixed decay, 1 matrix memory, 2 delta rule, 3 bonus rule, 4 state space.  The arguments are those of
+// ScanArgs, in its order.
 RB_EXPORT int rb_linear_scan(int mode, const void* q, const void* k, const void* v, int q_ld, int k_ld, int v_ld,
                              int q_f32, int k_f32, int v_f32, const float* gate_a, const float* gate_b,
                              const float* extra, float cap,
@@ -387,7 +355,6 @@ RB_EXPORT int rb_linear_scan(int mode, const void* q, const void* k, const void*
     if (mode == MODE_BONUS) return extra ? launch_scan<MODE_BONUS>(a, segments, st) : (int)cudaErrorInvalidValue;
     if (mode == MODE_SSM) return extra && gate_b ? launch_scan<MODE_SSM>(a, segments, st) : (int)cudaErrorInvalidValue;
     if (mode == MODE_DELTA_HEAD) return gate_b ? launch_scan<MODE_DELTA_HEAD>(a, segments, st) : (int)cudaErrorInvalidValue;
-    if (mode == MODE_GENERAL_DELTA) return gate_b ? launch_scan<MODE_GENERAL_DELTA>(a, segments, st) : (int)cudaErrorInvalidValue;
     return (int)cudaErrorInvalidValue;
 }
 
@@ -701,17 +668,314 @@ RB_EXPORT int rb_delta_prep(const void* x, int ld, const void* taps, int taps_dt
     return rb_launch_status();
 }
 
-// ---------------------------------------------------------------- what the general delta rule needs of a token
-// Per (token, head), one warp, in float32:
+// ---------------------------------------------------------------- the general delta rule
+// Per head a [D, D] state S, read out as o = S^T q.  A token with decays g and a removal vector c per key row:
+//     S <- g * S (row i by g_i) - c (k^T S) + k v^T,  both terms of the old S;   o = S^T q
+// in float32, token by token like the scan above, so a token's result does not depend on how a prompt was cut.
+//
+// A CTA of 128 threads owns 16 value columns of one head of one segment: sixteen neighbouring lanes share a pair of
+// columns and split the key rows, lane r holding rows 64 m + 4 r .. + 3.  A token's q, k, g and -c lie in shared memory
+// as they are; a lane reads four rows of each in 16 bytes and uses them for both columns, and the arithmetic goes two rows
+// an instruction (fma.rn.f32x2).  The sum over the lanes that a token's removal waits for is a butterfly of four shuffles;
+// the decay and the new pair do not wait for it.  A token's time is the latency of one warp's instructions for it, so
+// the work is spread over warps: eight lanes a pair of columns, with half the warps, took 415 ns a token.  Chunks of tokens are double-buffered: float32 vectors come by
+// cp.async, bfloat16 ones through registers (16 bytes a load) and are converted on the way in.
+// The state lies in the request's slot as [head][column][row], rows padded to whole float4s.
+#define GD_THREADS 128
+#define GD_LANES 16            // lanes that share a pair of columns
+#define GD_COLS 16
+#define GD_TC 8                 // tokens of a chunk
+
+struct GeneralDeltaArgs {
+    const void* q; const void* k; const void* v;        // (t, head, i) at base + t * ld + head * D + i, of the activation type
+    int ld;
+    const float* decay; const float* neg_removal;       // [T, H * D]
+    float* state; long long state_stride; int s_off;
+    const int* cu_q; const int* seg_slot;
+    float* out;                                         // [T, H * D]
+    int H, D;
+};
+
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 gd_pack(float lo, float hi) {
+    f32x2 v;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(lo), "f"(hi));
+    return v;
+}
+__device__ __forceinline__ float gd_sum(f32x2 v) {      // of the two halves
+    float lo, hi;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+    return lo + hi;
+}
+__device__ __forceinline__ f32x2 gd_fma(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 gd_mul(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ f32x2 gd_add(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ void gd_cp16(void* smem, const void* gmem) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((unsigned)__cvta_generic_to_shared(smem)), "l"(gmem));
+}
+
+// M: groups of 64 key rows (D <= 64 M).  VEC: D, the row stride and every pointer allow 16-byte pieces; otherwise the
+// chunks are copied element by element.
+template <typename TA, int M, bool VEC>
+__global__ void __launch_bounds__(GD_THREADS, M <= 2 ? 5 : 3)
+general_delta_scan_kernel(const GeneralDeltaArgs a) {
+    constexpr int DP = 4 * GD_LANES * M;
+    constexpr bool BF = sizeof(TA) == 2;
+    constexpr int VECTOR = GD_TC * DP;                              // floats of one vector's chunk
+    extern __shared__ __align__(16) float gd_smem[];                // [2][q, k, g, -c][GD_TC][DP], then [2][GD_TC][GD_COLS] values
+    float* sv = gd_smem + 2 * 4 * VECTOR;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int h = blockIdx.y, j0 = blockIdx.x * GD_COLS;
+    const int r = lane % GD_LANES, jp = (warp * (32 / GD_LANES) + lane / GD_LANES) * 2;     // columns jp and jp + 1 of the CTA's
+    const int H = a.H, D = a.D, DR = (D + 3) & ~3;
+    if (D != DP) {                                                  // rows that do not exist read as zero
+        for (int i = tid; i < 2 * VECTOR; i += GD_THREADS) *reinterpret_cast<float4*>(gd_smem + 4 * i) = make_float4(0.f, 0.f, 0.f, 0.f);
+        __syncthreads();
+    }
+    pdl_wait();
+    const int seg = blockIdx.z;
+    const int t0 = a.cu_q[seg], t1 = a.cu_q[seg + 1];
+    float* Sg = a.state + (long long)a.seg_slot[seg] * a.state_stride + a.s_off + (size_t)h * D * DR;
+    const TA* q = (const TA*)a.q + (size_t)h * D;
+    const TA* k = (const TA*)a.k + (size_t)h * D;
+    const TA* v = (const TA*)a.v + (size_t)h * D + j0;
+    const size_t HD = (size_t)H * D;
+    const float* dec = a.decay + (size_t)h * D;
+    const float* rem = a.neg_removal + (size_t)h * D;
+    const int jn = min(GD_COLS, D - j0);                            // columns that exist
+
+    f32x2 S[2][2 * M];
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+            ulonglong2 x = make_ulonglong2(0ull, 0ull);
+            const int row = 4 * GD_LANES * m + 4 * r;
+            if (jp + c < jn && row < DR) x = *reinterpret_cast<const ulonglong2*>(Sg + (size_t)(j0 + jp + c) * DR + row);
+            S[c][2 * m] = x.x;
+            S[c][2 * m + 1] = x.y;
+        }
+
+    constexpr int QPER = VECTOR / 8 / GD_THREADS > 0 ? VECTOR / 8 / GD_THREADS : 1;      // 16-byte pieces of q (and k) of a thread
+    uint4 rq[BF && VEC ? QPER : 1], rk[BF && VEC ? QPER : 1];
+    const int per8 = D >> 3, per4 = D >> 2;                         // pieces of a token (VEC: D % 8 == 0)
+    constexpr int VPER = GD_TC * GD_COLS / GD_THREADS;
+    TA rv[VPER];
+    // the part of a chunk's copy that can be on its way while another chunk is worked on
+    auto fetch = [&](int tc, int buf) {
+        const int nt = min(GD_TC, t1 - tc);
+#pragma unroll
+        for (int u = 0; u < VPER; ++u) {
+            const int e = tid + u * GD_THREADS, tt = e / GD_COLS, j = e % GD_COLS;
+            if (tt < nt && j < jn) rv[u] = v[(size_t)(tc + tt) * a.ld + j];
+        }
+        if (!VEC) return;
+        float* base = gd_smem + buf * 4 * VECTOR;
+        for (int e = tid; e < nt * per4; e += GD_THREADS) {
+            const int tt = e / per4, i = (e - tt * per4) * 4;
+            const size_t t = (size_t)(tc + tt);
+            gd_cp16(base + 2 * VECTOR + tt * DP + i, dec + t * HD + i);
+            gd_cp16(base + 3 * VECTOR + tt * DP + i, rem + t * HD + i);
+            if (!BF) {
+                gd_cp16(base + tt * DP + i, q + t * a.ld + i);
+                gd_cp16(base + VECTOR + tt * DP + i, k + t * a.ld + i);
+            }
+        }
+        asm volatile("cp.async.commit_group;\n" ::);
+        if (BF) {
+#pragma unroll
+            for (int u = 0; u < QPER; ++u) {
+                const int e = tid + u * GD_THREADS;
+                if (e < nt * per8) {
+                    const int tt = e / per8, i = (e - tt * per8) * 8;
+                    rq[u] = *reinterpret_cast<const uint4*>(q + (size_t)(tc + tt) * a.ld + i);
+                    rk[u] = *reinterpret_cast<const uint4*>(k + (size_t)(tc + tt) * a.ld + i);
+                }
+            }
+        }
+    };
+    auto spread = [](float* at, const uint4& x) {                    // eight bfloat16 as eight floats
+        const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&x);
+        const float2 f0 = __bfloat1622float2(p[0]), f1 = __bfloat1622float2(p[1]);
+        const float2 f2 = __bfloat1622float2(p[2]), f3 = __bfloat1622float2(p[3]);
+        *reinterpret_cast<float4*>(at) = make_float4(f0.x, f0.y, f1.x, f1.y);
+        *reinterpret_cast<float4*>(at + 4) = make_float4(f2.x, f2.y, f3.x, f3.y);
+    };
+    // the rest of it, into the half that nobody reads
+    auto settle = [&](int tc, int buf) {
+        const int nt = min(GD_TC, t1 - tc);
+        float* base = gd_smem + buf * 4 * VECTOR;
+        if (!VEC) {
+            for (int e = tid; e < nt * D; e += GD_THREADS) {
+                const int tt = e / D, i = e - tt * D;
+                const size_t t = (size_t)(tc + tt);
+                base[tt * DP + i] = to_f32(q[t * a.ld + i]);
+                base[VECTOR + tt * DP + i] = to_f32(k[t * a.ld + i]);
+                base[2 * VECTOR + tt * DP + i] = dec[t * HD + i];
+                base[3 * VECTOR + tt * DP + i] = rem[t * HD + i];
+            }
+        } else if (BF) {
+#pragma unroll
+            for (int u = 0; u < QPER; ++u) {
+                const int e = tid + u * GD_THREADS;
+                if (e < nt * per8) {
+                    const int tt = e / per8, i = (e - tt * per8) * 8;
+                    spread(base + tt * DP + i, rq[u]);
+                    spread(base + VECTOR + tt * DP + i, rk[u]);
+                }
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < VPER; ++u) {
+            const int e = tid + u * GD_THREADS;
+            sv[buf * GD_TC * GD_COLS + e] = (e / GD_COLS < nt && e % GD_COLS < jn) ? to_f32(rv[u]) : 0.f;
+        }
+        asm volatile("cp.async.wait_group 0;\n" ::);
+        __syncthreads();
+    };
+    auto quad = [&](const float* at, ulonglong2 (&x)[M]) {
+#pragma unroll
+        for (int m = 0; m < M; ++m) x[m] = *reinterpret_cast<const ulonglong2*>(at + 4 * GD_LANES * m + 4 * r);
+    };
+
+    if (t0 < t1) { fetch(t0, 0); settle(t0, 0); }
+    int buf = 0;
+    for (int tc = t0; tc < t1; tc += GD_TC, buf ^= 1) {
+        const int nt = min(GD_TC, t1 - tc);
+        const bool more = tc + GD_TC < t1;
+        if (more) fetch(tc + GD_TC, buf ^ 1);
+        const float* base = gd_smem + buf * 4 * VECTOR;
+        ulonglong2 kk[M];
+        quad(base + VECTOR, kk);
+        auto token = [&](int tt) {
+            ulonglong2 gg[M], cc[M], qq[M];
+            quad(base + 2 * VECTOR + tt * DP, gg);
+            const float2 vv = *reinterpret_cast<const float2*>(sv + (buf * GD_TC + tt) * GD_COLS + jp);
+            const f32x2 v0 = gd_pack(vv.x, vv.x), v1 = gd_pack(vv.y, vv.y);
+            f32x2 d0[2] = {0ull, 0ull}, d1[2] = {0ull, 0ull};
+#pragma unroll
+            for (int m = 0; m < M; ++m) {
+                d0[0] = gd_fma(S[0][2 * m], kk[m].x, d0[0]);
+                d1[0] = gd_fma(S[1][2 * m], kk[m].x, d1[0]);
+                d0[1] = gd_fma(S[0][2 * m + 1], kk[m].y, d0[1]);
+                d1[1] = gd_fma(S[1][2 * m + 1], kk[m].y, d1[1]);
+            }
+            float h0 = gd_sum(gd_add(d0[0], d0[1])), h1 = gd_sum(gd_add(d1[0], d1[1]));
+            quad(base + 3 * VECTOR + tt * DP, cc);
+            quad(base + tt * DP, qq);
+            h0 += __shfl_xor_sync(0xffffffffu, h0, 1);
+            h1 += __shfl_xor_sync(0xffffffffu, h1, 1);
+#pragma unroll
+            for (int m = 0; m < M; ++m) {
+                S[0][2 * m] = gd_fma(gg[m].x, S[0][2 * m], gd_mul(kk[m].x, v0));
+                S[1][2 * m] = gd_fma(gg[m].x, S[1][2 * m], gd_mul(kk[m].x, v1));
+                S[0][2 * m + 1] = gd_fma(gg[m].y, S[0][2 * m + 1], gd_mul(kk[m].y, v0));
+                S[1][2 * m + 1] = gd_fma(gg[m].y, S[1][2 * m + 1], gd_mul(kk[m].y, v1));
+            }
+            quad(base + VECTOR + min(tt + 1, GD_TC - 1) * DP, kk);            // the next token's key
+#pragma unroll
+            for (int o = 2; o < GD_LANES; o <<= 1) {
+                h0 += __shfl_xor_sync(0xffffffffu, h0, o);
+                h1 += __shfl_xor_sync(0xffffffffu, h1, o);
+            }
+            const f32x2 hh0 = gd_pack(h0, h0), hh1 = gd_pack(h1, h1);
+            f32x2 o0[2] = {0ull, 0ull}, o1[2] = {0ull, 0ull};
+#pragma unroll
+            for (int m = 0; m < M; ++m) {
+                S[0][2 * m] = gd_fma(cc[m].x, hh0, S[0][2 * m]);
+                S[1][2 * m] = gd_fma(cc[m].x, hh1, S[1][2 * m]);
+                S[0][2 * m + 1] = gd_fma(cc[m].y, hh0, S[0][2 * m + 1]);
+                S[1][2 * m + 1] = gd_fma(cc[m].y, hh1, S[1][2 * m + 1]);
+                o0[0] = gd_fma(S[0][2 * m], qq[m].x, o0[0]);
+                o1[0] = gd_fma(S[1][2 * m], qq[m].x, o1[0]);
+                o0[1] = gd_fma(S[0][2 * m + 1], qq[m].y, o0[1]);
+                o1[1] = gd_fma(S[1][2 * m + 1], qq[m].y, o1[1]);
+            }
+            // even lanes end with the first column's sum, odd ones with the second's
+            const float u0 = gd_sum(gd_add(o0[0], o0[1])), u1 = gd_sum(gd_add(o1[0], o1[1]));
+            float o = (lane & 1) ? u1 : u0;
+            o += __shfl_xor_sync(0xffffffffu, (lane & 1) ? u0 : u1, 1);
+#pragma unroll
+            for (int x = 2; x < GD_LANES; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
+            if (r < 2 && jp + r < jn) a.out[(size_t)(tc + tt) * HD + (size_t)h * D + j0 + jp + r] = o;
+        };
+        if (nt == GD_TC) {
+#pragma unroll 4
+            for (int tt = 0; tt < GD_TC; ++tt) token(tt);
+        } else {
+#pragma unroll 1
+            for (int tt = 0; tt < nt; ++tt) token(tt);
+        }
+        if (more) settle(tc + GD_TC, buf ^ 1);
+    }
+    pdl_trigger_late();
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+            const int row = 4 * GD_LANES * m + 4 * r;
+            if (jp + c < jn && row < DR)
+                *reinterpret_cast<ulonglong2*>(Sg + (size_t)(j0 + jp + c) * DR + row) = make_ulonglong2(S[c][2 * m], S[c][2 * m + 1]);
+        }
+}
+
+template <typename TA, int M, bool VEC>
+static int launch_general_delta(const GeneralDeltaArgs& a, int segments, cudaStream_t st) {
+    constexpr int smem = (2 * 4 * GD_TC * 4 * GD_LANES * M + 2 * GD_TC * GD_COLS) * (int)sizeof(float);
+    static PerDevice configured;
+    const int rc = configured.once([](int) {
+        return cudaFuncSetAttribute(general_delta_scan_kernel<TA, M, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    });
+    if (rc != 0) return rc;
+    dim3 grid((a.D + GD_COLS - 1) / GD_COLS, a.H, segments);
+    return rb_launch_pdl(general_delta_scan_kernel<TA, M, VEC>, grid, dim3(GD_THREADS), smem, st, a);
+}
+
+template <typename TA, bool VEC>
+static int launch_general_delta_any(const GeneralDeltaArgs& a, int segments, cudaStream_t st) {
+    if (a.D <= 64) return launch_general_delta<TA, 1, VEC>(a, segments, st);
+    if (a.D <= 128) return launch_general_delta<TA, 2, VEC>(a, segments, st);
+    return launch_general_delta<TA, 4, VEC>(a, segments, st);
+}
+
+RB_EXPORT int rb_general_delta_scan(const void* q, const void* k, const void* v, int ld, int act_dtype, const float* decay,
+                                    const float* neg_removal, float* state, long long state_stride, int s_off, const int* cu_q,
+                                    const int* seg_slot, float* out, int H, int D, int segments, cudaStream_t st) {
+    if (segments <= 0) return 0;
+    if (D < 1 || D > 256 || H < 1 || state_stride % 4 || s_off % 4 || ((uintptr_t)state & 15)) return (int)cudaErrorInvalidValue;
+    GeneralDeltaArgs a;
+    a.q = q; a.k = k; a.v = v; a.ld = ld; a.decay = decay; a.neg_removal = neg_removal;
+    a.state = state; a.state_stride = state_stride; a.s_off = s_off; a.cu_q = cu_q; a.seg_slot = seg_slot;
+    a.out = out; a.H = H; a.D = D;
+    auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    const bool vec = D % 8 == 0 && ld % 8 == 0 && al(q) && al(k) && al(decay) && al(neg_removal);
+    if (act_dtype == RB_F32)
+        return vec ? launch_general_delta_any<float, true>(a, segments, st) : launch_general_delta_any<float, false>(a, segments, st);
+    return vec ? launch_general_delta_any<bf16, true>(a, segments, st) : launch_general_delta_any<bf16, false>(a, segments, st);
+}
+
+// What the general delta rule's scan needs of a token.  Per (token, head), one warp, in float32:
 //   decay[t, h, i] = exp(-scale * sigmoid(decay[t, h, i] + w0[h, i]))              (in place over the projection's output)
-//   removal[t, h, i] = sigmoid(a[t, h, i] + a_bias[h, i]) * k[t, h, i] / (sum_i k^2 + unit_eps)
-// With u = k / sqrt(sum k^2 + unit_eps) the scan's removal (rate * u)(u^T S) is removal (k^T S).  k and a are runs of
+//   neg_removal[t, h, i] = -sigmoid(a[t, h, i] + a_bias[h, i]) * k[t, h, i] / (sum_i k^2 + unit_eps)
+// With u = k / sqrt(sum k^2 + unit_eps) the removal -(rate * u)(u^T S) is neg_removal (k^T S).  k and a are runs of
 // columns of the projection rows.
 template <typename TA>
 __global__ void __launch_bounds__(128)
 general_delta_prep_kernel(const TA* __restrict__ proj, int ld, int k_off, int a_off, const void* __restrict__ a_bias,
                           const void* __restrict__ w0, int vec_dtype, float scale, float unit_eps, float* __restrict__ decay,
-                          float* __restrict__ removal, int rows, int H, int D) {
+                          float* __restrict__ neg_removal, int rows, int H, int D) {
     pdl_wait();
     const int row = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
     if (row >= rows) return;
@@ -719,7 +983,7 @@ general_delta_prep_kernel(const TA* __restrict__ proj, int ld, int k_off, int a_
     const TA* k = proj + (size_t)t * ld + k_off + (size_t)h * D;
     const TA* a = proj + (size_t)t * ld + a_off + (size_t)h * D;
     float* dc = decay + (size_t)row * D;
-    float* rm = removal + (size_t)row * D;
+    float* rm = neg_removal + (size_t)row * D;
     float kv[8], ss = 0.f;                                // up to 256 key rows
 #pragma unroll
     for (int u = 0; u < 8; ++u) {
@@ -735,21 +999,21 @@ general_delta_prep_kernel(const TA* __restrict__ proj, int ld, int k_off, int a_
         if (i >= D) break;
         const size_t e = (size_t)h * D + i;
         dc[i] = expf(-scale * sigmoid_f(dc[i] + load_as_f32(w0, vec_dtype, e)));
-        rm[i] = sigmoid_f(to_f32(a[i]) + load_as_f32(a_bias, vec_dtype, e)) * kv[u] * inv;
+        rm[i] = -sigmoid_f(to_f32(a[i]) + load_as_f32(a_bias, vec_dtype, e)) * kv[u] * inv;
     }
 }
 
 RB_EXPORT int rb_general_delta_prep(const void* proj, int ld, int k_off, int a_off, const void* a_bias, const void* w0,
-                                    int vec_dtype, float scale, float unit_eps, float* decay, float* removal, int act_dtype,
+                                    int vec_dtype, float scale, float unit_eps, float* decay, float* neg_removal, int act_dtype,
                                     int T, int H, int D, cudaStream_t st) {
     if (T <= 0) return 0;
     if (D < 1 || D > 256) return (int)cudaErrorInvalidValue;
     const int rows = T * H;
     if (act_dtype == RB_F32)
         return rb_launch_pdl(general_delta_prep_kernel<float>, dim3((rows + 3) / 4), dim3(128), 0, st, (const float*)proj, ld, k_off,
-                             a_off, a_bias, w0, vec_dtype, scale, unit_eps, decay, removal, rows, H, D);
+                             a_off, a_bias, w0, vec_dtype, scale, unit_eps, decay, neg_removal, rows, H, D);
     return rb_launch_pdl(general_delta_prep_kernel<bf16>, dim3((rows + 3) / 4), dim3(128), 0, st, (const bf16*)proj, ld, k_off,
-                         a_off, a_bias, w0, vec_dtype, scale, unit_eps, decay, removal, rows, H, D);
+                         a_off, a_bias, w0, vec_dtype, scale, unit_eps, decay, neg_removal, rows, H, D);
 }
 
 // The conv state after a step: the last K - 1 inputs of each channel, oldest first.  A segment shorter than K - 1

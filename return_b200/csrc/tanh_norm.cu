@@ -90,15 +90,20 @@ tanh_joint_kernel(const JointArgs a) {
     pdl_wait();
     if (!live) return;
 
-    auto stream_at = [&](int t, float (&x)[N]) {
+    auto load = [&](int t, float (&x)[N], float (&y)[N]) {
         const size_t at = (size_t)t * a.H + c;
         ld_f32<N>(a.x_in + at, x);
-        if (has_y) {
-            float y[N];
-            ld_any<N>(a.y, a.y_f32, at, y);
+        if (has_y) ld_any<N>(a.y, a.y_f32, at, y);
+    };
+    auto add = [&](float (&x)[N], const float (&y)[N]) {
+        if (!has_y) return;
 #pragma unroll
-            for (int i = 0; i < N; ++i) x[i] += post ? fmaf(squash<FAST>(pa * y[i]), pw[i], pb[i]) : y[i];
-        }
+        for (int i = 0; i < N; ++i) x[i] += post ? fmaf(squash<FAST>(pa * y[i]), pw[i], pb[i]) : y[i];
+    };
+    auto stream_at = [&](int t, float (&x)[N]) {
+        float y[N];
+        load(t, x, y);
+        add(x, y);
     };
     auto normed = [&](const float (&x)[N], float (&h)[N]) {
 #pragma unroll
@@ -106,12 +111,16 @@ tanh_joint_kernel(const JointArgs a) {
     };
 
     const int r0 = blockIdx.x * a.run, r1 = min(a.T, r0 + a.run);
-    float prev[N];
+    float prev[N], x_next[N], y_next[N];
     bool have_prev = false;
+    if (r0 < r1) load(a.rows ? a.rows[r0] : r0, x_next, y_next);
     for (int r = r0; r < r1; ++r) {
         const int t = a.rows ? a.rows[r] : r;
-        float x[N], h[N];
-        stream_at(t, x);
+        float x[N], y[N], h[N];
+#pragma unroll
+        for (int i = 0; i < N; ++i) { x[i] = x_next[i]; y[i] = y_next[i]; }
+        if (r + 1 < r1) load(a.rows ? a.rows[r + 1] : r + 1, x_next, y_next);      // on its way while this row is worked on
+        add(x, y);
         if (a.x_out) st_f32<N>(a.x_out + (size_t)t * a.H + c, x);
         if (!next) continue;
         normed(x, h);

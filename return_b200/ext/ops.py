@@ -127,7 +127,8 @@ def build_all():
     paths = [build.library_path("return_core", _CORE_SOURCES, {"RB_PDL_MODE": PDL_MODE})]
     paths.append(build.library_path("return_tc5", _TC5_SOURCES, _tc5_defines()))
     paths.append(build.library_path("return_recurrent", _RECURRENT_SOURCES, {"RB_PDL_MODE": PDL_MODE}))
-    paths.append(build.library_path("return_attn_conv", _ATTN_CONV_SOURCES, {"RB_PDL_MODE": PDL_MODE}))
+    for key in PREBUILT_CONV:
+        paths.append(build.library_path("return_attn_conv_h%d_k%d" % key, _ATTN_CONV_SOURCES, _attn_conv_defines(*key)))
     paths.append(build.library_path("return_tanh_norm", _TANH_NORM_SOURCES, {"RB_PDL_MODE": PDL_MODE}))
     paths.append(build.library_path("return_latent", _LATENT_SOURCES, {"RB_PDL_MODE": PDL_MODE}))
     paths.append(build.library_path("return_moe", _MOE_SOURCES, {"RB_PDL_MODE": PDL_MODE}))
@@ -971,42 +972,50 @@ def attention_gate(o, gate, g_off: int, per_head: bool, num_heads: int, vdim: in
 
 # ------------------------------------------------------------------------------- attention behind a convolution
 
-_attn_conv = None
+_attn_conv_libs = {}
 _ATTN_CONV_SOURCES = ["attention_conv.cu"]
+CONV_REGISTER_TAPS = 4           # filters of up to so many taps are compiled for their length; longer ones share a kernel
+PREBUILT_CONV = ((64, 4), (128, 4), (64, 3), (64, 2), (64, 1), (64, 0))      # compiled ahead of time by build_all()
 
 
-def attention_conv_lib() -> ctypes.CDLL:
-    """The kernel between the projections and the attention of heads that pass a short convolution (csrc/attention_conv.cu);
-    compiled when a model that has such an attention is first run."""
-    global _attn_conv
-    if _attn_conv is None:
-        lib = build.load("return_attn_conv", _ATTN_CONV_SOURCES, {"RB_PDL_MODE": PDL_MODE})
+def _attn_conv_defines(lanes: int, taps: int):
+    return {"HEAD_LANES": lanes, "CONV_TAPS": taps, "RB_PDL_MODE": PDL_MODE}
+
+
+def attention_conv_lib(head_dim: int, taps: int) -> ctypes.CDLL:
+    """The kernel between the projections and the attention of heads that pass a short convolution (csrc/attention_conv.cu),
+    compiled on first use for a filter length and for heads of up to 64, 128 or 256 elements."""
+    key = (64 if head_dim <= 64 else 128 if head_dim <= 128 else 256, taps if taps <= CONV_REGISTER_TAPS else 0)
+    lib = _attn_conv_libs.get(key)
+    if lib is None:
+        lib = build.load("return_attn_conv_h%d_k%d" % key, _ATTN_CONV_SOURCES, _attn_conv_defines(*key))
         P, I, F, L = c_void_p, c_int, c_float, ctypes.c_longlong
-        lib.rb_attn_conv_prep.argtypes = [P, I, P, I, I, P, L, I, P, P, P, P, P, I, I, P, P, P, I, I, I, I, I, I, I, I, I, I, F, F, I, P]
+        lib.rb_attn_conv_prep.argtypes = [P, I, P, I, P, L, I, P, P, P, P, P, I, I, P, P, P, I, I, I, I, I, I, I, I, I, I, F, F, I, P]
         lib.rb_attn_conv_prep.restype = c_int
-        _attn_conv = lib
-    return _attn_conv
+        _attn_conv_libs[key] = lib
+    return lib
 
 
 def attention_conv_prepare(proj, taps, kept, kept_off: int, batch, kv, q_out, num_heads: int, num_kv_heads: int, dim: int,
                            vdim: int, head_dim: int, norm_eps: Optional[float] = None, temperature=None, own_kv: bool = True,
                            write_kv: bool = True) -> None:
     """From projection rows [q | k | v] (only q without ``own_kv``) to what the paged attention reads: every channel through
-    its causal filter ``taps`` [channels, K] (last column: the token itself), q and k heads over their root mean square
+    its causal filter ``taps`` (float32 [K, channels], last row: the token itself), q and k heads over their root mean square
     (``norm_eps``; None: not normed), q heads times 1 + coef ln(floor((p + 1) / every) + 1) (``temperature`` = (coef, every)),
     q heads padded to ``head_dim`` into q_out, k and v heads into their pages.  ``kept`` (float32 [slots, n]): a request's
     last K - 1 rows of inputs from column kept_off, read and renewed."""
     T = proj.shape[0]
-    K = taps.shape[1]
+    K = taps.shape[0]
     channels = num_heads * dim + (num_kv_heads * (dim + vdim) if own_kv else 0)
-    assert proj.stride(1) == 1 and proj.shape[1] >= channels and taps.shape[0] == channels and taps.is_contiguous()
+    assert proj.stride(1) == 1 and proj.shape[1] >= channels and taps.shape[1] == channels and taps.is_contiguous()
+    assert taps.dtype == torch.float32
     assert q_out.is_contiguous() and q_out.dtype == proj.dtype and q_out.shape == (T, num_heads * head_dim)
     assert kv.k.dtype == kv.v.dtype == proj.dtype and kv.k.shape[-1] == head_dim
     if K > 1:
         assert kept.dtype == torch.float32 and kept.is_contiguous() and kept.shape[1] >= kept_off + (K - 1) * channels
     coef, every = temperature if temperature is not None else (0.0, 0)
-    _check(attention_conv_lib().rb_attn_conv_prep(
-        _ptr(proj), proj.stride(0), _ptr(taps), dtype_code(taps.dtype), K, _ptr(kept) if K > 1 else None,
+    _check(attention_conv_lib(head_dim, K).rb_attn_conv_prep(
+        _ptr(proj), proj.stride(0), _ptr(taps), K, _ptr(kept) if K > 1 else None,
         kept.stride(0) if K > 1 else 0, kept_off, _ptr(batch.pos), _ptr(batch.tok_seg), _ptr(batch.cu_q), _ptr(batch.seg_slot),
         _ptr(kv.block_table), kv.block_table.stride(0), kv.page_size, _ptr(kv.k), _ptr(kv.v), _ptr(q_out),
         dtype_code(proj.dtype), T, num_heads, num_kv_heads, dim, vdim, head_dim, 1 if own_kv else 0, 1 if write_kv else 0,
@@ -1069,7 +1078,7 @@ def tanh_joint(x_in, x_out, y, post, nxt, out, shift=None, batch=None, rows=None
 
 _recurrent = None
 _RECURRENT_SOURCES = ["recurrent.cu"]
-SCAN_DECAY, SCAN_MEMORY, SCAN_DELTA, SCAN_BONUS, SCAN_SSM, SCAN_DELTA_HEAD, SCAN_GENERAL_DELTA = 0, 1, 2, 3, 4, 5, 6
+SCAN_DECAY, SCAN_MEMORY, SCAN_DELTA, SCAN_BONUS, SCAN_SSM, SCAN_DELTA_HEAD = 0, 1, 2, 3, 4, 5
 SCAN_MAX_KEY_DIM = 256
 
 
@@ -1100,6 +1109,8 @@ def recurrent_lib() -> ctypes.CDLL:
         lib.rb_gated_conv.restype = lib.rb_gated_recurrence.restype = lib.rb_gated_pieces_combine.restype = c_int
         lib.rb_general_delta_prep.argtypes = [P, I, I, I, P, P, I, F, F, P, P, I, I, I, I, P]
         lib.rb_general_delta_prep.restype = c_int
+        lib.rb_general_delta_scan.argtypes = [P, P, P, I, I, P, P, P, L, I, P, P, P, I, I, I, P]
+        lib.rb_general_delta_scan.restype = c_int
         lib.rb_conv_state_update.argtypes = [P, I, I, P, L, I, P, P, I, I, I, P]
         lib.rb_head_norm_gate.argtypes = [P, P, I, P, I, I, I, F, P, I, I, I, I, P]
         lib.rb_add_dual_norm.argtypes = [P, P, I, F, P, I, F, P, P, P, I, F, F, P, P, I, I, I, P]
@@ -1129,8 +1140,7 @@ def linear_scan(mode: int, q, k, v, gate_a, gate_b, state, offsets, batch, out, 
     matrix, the normaliser and the running maximum start inside a row (the last two for ``SCAN_MEMORY`` only).
     ``gate_a`` / ``gate_b`` by mode: SCAN_DECAY: [heads] decays / None; SCAN_MEMORY: [T, 2 heads] gate
     pre-activations (input, forget) / [2 heads] biases; SCAN_DELTA: [T, heads, dim] row decays / [T, heads] beta;
-    SCAN_DELTA_HEAD: [T, heads] decays / [T, heads] beta; SCAN_GENERAL_DELTA (S <- g * S - c (k^T S) + k v^T, o = S^T q):
-    [T, heads, dim] row decays / [T, heads, dim] removal vectors c;
+    SCAN_DELTA_HEAD: [T, heads] decays / [T, heads] beta;
     SCAN_BONUS (o = (S + diag(u) k v^T)^T q, then S <- g * S + k v^T): [T, heads, dim] row decays / None, ``extra`` = u
     [heads, dim]; SCAN_SSM (S <- a S + dt k v^T, o = S^T q + d v): [T, heads] decays / [T, heads] steps, ``extra`` = d
     [heads].
@@ -1235,18 +1245,34 @@ def delta_prep(x, taps, state, conv_off: int, batch, q32, k32, v32, a, A_log, dt
         q_scale, 1 if head_decay else 0, _stream()), "delta_prep")
 
 
-def general_delta_prep(proj, k_off: int, a_off: int, a_bias, w0, scale: float, unit_eps: float, decay, removal, heads: int,
+def general_delta_scan(q, k, v, decay, neg_removal, state, s_off: int, batch, out, heads: int, dim: int) -> None:
+    """S <- g * S - c (k^T S) + k v^T (both terms of the old S), o = S^T q per head over every segment of the step, token by
+    token.  q, k, v: column views of one projection buffer (from where each begins); decay g and removal c: float32
+    [T, heads * dim], c as its negative; ``state``: float32 [slots, n], S from column s_off of a segment's row as
+    [head][column][row] with the rows padded to a multiple of four; out: float32 [T, heads * dim]."""
+    n = heads * dim
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous() and dim <= SCAN_MAX_KEY_DIM
+    assert q.dtype == k.dtype == v.dtype and q.stride(0) == k.stride(0) == v.stride(0) and q.stride(1) == k.stride(1) == v.stride(1) == 1
+    for t in (decay, neg_removal, out):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.shape == (q.shape[0], n)
+    _check(recurrent_lib().rb_general_delta_scan(_ptr(q), _ptr(k), _ptr(v), q.stride(0), dtype_code(q.dtype), _ptr(decay),
+                                                 _ptr(neg_removal), _ptr(state), state.stride(0), s_off, _ptr(batch.cu_q),
+                                                 _ptr(batch.seg_slot), _ptr(out), heads, dim, batch.num_segments, _stream()),
+           "general_delta_scan")
+
+
+def general_delta_prep(proj, k_off: int, a_off: int, a_bias, w0, scale: float, unit_eps: float, decay, neg_removal, heads: int,
                        dim: int) -> None:
     """What the general delta rule's scan needs per token, head and key row: decay = exp(-scale * sigmoid(decay + w0)) in place
-    (float32 [T, heads * dim]) and removal = sigmoid(a + a_bias) * k / (sum of the head's k^2 + unit_eps), with k and a the
-    columns of ``proj`` from k_off and a_off."""
+    (float32 [T, heads * dim]) and neg_removal = -sigmoid(a + a_bias) * k / (sum of the head's k^2 + unit_eps), with k and a
+    the columns of ``proj`` from k_off and a_off."""
     T = proj.shape[0]
     n = heads * dim
     assert proj.stride(1) == 1 and a_bias.dtype == w0.dtype and a_bias.numel() == w0.numel() == n
-    for t in (decay, removal):
+    for t in (decay, neg_removal):
         assert t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n)
     _check(recurrent_lib().rb_general_delta_prep(_ptr(proj), proj.stride(0), k_off, a_off, _ptr(a_bias), _ptr(w0),
-                                                 dtype_code(w0.dtype), scale, unit_eps, _ptr(decay), _ptr(removal),
+                                                 dtype_code(w0.dtype), scale, unit_eps, _ptr(decay), _ptr(neg_removal),
                                                  dtype_code(proj.dtype), T, heads, dim, _stream()), "general_delta_prep")
 
 

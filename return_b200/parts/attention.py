@@ -225,8 +225,8 @@ class GatedAttention(Mixer):
         if s.fixed_sink is not None:
             self._sink = torch.full((s.num_heads,), float(s.fixed_sink), dtype=torch.float32, device=self.env.device)
         if self.by_head:                    # without a convolution: a filter of the token itself
-            self._taps = self.p_conv.contiguous() if s.conv_taps else torch.ones(
-                (self.nq + self.nk + self.nv, 1), dtype=torch.float32, device=self.env.device)
+            self._taps = self.p_conv.float().t().contiguous() if s.conv_taps else torch.ones(
+                (1, self.nq + self.nk + self.nv), dtype=torch.float32, device=self.env.device)
         if s.distance_bias is not None:     # the table by distance instead of by row, [heads, distances]
             rows = torch.tensor(distance_rows(*s.distance_bias), dtype=torch.int64, device=self.p_rel.device)
             self._bias = self.p_rel.float()[rows].t().contiguous()

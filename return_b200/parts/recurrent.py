@@ -454,8 +454,8 @@ class GatedDelta(_StateMixer):
 @MIXERS.register("general_delta")
 class GeneralDelta(_StateMixer):
     """``GeneralDeltaSpec``: one product gives [r | k | v | gate | rate | low rank]; the decay's second product follows; a
-    small kernel makes decays and removal vectors; the scan, per-head norm, gate and output projection are those of the
-    other state mixers.  The request's state row holds S."""
+    small kernel makes decays and removal vectors; a scan kernel of its own walks the segments; per-head norm, gate and
+    output projection are those of the other state mixers.  The request's state row holds S, column by column."""
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
@@ -465,7 +465,7 @@ class GeneralDelta(_StateMixer):
             raise ValueError(f"key_dim={self.D}: the scan kernel holds up to {ops.SCAN_MAX_KEY_DIM} key rows a head")
         if s.decay_rank <= 0:
             raise ValueError("decay_rank must be positive")
-        self.s_floats = self.H * _pad8(self.D) * self.V
+        self.s_floats = self.H * self.V * ((self.D + 3) // 4 * 4)           # [head][column][row], rows in whole float4s
 
     def params(self):
         s = self.spec
@@ -497,8 +497,7 @@ class GeneralDelta(_StateMixer):
         removal = ctx.buffer("general_delta.removal", (T, HD), torch.float32, dev)
         ops.general_delta_prep(proj, HD, 4 * HD, self._rate_bias, self._w0, s.decay_scale, s.unit_eps, decay, removal, self.H, self.D)
         o = ctx.buffer("general_delta.o", (T, HD), torch.float32, dev)
-        ops.linear_scan(ops.SCAN_GENERAL_DELTA, proj, proj[:, HD:], proj[:, 2 * HD:], decay, removal, ctx.state, (0, 0, 0), b, o,
-                        self.H, self.H, self.D, self.V)
+        ops.general_delta_scan(proj, proj[:, HD:], proj[:, 2 * HD:], decay, removal, ctx.state, 0, b, o, self.H, self.D)
         mixed = ctx.buffer("general_delta.mixed", (T, HD), dt, dev)
         ops.head_norm_gate(o, proj[:, 3 * HD:], self.p_norm, 2, 1, s.eps, mixed, self.H, self.V)
         return self._project_out(mixed, ctx)
