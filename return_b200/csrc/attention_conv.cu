@@ -280,8 +280,11 @@ RB_EXPORT int rb_attn_conv_prep(const void* proj, int ld, const float* taps, int
                      al(kpool) && al(vpool);
     constexpr int LPH = HEAD_LANES / 8;                    // lanes of a head when each holds eight neighbouring elements
     const int head_ctas = vec ? (heads + 128 / LPH - 1) / (128 / LPH) : (heads + 3) / 4;
-    a.run = 1;
-    while (a.run < 16 && (long long)(T / (2 * a.run)) * head_ctas >= 148 * 4) a.run *= 2;
+    // runs just long enough that one wave of CTAs (four an SM) covers the step; very long steps take several waves
+    const long long slots = 4LL * rb_num_sms();
+    a.run = slots > 0 ? (int)(((long long)T * head_ctas + slots - 1) / slots) : 16;
+    if (a.run > 2) a.run = (a.run + AHEAD - 1) / AHEAD * AHEAD;
+    if (a.run > 64) a.run = 64;
     dim3 grid((T + a.run - 1) / a.run, head_ctas);
     if (vec) return rb_launch_pdl(attn_conv_prep_kernel<bf16, 8, 1, LPH>, grid, dim3(128), 0, st, a);
     // any sizes: single elements, as many groups of 32 as the head has
