@@ -9,12 +9,13 @@ for other architectures, ``LinearStateCache`` slots of fixed size per resident s
 (rollout/cache.py:340-472).  What is different here:
 
 * Layers are put into **groups** by what they need.  A group of full-attention layers keeps
-  every key; a group of sliding-window layers keeps a window of them.  Each group has pages of
+  every key; a group of sliding-window layers keeps a window of them, and the sequence's first keys
+  beside it if its layers keep those in sight.  Each group has pages of
   its own (its own pool, free list and block tables), because a window group gives pages back
   while a request is still running and a full group does not.
 * Only the last page of a request is partly filled, so a block table is a list of page ids
-  indexed by ``position // page_size``; ``-1`` marks a block that the window has passed and
-  whose page went back to the pool.
+  indexed by ``position // page_size``; ``-1`` marks a block that the window has passed (and that
+  holds no kept first key) and whose page went back to the pool.
 * Every request holds one **slot** (0 .. max_requests-1) for its fixed-size state and as its
   row in device-side tables, whether or not the architecture has such state.
 """
@@ -30,11 +31,18 @@ class KVCapacityError(MemoryError):
 
 @dataclass(frozen=True)
 class GroupSpec:
-    """What one group of cache layers needs.  ``window`` None: all keys; else the last ``window`` keys."""
+    """What one group of cache layers needs.  ``window`` None: all keys; else the last ``window`` keys and the sequence's first
+    ``keep_first`` ones."""
     name: str
     page_size: int
     num_pages: int
     window: Optional[int] = None
+    keep_first: int = 0
+
+    @property
+    def kept_blocks(self) -> int:
+        """Blocks from the start of a sequence that never go back while the request runs."""
+        return (self.keep_first + self.page_size - 1) // self.page_size if self.window is not None else 0
 
 
 class PagePool:
@@ -146,10 +154,15 @@ class CacheManager:
 
     # ------------------------------------------------------------------ pages
     def _first_needed_block(self, g: GroupSpec, length: int) -> int:
-        """Blocks below this index hold only keys that no query at position >= length can see."""
+        """Blocks below this index, but for a group's kept first ones, hold only keys that no query at position >= length
+        can see."""
         if g.window is None:
             return 0
         return max(0, length - g.window + 1) // g.page_size
+
+    def _passed_blocks(self, g: GroupSpec, blocks: Sequence[int], length: int) -> List[int]:
+        """Indices of the blocks whose pages can go back to the pool."""
+        return [b for b in range(g.kept_blocks, min(self._first_needed_block(g, length), len(blocks))) if blocks[b] >= 0]
 
     def pages_needed(self, rid, n_tokens: int) -> List[int]:
         """Per group: pages that ``append(rid, n_tokens)`` would take beyond those it gives back."""
@@ -158,9 +171,7 @@ class CacheManager:
         for g, blocks in zip(self.groups, st.blocks):
             end_blocks = (st.length + n_tokens + g.page_size - 1) // g.page_size
             new = max(0, end_blocks - len(blocks))
-            first = self._first_needed_block(g, st.length)
-            released = sum(1 for b in range(min(first, len(blocks))) if blocks[b] >= 0)
-            out.append(new - released)
+            out.append(new - len(self._passed_blocks(g, blocks, st.length)))
         return out
 
     def fits(self, rid, n_tokens: int) -> bool:
@@ -189,8 +200,7 @@ class CacheManager:
                      if need > pool.num_free]
             raise KVCapacityError(f"request {rid!r}: pages (group, needed, free) {short}")
         for g, pool, blocks in zip(self.groups, self.pools, st.blocks):
-            first = self._first_needed_block(g, st.length)
-            gone = [b for b in range(min(first, len(blocks))) if blocks[b] >= 0]
+            gone = self._passed_blocks(g, blocks, st.length)
             if gone:
                 pool.give_back([blocks[b] for b in gone])
                 for b in gone:

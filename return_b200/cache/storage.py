@@ -1,7 +1,7 @@
 """The device side of the cache: pools of pages per group of layers, and state slots.
 
 Layers (runs of the schedule that own a cache) are grouped by what their mixers ask for:
-paged keys and values with the same window, number of KV heads and head size share a group,
+paged keys and values with the same window (and kept first keys), number of KV heads and head size share a group,
 hence a page pool, a free list and block tables (``return_b200/cache/manager.py``).  The pool of
 a group is one tensor ``[layers, 2, num_pages, Hkv, page_size, D]`` in the activation dtype
 (index 0 of the second axis: keys, 1: values), so one page id addresses a slab in every layer of
@@ -29,7 +29,7 @@ class CacheStorage:
         """``num_pages``: pages of a group that keeps every key (the pool's capacity in tokens / page size).
         A group that keeps a window gets only what ``max_reside`` requests can hold of it at a time: the
         window plus the longest run of tokens one step may append (``longest_append``; None: unknown, the
-        group then gets ``num_pages`` too), in pages, plus one for the ragged ends.  ``kept``: per run of the schedule,
+        group then gets ``num_pages`` too), in pages, plus one for the ragged ends, plus those of the kept first keys.  ``kept``: per run of the schedule,
         what it keeps per request for itself, whichever cache it owns or reads (``LayerContext.kept``)."""
         self.env = env
         self.page_size = page_size
@@ -53,19 +53,20 @@ class CacheStorage:
             elif isinstance(need, (KVCacheNeed, LatentCacheNeed)):
                 latent = isinstance(need, LatentCacheNeed)
                 # a latent is one vector a token: stored as "0 heads" of its width, one tensor instead of keys and values
-                sig = (need.window, 0, need.width) if latent else (need.window, need.num_kv_heads, need.head_dim)
+                keep = 0 if latent or need.window is None else need.keep_first
+                sig = (need.window, keep) + ((0, need.width) if latent else (need.num_kv_heads, need.head_dim))
                 if sig not in signature_to_group:
                     signature_to_group[sig] = len(self.group_specs)
-                    name = "full" if need.window is None else f"window{need.window}"
+                    name = "full" if need.window is None else f"window{need.window}" + (f"_first{keep}" if keep else "")
                     pages = num_pages
                     if need.window is not None and longest_append is not None:
-                        per_request = (need.window + longest_append + page_size - 1) // page_size + 1
+                        per_request = (need.window + longest_append + page_size - 1) // page_size + 1 + (keep + page_size - 1) // page_size
                         pages = max(1, min(num_pages, max_reside * per_request))
                     self.group_specs.append(GroupSpec(f"{name}_latent{need.width}" if latent else
                                                       f"{name}_h{need.num_kv_heads}_d{need.head_dim}",
-                                                      page_size, pages, need.window))
+                                                      page_size, pages, need.window, keep))
                     self._group_layers.append(0)
-                    self._group_shape.append(sig[1:])
+                    self._group_shape.append(sig[2:])
                 g = signature_to_group[sig]
                 self.entry_place[key] = (g, self._group_layers[g])
                 self._group_layers[g] += 1

@@ -111,6 +111,12 @@ def _register_builtin() -> None:
         name="Losorax", model_type="losorax", config_cls=LosoraxConfig,
         decoder_spec=losorax.decoder_spec, weight_sources=losorax.weight_sources,
         ignorable_tensors=losorax.ignorable_tensors, checkpoint_shapes=losorax.checkpoint_shapes))
+    from ..models import sizudra
+    from .sizudra_config import SizudraConfig
+    register_architecture(Architecture(
+        name="Sizudra", model_type="sizudra", config_cls=SizudraConfig,
+        decoder_spec=sizudra.decoder_spec, weight_sources=sizudra.weight_sources,
+        ignorable_tensors=sizudra.ignorable_tensors, checkpoint_shapes=sizudra.checkpoint_shapes))
 
 
 _register_builtin()

@@ -17,7 +17,9 @@
 // `chunk` positions (instead of a window), scores capped softly (cap * tanh(s / cap)), a penalty per head that
 // grows with the distance, slopes[h] * (i - j), taken off before the softmax, and a bias per head and distance,
 // bias[h, min(i - j, bias_n - 1)], added to the score: a table in global memory that only key tiles within its reach
-// look up; behind it the last entry is a constant.
+// look up; behind it the last entry is a constant.  With a window they can also keep the first `keep` positions visible for
+// every later query: the key tiles are then walked in two runs, the tiles of the kept positions that lie before the window's
+// first tile, then the window's.
 //
 // K and V of one layer: [num_pages, Hkv, P, D] bfloat16.  Shared-memory tiles are [rows][D] with
 // the 16-byte chunks of a row XOR-swizzled by the row index, which keeps ldmatrix conflict-free.
@@ -104,6 +106,7 @@ struct ScoreMod {
     int chunk;                 // 0: none
     const float* bias;         // [Hq, bias_n] or null
     int bias_n;
+    int keep;                  // with a window: the first `keep` positions stay visible (0: none)
 };
 // `brow`: the head's row of the bias table for a distance that may lie within it, or null: then `blast` (its last entry,
 // or zero without a table) is added.
@@ -155,17 +158,17 @@ __device__ __forceinline__ StagedTable stage_table(int* smem_bt, const int* bt_r
 // Copies ROWS keys starting at absolute position j0 (rows of D elements) of one kv head into a
 // swizzled tile, with NTHREADS threads: a group of NTHREADS / ROWS threads owns a row, looks its
 // page up once, and its threads take neighbouring 16-byte chunks so that each 32-byte sector is
-// asked for once.  A key outside [lo, hi] (or on a page that was given back) is zero-filled and
-// never read.
+// asked for once.  A key outside [lo, hi] and not below keep (or on a page that was given back) is zero-filled
+// and never read.
 template <int ROWS, int NTHREADS>
 __device__ __forceinline__ void load_kv_rows(bf16* tile, const bf16* pool, const StagedTable& bt, const Paging& pg,
-                                             int Hkv, int kvh, int j0, int lo, int hi, int tid) {
+                                             int Hkv, int kvh, int j0, int lo, int hi, int tid, int keep = 0) {
     constexpr int TPR = NTHREADS / ROWS;          // threads per row
     constexpr int CPT = CHUNKS / TPR;             // chunks per thread
     static_assert(NTHREADS % ROWS == 0 && CHUNKS % TPR == 0, "rows and chunks must divide evenly");
     const int r = tid / TPR, sub = tid - r * TPR;
     const int j = j0 + r;
-    bool pred = j >= lo && j <= hi;
+    bool pred = (j >= lo || j < keep) && j <= hi;
     const bf16* src = pool;
     if (pred) {
         const int page = bt.page(pg.block(j));
@@ -208,7 +211,11 @@ attn_prefill_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__
     const int p_last = p0 + m_rows - 1;
     const int chunk = MOD ? sm.chunk : 0;
     const int lo_min = window > 0 ? max(0, p0 - window + 1) : chunk > 0 ? (p0 / chunk) * chunk : 0;
-    const int jt_begin = lo_min / PF_N, jt_end = p_last / PF_N;
+    const int jt_first = lo_min / PF_N, jt_end = p_last / PF_N;
+    const int keep = MOD && window > 0 ? sm.keep : 0;
+    const int n_keep = min((keep + PF_N - 1) / PF_N, jt_first);              // tiles of kept positions before the window's first
+    const int n_tiles = n_keep + jt_end - jt_first + 1;
+    auto tile_of = [&](int i) { return i < n_keep ? i : jt_first + i - n_keep; };
     const Paging pg(page_size);
     const StagedTable bt = stage_table(sBT, block_table + (size_t)seg * bt_stride, pg.block(lo_min), pg.block(p_last), tid, 128);
     __syncthreads();
@@ -219,8 +226,8 @@ attn_prefill_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__
         const bf16* src = pred ? q + (size_t)(q_begin + row0 + r) * ld + (size_t)h * D + ch * 8 : q;
         cp_async16(sQ + soff(r, ch), src, pred);
     }
-    load_kv_rows<PF_N, 128>(sK, kpool, bt, pg, Hkv, kvh, jt_begin * PF_N, lo_min, p_last, tid);
-    load_kv_rows<PF_N, 128>(sV, vpool, bt, pg, Hkv, kvh, jt_begin * PF_N, lo_min, p_last, tid);
+    load_kv_rows<PF_N, 128>(sK, kpool, bt, pg, Hkv, kvh, tile_of(0) * PF_N, lo_min, p_last, tid, keep);
+    load_kv_rows<PF_N, 128>(sV, vpool, bt, pg, Hkv, kvh, tile_of(0) * PF_N, lo_min, p_last, tid, keep);
     cp_async_commit();
 
     unsigned qf[KSTEPS][4];
@@ -237,18 +244,18 @@ attn_prefill_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__
     const float* bias_row = (MOD && sm.bias) ? sm.bias + (size_t)h * sm.bias_n : nullptr;
     const float bias_last = (MOD && sm.bias) ? bias_row[sm.bias_n - 1] : 0.f;
 
-    for (int jt = jt_begin; jt <= jt_end; ++jt) {
-        const int stage = (jt - jt_begin) & 1;
-        if (jt < jt_end) {
-            load_kv_rows<PF_N, 128>(sK + (stage ^ 1) * PF_N * D, kpool, bt, pg, Hkv, kvh, (jt + 1) * PF_N, lo_min, p_last, tid);
-            load_kv_rows<PF_N, 128>(sV + (stage ^ 1) * PF_N * D, vpool, bt, pg, Hkv, kvh, (jt + 1) * PF_N, lo_min, p_last, tid);
+    for (int it = 0; it < n_tiles; ++it) {
+        const int stage = it & 1, jt = tile_of(it);
+        if (it + 1 < n_tiles) {
+            load_kv_rows<PF_N, 128>(sK + (stage ^ 1) * PF_N * D, kpool, bt, pg, Hkv, kvh, tile_of(it + 1) * PF_N, lo_min, p_last, tid, keep);
+            load_kv_rows<PF_N, 128>(sV + (stage ^ 1) * PF_N * D, vpool, bt, pg, Hkv, kvh, tile_of(it + 1) * PF_N, lo_min, p_last, tid, keep);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
             cp_async_wait<0>();
         }
         __syncthreads();
-        if (jt == jt_begin) {
+        if (it == 0) {
 #pragma unroll
             for (int kk = 0; kk < KSTEPS; ++kk)
                 ldsm_x4(qf[kk], sQ + soff(wrow + (lane & 7) + ((lane >> 3) & 1) * 8, 2 * kk + (lane >> 4)));
@@ -256,7 +263,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__
         const int j_base = jt * PF_N;
         // a tile that starts above the warp's last row, or ends below its first row's window, adds nothing
         const bool skip = !warp_active || j_base > p0 + wrow + 15 ||
-                          (window > 0 && j_base + PF_N - 1 <= p0 + wrow - window) ||
+                          (window > 0 && j_base + PF_N - 1 <= p0 + wrow - window && (!MOD || j_base >= keep)) ||
                           (chunk > 0 && j_base + PF_N - 1 < lo_warp);
         if (!skip) {
             const bf16* tK = sK + stage * PF_N * D;
@@ -283,7 +290,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__
                 for (int e = 0; e < 4; ++e) {
                     const int j = j_base + nt * 8 + 2 * t4 + (e & 1);
                     const int pr = (e & 2) ? pos_r1 : pos_r0;
-                    const bool vis = j <= pr && (window <= 0 || j > pr - window) && (!MOD || j >= ((e & 2) ? lo_r1 : lo_r0));
+                    const bool vis = j <= pr && (window <= 0 || j > pr - window || (MOD && j < keep)) && (!MOD || j >= ((e & 2) ? lo_r1 : lo_r0));
                     const float v = !vis ? -INFINITY : MOD ? mod_score(s[nt][e], sm, slope, pr - j, brow, bias_last) : s[nt][e] * scale_log2;
                     s[nt][e] = v;
                     if (e & 2) mx1 = fmaxf(mx1, v); else mx0 = fmaxf(mx0, v);
@@ -371,6 +378,11 @@ struct FusedRope {
     bf16* kpool;               // the pools again, to write to
     bf16* vpool;
     int write_kv;
+    int norm_n;                // elements of a head that the norm's mean runs over (heads may be padded with zeros to D)
+    const bf16* v_first;       // the new token's value is blended with an earlier layer's before it is cached (rope_cache.cu)
+    int v_first_ld, v_first_head_stride, v_first_n;
+    const void* v_share;
+    int v_share_dtype;
 };
 
 __device__ __forceinline__ float2 ld_pair(const bf16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
@@ -379,7 +391,7 @@ __device__ __forceinline__ void st_pair(bf16* p, float2 v) { *reinterpret_cast<_
 // One warp norms and rotates one head x[0..D) at position p; dst(i) is where elements i, i + 1 go.
 template <typename DstFn>
 __device__ __forceinline__ void warp_norm_rope(const bf16* __restrict__ x, const void* __restrict__ w, int w_dtype,
-                                               float eps, float offset, const float* __restrict__ cos_t,
+                                               float eps, float offset, int norm_n, const float* __restrict__ cos_t,
                                                const float* __restrict__ sin_t, int rot_dim, int p, int lane, DstFn dst) {
     const int half = rot_dim >> 1;
     const float* cs = cos_t + (size_t)p * half;
@@ -413,7 +425,7 @@ __device__ __forceinline__ void warp_norm_rope(const bf16* __restrict__ x, const
     float rstd = 1.f;
     if (w) {
         ss = warp_sum(ss);
-        rstd = 1.0f / sqrtf(ss / (float)D + eps);
+        rstd = 1.0f / sqrtf(ss / (float)norm_n + eps);
     }
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -469,13 +481,20 @@ attn_decode_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__ 
     const int lo = window > 0 ? max(0, kv_len - window)              // first visible key
                    : (MOD && sm.chunk > 0) ? ((kv_len - 1) / sm.chunk) * sm.chunk : 0;
     const int hi = kv_len - 1;                                       // the query's own position
-    const int first = lo / DC_N, n_tiles = hi / DC_N - first + 1;
+    const int keep = MOD && window > 0 ? sm.keep : 0;
+    const int w_first = lo / DC_N;                                   // the window's first tile
+    const int n_keep = min((keep + DC_N - 1) / DC_N, w_first);       // tiles of kept positions before it
+    // tile i of the walk is tile i of the keys for i < n_keep, then the window's tiles in turn: `first` is the walk's start,
+    // `skipped` what lies between the two runs
+    const int first = MOD ? 0 : w_first, skipped = w_first - n_keep;
+    const int n_tiles = hi / DC_N - w_first + 1 + (MOD ? n_keep : 0);
+    auto tile_of = [&](int i) { return !MOD ? i : i < n_keep ? i : i + skipped; };
     const int per_split = (n_tiles + num_splits - 1) / num_splits;
     const int t_begin = first + split * per_split;
     const int t_end = min(first + n_tiles, t_begin + per_split);     // exclusive
     const Paging pg(page_size);
-    const StagedTable bt = stage_table(sBT, block_table + (size_t)seg * bt_stride, pg.block(max(lo, t_begin * DC_N)),
-                                       pg.block(min(hi, t_end * DC_N - 1)), tid, DC_WARPS * 32);
+    const StagedTable bt = stage_table(sBT, block_table + (size_t)seg * bt_stride, pg.block(max(lo, tile_of(t_begin) * DC_N)),
+                                       pg.block(min(hi, (tile_of(t_end - 1) + 1) * DC_N - 1)), tid, DC_WARPS * 32);
 
     __syncthreads();                                              // the staged block table
 
@@ -505,8 +524,8 @@ attn_decode_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__ 
     const int n_my = t_begin + warp < t_end ? (t_end - t_begin - warp + DC_WARPS - 1) / DC_WARPS : 0;
     auto issue = [&](int i, int stage) {
         const unsigned st = my_u + stage * STAGE_BYTES;
-        const int j = (t_begin + warp + i * DC_WARPS) * DC_N + lr;
-        bool pred = j >= lo && j <= hi;
+        const int j = tile_of(t_begin + warp + i * DC_WARPS) * DC_N + lr;
+        bool pred = (j >= lo || j < keep) && j <= hi;
         size_t eoff = 0;
         if (pred) {
             const int page = bt.page(pg.block(j));
@@ -523,8 +542,9 @@ attn_decode_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__ 
     // The first tiles are requested before anything else is done; only when this CTA is about to write
     // the new token into the cache and that token's tile is among the first, the requests wait for
     // the write.
-    const bool writes_new = FUSED && fr.write_kv && hi / DC_N >= t_begin && hi / DC_N < t_end;
-    const bool early = !writes_new || hi / DC_N - t_begin >= DC_WARPS * (DC_STAGES - 1);
+    const int t_new = first + n_tiles - 1;                           // the walk's tile that holds the new token: the last
+    const bool writes_new = FUSED && fr.write_kv && t_new >= t_begin && t_new < t_end;
+    const bool early = !writes_new || t_new - t_begin >= DC_WARPS * (DC_STAGES - 1);
     if (early) {
 #pragma unroll
         for (int s = 0; s < DC_STAGES - 1; ++s) {
@@ -544,19 +564,30 @@ attn_decode_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__ 
                 const size_t slot = (((size_t)page * Hkv + kvh) * pg.page_size + pg.row(hi)) * D;
                 if (warp == 0) {
                     bf16* kd = fr.kpool + slot;
-                    warp_norm_rope(tok + (size_t)(Hq + kvh) * D, fr.kw, fr.w_dtype, fr.eps, fr.offset, fr.cos_t, fr.sin_t,
+                    warp_norm_rope(tok + (size_t)(Hq + kvh) * D, fr.kw, fr.w_dtype, fr.eps, fr.offset, fr.norm_n, fr.cos_t, fr.sin_t,
                                    fr.rot_dim, hi, lane, [&](int i) { return kd + i; });
                 } else {
                     const bf16* vs = tok + (size_t)(Hq + Hkv + kvh) * D;
-                    for (int ch = lane; ch < CHUNKS; ch += 32)
-                        *reinterpret_cast<uint4*>(fr.vpool + slot + ch * 8) = *reinterpret_cast<const uint4*>(vs + ch * 8);
+                    if (fr.v_first != nullptr) {
+                        const bf16* vf = fr.v_first + (size_t)tok_row * fr.v_first_ld + (size_t)kvh * fr.v_first_head_stride;
+                        const float share = load_as_f32(fr.v_share, fr.v_share_dtype, 0), own = 1.0f - share;
+                        for (int i = 2 * lane; i < D; i += 64) {
+                            const float2 v = ld_pair(vs + i);
+                            const float f0 = i < fr.v_first_n ? __bfloat162float(vf[i]) : 0.f;
+                            const float f1 = i + 1 < fr.v_first_n ? __bfloat162float(vf[i + 1]) : 0.f;
+                            st_pair(fr.vpool + slot + i, make_float2(own * v.x + share * f0, own * v.y + share * f1));
+                        }
+                    } else {
+                        for (int ch = lane; ch < CHUNKS; ch += 32)
+                            *reinterpret_cast<uint4*>(fr.vpool + slot + ch * 8) = *reinterpret_cast<const uint4*>(vs + ch * 8);
+                    }
                 }
             }
         }
         // the query heads, starting with the warps that had no key or value to write
         for (int r = (warp + 2) % DC_WARPS; r < 16; r += DC_WARPS) {
             if (r < rows_valid) {
-                warp_norm_rope(tok + (size_t)(h0 + r) * D, fr.qw, fr.w_dtype, fr.eps, fr.offset, fr.cos_t, fr.sin_t,
+                warp_norm_rope(tok + (size_t)(h0 + r) * D, fr.qw, fr.w_dtype, fr.eps, fr.offset, fr.norm_n, fr.cos_t, fr.sin_t,
                                fr.rot_dim, hi, lane, [&](int i) { return sQ + soff(r, i >> 3) + (i & 7); });
             } else {
                 for (int ch = lane; ch < CHUNKS; ch += 32) *reinterpret_cast<uint4*>(sQ + soff(r, ch)) = make_uint4(0u, 0u, 0u, 0u);
@@ -600,7 +631,7 @@ attn_decode_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__ 
         cp_async_wait<DC_STAGES - 1>();
         __syncwarp();
         const unsigned tile = my_u + stage * STAGE_BYTES;
-        const int j_base = (t_begin + warp + i * DC_WARPS) * DC_N;
+        const int j_base = tile_of(t_begin + warp + i * DC_WARPS) * DC_N;
         float s[2][4], s2[2][4];                  // two chains over the head dim, added at the end
 #pragma unroll
         for (int e = 0; e < 4; ++e) { s[0][e] = s[1][e] = s2[0][e] = s2[1][e] = 0.f; }
@@ -628,7 +659,7 @@ attn_decode_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__ 
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int j = j_base + nt * 8 + 2 * t4 + (e & 1);
-                    const float v = (j >= lo && j <= hi) ? mod_score(s[nt][e] + s2[nt][e], sm, (e & 2) ? sl1 : sl0, hi - j, (e & 2) ? br1 : br0, (e & 2) ? last1 : last0) : -INFINITY;
+                    const float v = ((j >= lo || j < keep) && j <= hi) ? mod_score(s[nt][e] + s2[nt][e], sm, (e & 2) ? sl1 : sl0, hi - j, (e & 2) ? br1 : br0, (e & 2) ? last1 : last0) : -INFINITY;
                     s[nt][e] = v;
                     if (e & 2) mx1 = fmaxf(mx1, v); else mx0 = fmaxf(mx0, v);
                 }
@@ -817,16 +848,29 @@ attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ 
 
 RB_EXPORT int rb_attn_head_dim() { return D; }
 
-// softcap 0, slopes null, bias null and chunk 0: the plain kernel; anything else: the MOD kernel (a window and a chunk exclude
-// each other).
+namespace {
+// Whether the score options ask for the MOD kernel, and whether they fit each other (a window and a chunk exclude each other;
+// kept first positions go with a window).
+inline bool wants_mod(const ScoreMod& m) { return m.chunk > 0 || m.softcap > 0.f || m.slopes != nullptr || m.bias != nullptr || m.keep > 0; }
+inline bool fits(const ScoreMod& m, int window) {
+    return !(m.bias != nullptr && m.bias_n < 1) && !(window > 0 && m.chunk > 0) && m.keep >= 0 && !(m.keep > 0 && window <= 0);
+}
+inline ScoreMod score_mod(float scale, int chunk, float softcap, const float* slopes, const float* bias, int bias_n, int keep) {
+    ScoreMod m;
+    m.scale = scale; m.softcap = softcap; m.slopes = slopes; m.chunk = chunk; m.bias = bias; m.bias_n = bias ? bias_n : 0; m.keep = keep;
+    return m;
+}
+}  // namespace
+
+// softcap 0, slopes null, bias null, chunk 0 and keep 0: the plain kernel; anything else: the MOD kernel.
 RB_EXPORT int rb_attn_prefill_mod(const void* q, int ld, const void* kpool, const void* vpool, const int* tiles,
                                   int n_tiles, const int* cu_q, const int* seg_pos0, const int* block_table,
                                   int bt_stride, int page_size, void* out, int Hq, int Hkv, float scale,
                                   int window, const float* sink, int chunk, float softcap, const float* slopes,
-                                  const float* bias, int bias_n, cudaStream_t st) {
+                                  const float* bias, int bias_n, int keep, cudaStream_t st) {
     if (n_tiles <= 0) return 0;
-    if (bias != nullptr && bias_n < 1) return (int)cudaErrorInvalidValue;
-    if (window > 0 && chunk > 0) return (int)cudaErrorInvalidValue;
+    const ScoreMod sm = score_mod(scale, chunk, softcap, slopes, bias, bias_n, keep);
+    if ((bias != nullptr && bias_n < 1) || !fits(sm, window)) return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)(PF_M + 4 * PF_N) * D * sizeof(bf16) + BT_CAP * sizeof(int);
     static PerDevice configured;
     const int cfg = configured.once([&](int) {
@@ -836,9 +880,7 @@ RB_EXPORT int rb_attn_prefill_mod(const void* q, int ld, const void* kpool, cons
     });
     if (cfg != 0) return cfg;
     dim3 grid(n_tiles, Hq);
-    ScoreMod sm;
-    sm.scale = scale; sm.softcap = softcap; sm.slopes = slopes; sm.chunk = chunk; sm.bias = bias; sm.bias_n = bias ? bias_n : 0;
-    if (chunk > 0 || softcap > 0.f || slopes != nullptr || bias != nullptr)
+    if (wants_mod(sm))
         return rb_launch_pdl(attn_prefill_kernel<true>, grid, dim3(128), smem, st, (const bf16*)q, ld, (const bf16*)kpool,
                              (const bf16*)vpool, tiles, cu_q, seg_pos0, block_table, bt_stride, page_size, (bf16*)out,
                              Hq, Hkv, scale * LOG2E, window, sink, sm);
@@ -852,7 +894,7 @@ RB_EXPORT int rb_attn_prefill(const void* q, int ld, const void* kpool, const vo
                               int bt_stride, int page_size, void* out, int Hq, int Hkv, float scale,
                               int window, const float* sink, cudaStream_t st) {
     return rb_attn_prefill_mod(q, ld, kpool, vpool, tiles, n_tiles, cu_q, seg_pos0, block_table, bt_stride, page_size, out,
-                               Hq, Hkv, scale, window, sink, 0, 0.f, nullptr, nullptr, 0, st);
+                               Hq, Hkv, scale, window, sink, 0, 0.f, nullptr, nullptr, 0, 0, st);
 }
 
 // Floats of scratch that rb_attn_decode needs: part_o [n_dec, Hq, splits, D], part_ml [n_dec, Hq, splits, 2].
@@ -878,6 +920,7 @@ int launch_decode(const void* q, int ld, const void* kpool, const void* vpool, c
         cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_decode_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_decode_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_decode_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         return e;
     });
     if (cfg != 0) return cfg;
@@ -887,8 +930,11 @@ int launch_decode(const void* q, int ld, const void* kpool, const void* vpool, c
     FusedRope none = {};
     ScoreMod plain = {};
     int rc;
-    if (mod != nullptr && fused != nullptr) return (int)cudaErrorInvalidValue;
-    if (mod != nullptr)
+    if (mod != nullptr && fused != nullptr)
+        rc = rb_launch_pdl(attn_decode_kernel<true, true>, grid, dim3(DC_WARPS * 32), smem, st,
+            (const bf16*)q, ld, (const bf16*)kpool, (const bf16*)vpool, dec_segs, cu_q, seg_kv_len, block_table,
+            bt_stride, page_size, part_o, part_ml, (bf16*)out, Hq, Hkv, m_tiles, scale * LOG2E, window, num_splits, *fused, sink, *mod);
+    else if (mod != nullptr)
         rc = rb_launch_pdl(attn_decode_kernel<false, true>, grid, dim3(DC_WARPS * 32), smem, st,
             (const bf16*)q, ld, (const bf16*)kpool, (const bf16*)vpool, dec_segs, cu_q, seg_kv_len, block_table,
             bt_stride, page_size, part_o, part_ml, (bf16*)out, Hq, Hkv, m_tiles, scale * LOG2E, window, num_splits, none, sink, *mod);
@@ -920,32 +966,38 @@ RB_EXPORT int rb_attn_decode_mod(const void* q, int ld, const void* kpool, const
                                  int n_dec, const int* cu_q, const int* seg_kv_len, const int* block_table,
                                  int bt_stride, int page_size, float* scratch, void* out, int Hq, int Hkv,
                                  float scale, int window, int num_splits, const float* sink, int chunk, float softcap,
-                                 const float* slopes, const float* bias, int bias_n, cudaStream_t st) {
-    if ((window > 0 && chunk > 0) || (bias != nullptr && bias_n < 1)) return (int)cudaErrorInvalidValue;
-    if (chunk <= 0 && softcap <= 0.f && slopes == nullptr && bias == nullptr)
-        return launch_decode(q, ld, kpool, vpool, dec_segs, n_dec, cu_q, seg_kv_len, block_table, bt_stride, page_size,
-                             scratch, out, Hq, Hkv, scale, window, num_splits, nullptr, sink, st);
-    ScoreMod sm;
-    sm.scale = scale; sm.softcap = softcap; sm.slopes = slopes; sm.chunk = chunk; sm.bias = bias; sm.bias_n = bias ? bias_n : 0;
+                                 const float* slopes, const float* bias, int bias_n, int keep, cudaStream_t st) {
+    const ScoreMod sm = score_mod(scale, chunk, softcap, slopes, bias, bias_n, keep);
+    if ((bias != nullptr && bias_n < 1) || !fits(sm, window)) return (int)cudaErrorInvalidValue;
     return launch_decode(q, ld, kpool, vpool, dec_segs, n_dec, cu_q, seg_kv_len, block_table, bt_stride, page_size,
-                         scratch, out, Hq, Hkv, scale, window, num_splits, nullptr, sink, st, &sm);
+                         scratch, out, Hq, Hkv, scale, window, num_splits, nullptr, sink, st, wants_mod(sm) ? &sm : nullptr);
 }
 
-// The same for a step of single tokens only, with the q/k norm, the rotation and the cache write of
-// those tokens done inside (qkv holds the raw projections; nothing else has touched them).
+// The same for a step of single tokens only, with the q/k norm, the rotation, the blend of the values and the cache write of
+// those tokens done inside (qkv holds the raw projections; nothing else has touched them).  norm_n 0: the norm's mean
+// runs over all of a head.  v_first null: no blend.
 RB_EXPORT int rb_attn_decode_fused(const void* qkv, int ld, void* kpool, void* vpool, const int* dec_segs,
                                    int n_dec, const int* cu_q, const int* seg_kv_len, const int* block_table,
                                    int bt_stride, int page_size, float* scratch, void* out, int Hq, int Hkv,
                                    float scale, int window, int num_splits, const void* qw, const void* kw,
                                    int w_dtype, float eps, float offset, const float* cos_t, const float* sin_t,
-                                   int rot_dim, int write_kv, cudaStream_t st) {
+                                   int rot_dim, int write_kv, int norm_n, const void* v_first, int v_first_ld,
+                                   int v_first_head_stride, int v_first_n, const void* v_share, int v_share_dtype,
+                                   const float* sink, int chunk, float softcap, const float* slopes, const float* bias,
+                                   int bias_n, int keep, cudaStream_t st) {
+    const ScoreMod sm = score_mod(scale, chunk, softcap, slopes, bias, bias_n, keep);
+    if ((bias != nullptr && bias_n < 1) || !fits(sm, window)) return (int)cudaErrorInvalidValue;
     if (rot_dim > D || (rot_dim & 3) || rot_dim > 256) return (int)cudaErrorInvalidValue;
+    if (norm_n < 0 || norm_n > D || (v_first != nullptr && v_share == nullptr)) return (int)cudaErrorInvalidValue;
     FusedRope fr;
     fr.qw = qw; fr.kw = kw; fr.w_dtype = w_dtype; fr.eps = eps; fr.offset = offset;
     fr.cos_t = cos_t; fr.sin_t = sin_t; fr.rot_dim = rot_dim;
     fr.kpool = (bf16*)kpool; fr.vpool = (bf16*)vpool; fr.write_kv = write_kv;
+    fr.norm_n = norm_n ? norm_n : D;
+    fr.v_first = (const bf16*)v_first; fr.v_first_ld = v_first_ld; fr.v_first_head_stride = v_first_head_stride;
+    fr.v_first_n = v_first_n; fr.v_share = v_share; fr.v_share_dtype = v_share_dtype;
     return launch_decode(qkv, ld, kpool, vpool, dec_segs, n_dec, cu_q, seg_kv_len, block_table, bt_stride, page_size,
-                         scratch, out, Hq, Hkv, scale, window, num_splits, &fr, nullptr, st);
+                         scratch, out, Hq, Hkv, scale, window, num_splits, &fr, sink, st, wants_mod(sm) ? &sm : nullptr);
 }
 
 // ------------------------------------------------------------------ decode attention without allocation

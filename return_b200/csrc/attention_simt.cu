@@ -15,7 +15,7 @@
 // Options of the score, all off by default: `chunk` > 0 bounds the keys from below by the start of the query's own
 // block of `chunk` positions (blocks counted from position 0) instead of a window; `softcap` > 0 turns a scaled score
 // s into softcap * tanh(s / softcap); `slopes` [Hq] takes slopes[h] * (p - j) off the score of key j; `bias` [Hq, bias_n] adds
-// bias[h, min(p - j, bias_n - 1)] to it; `sink` [Hq] adds exp(sink[h]) to the softmax's denominator (a term with no key and
+// bias[h, min(p - j, bias_n - 1)] to it; `keep` > 0 (with a window) leaves the first `keep` positions visible for every later query; `sink` [Hq] adds exp(sink[h]) to the softmax's denominator (a term with no key and
 // no value).
 #include "common.cuh"
 
@@ -28,7 +28,7 @@ attention_simt_kernel(const TA* __restrict__ q, int ld, const TA* __restrict__ k
                       const int* __restrict__ tok_seg, const int* __restrict__ block_table,
                       int bt_stride, int page_size, TA* __restrict__ out, int Hq, int Hkv, int D,
                       float scale, int window, int chunk, float softcap, const float* __restrict__ slopes,
-                      const float* __restrict__ sink, const float* __restrict__ bias, int bias_n) {
+                      const float* __restrict__ sink, const float* __restrict__ bias, int bias_n, int keep) {
     extern __shared__ float qs_all[];                    // 4 warps x D floats
     const int t = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -50,9 +50,10 @@ attention_simt_kernel(const TA* __restrict__ q, int ld, const TA* __restrict__ k
     for (int i = 0; i < SIMT_MAX_D / 32; ++i) acc[i] = 0.f;
     const size_t head_stride = (size_t)page_size * D;    // one kv head of one page
 
-    for (int j0 = (lo / 32) * 32; j0 <= p; j0 += 32) {
+    const int first_tile = (lo / 32) * 32;               // the tiles of kept positions come first, then the window's
+    for (int j0 = keep > 0 ? 0 : first_tile; j0 <= p; j0 = j0 < first_tile && j0 + 32 >= keep ? first_tile : j0 + 32) {
         const int j = j0 + lane;
-        const bool valid = j >= lo && j <= p;
+        const bool valid = (j >= lo || j < keep) && j <= p;
         float s = -INFINITY;
         if (valid) {
             const int page = bt[j / page_size];
@@ -75,9 +76,10 @@ attention_simt_kernel(const TA* __restrict__ q, int ld, const TA* __restrict__ k
 #pragma unroll
         for (int i = 0; i < SIMT_MAX_D / 32; ++i) acc[i] *= alpha;
         const int jend = min(32, p - j0 + 1);
-        for (int jj = max(0, lo - j0); jj < jend; ++jj) {
+        for (int jj = j0 < keep ? 0 : max(0, lo - j0); jj < jend; ++jj) {
             const float pjj = __shfl_sync(0xffffffffu, pj, jj);
             const int jk = j0 + jj;
+            if (jk < lo && jk >= keep) continue;
             const int page = bt[jk / page_size];
             if (page < 0) continue;
             const TA* vr = vpool + ((size_t)page * Hkv + kvh) * head_stride + (size_t)(jk % page_size) * D;
@@ -103,21 +105,21 @@ RB_EXPORT int rb_attention_simt_mod(const void* q, int ld, const void* kpool, co
                                 const int* pos, const int* tok_seg, const int* block_table,
                                 int bt_stride, int page_size, void* out, int act_dtype, int T,
                                 int Hq, int Hkv, int D, float scale, int window, int chunk, float softcap,
-                                const float* slopes, const float* sink, const float* bias, int bias_n, cudaStream_t st) {
+                                const float* slopes, const float* sink, const float* bias, int bias_n, int keep, cudaStream_t st) {
     if (T <= 0) return 0;
     if (bias != nullptr && bias_n < 1) return (int)cudaErrorInvalidValue;
-    if (window > 0 && chunk > 0) return (int)cudaErrorInvalidValue;
+    if ((window > 0 && chunk > 0) || keep < 0 || (keep > 0 && window <= 0)) return (int)cudaErrorInvalidValue;
     if (D > SIMT_MAX_D || D <= 0 || Hkv <= 0 || Hq % Hkv) return (int)cudaErrorInvalidValue;
     dim3 grid(T, (Hq + 3) / 4);
     const size_t smem = (size_t)4 * D * sizeof(float);
     if (act_dtype == RB_F32)
         attention_simt_kernel<float><<<grid, 128, smem, st>>>(
             (const float*)q, ld, (const float*)kpool, (const float*)vpool, pos, tok_seg, block_table,
-            bt_stride, page_size, (float*)out, Hq, Hkv, D, scale, window, chunk, softcap, slopes, sink, bias, bias_n);
+            bt_stride, page_size, (float*)out, Hq, Hkv, D, scale, window, chunk, softcap, slopes, sink, bias, bias_n, keep);
     else
         attention_simt_kernel<bf16><<<grid, 128, smem, st>>>(
             (const bf16*)q, ld, (const bf16*)kpool, (const bf16*)vpool, pos, tok_seg, block_table,
-            bt_stride, page_size, (bf16*)out, Hq, Hkv, D, scale, window, chunk, softcap, slopes, sink, bias, bias_n);
+            bt_stride, page_size, (bf16*)out, Hq, Hkv, D, scale, window, chunk, softcap, slopes, sink, bias, bias_n, keep);
     return rb_launch_status();
 }
 
@@ -126,5 +128,5 @@ RB_EXPORT int rb_attention_simt(const void* q, int ld, const void* kpool, const 
                                 int bt_stride, int page_size, void* out, int act_dtype, int T,
                                 int Hq, int Hkv, int D, float scale, int window, cudaStream_t st) {
     return rb_attention_simt_mod(q, ld, kpool, vpool, pos, tok_seg, block_table, bt_stride, page_size, out, act_dtype, T,
-                                 Hq, Hkv, D, scale, window, 0, 0.f, nullptr, nullptr, nullptr, 0, st);
+                                 Hq, Hkv, D, scale, window, 0, 0.f, nullptr, nullptr, nullptr, 0, 0, st);
 }

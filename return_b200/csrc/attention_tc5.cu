@@ -40,7 +40,9 @@
 // with the distance, slopes[h] * (i - j), taken off before the softmax, and a bias per head and distance added to the
 // score, bias[h, min(i - j, bias_n - 1)]: only key tiles within the table's reach look it up (neighbouring rows read
 // neighbouring entries), behind it the last entry is a constant.  A row's thread does that to its 64 scores
-// of a key tile right after it has read them from tensor memory; everything else is the plain kernel.
+// of a key tile right after it has read them from tensor memory; everything else is the plain kernel.  With a window it can
+// also keep the first `keep` positions visible for every later query: the key tiles are then walked in two runs, the tiles
+// of the kept positions that lie before the window's first tile, then the window's.
 // A step with too few such CTAs to fill the GPU (a short portion of a long prompt) splits the keys of every
 // block over gridDim.z CTAs; each leaves its unnormalised O with its reference maximum and sum in float32,
 // and a second kernel merges them (the same arithmetic as the decode kernel's merge).
@@ -148,6 +150,7 @@ struct ScoreMod {
     int chunk;                 // 0: none
     const float* bias;         // [Hq, bias_n] or null
     int bias_n;
+    int keep;                  // with a window: the first `keep` positions stay visible (0: none)
 };
 
 template <bool MOD>
@@ -183,7 +186,13 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
     const int p_last = p0 + m_rows - 1;
     const int chunk = MOD ? sm.chunk : 0;
     const int lo_min = window > 0 ? max(0, p0 - window + 1) : chunk > 0 ? (p0 / chunk) * chunk : 0;
-    int jt_first = lo_min / KN;
+    const int keep = MOD && window > 0 ? sm.keep : 0;
+    const int jt_window = lo_min / KN;                    // the first key tile of the window (or of all keys)
+    const int n_keep = MOD ? min((keep + KN - 1) / KN, jt_window) : 0;       // tiles of kept positions before it
+    // the walk's tiles are numbered jt_first, jt_first + 1, ...; tile_of turns a number into a key tile.  With kept tiles they
+    // come first: the numbers then start at n_keep tiles below the window's
+    int jt_first = jt_window - n_keep;
+    auto tile_of = [&](int jt) { return !MOD || jt >= jt_window ? jt : jt - (jt_window - n_keep); };
     // key tiles of each query tile, counted from the first: B (if it has rows) needs all of the block's, A stops earlier
     int na = min(p_last, p0 + QM - 1) / KN - jt_first + 1;
     int nb = m_rows > QM ? p_last / KN - jt_first + 1 : 0;
@@ -252,10 +261,10 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
         const unsigned lane_addr = tmem + ((unsigned)((warp & 3) * 32) << 16);
         const unsigned o_addr = lane_addr + O_COL + qt * D;
         for (int t = 0; t < n_mine; ++t) {
-            const int j_base = (jt_begin + t) * KN;
+            const int j_base = tile_of(jt_begin + t) * KN;
             ok = mbar_wait(bar(B_S_FULL + qt * 2 + (t & 1)), (t >> 1) & 1) && ok;
             fence_after_sync();
-            const bool all_visible = full_tile && j_base + KN - 1 <= p0_t && (window <= 0 || j_base > p_last_t - window) &&
+            const bool all_visible = full_tile && j_base + KN - 1 <= p0_t && (window <= 0 || j_base > p_last_t - window || (MOD && j_base + KN - 1 < keep)) &&
                                      (chunk <= 0 || j_base >= (p_last_t / max(chunk, 1)) * chunk);
             unsigned a[64];
             tmem_ld32(lane_addr + (qt * 2 + (t & 1)) * KN, reinterpret_cast<unsigned(&)[32]>(a[0]));
@@ -295,7 +304,7 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
 #pragma unroll
                     for (int i = 0; i < 64; ++i) {
                         const int j = j_base + i;
-                        const bool vis = row_valid && j <= pos_r && (window <= 0 || j > pos_r - window) && j >= lo_r;
+                        const bool vis = row_valid && j <= pos_r && (window <= 0 || j > pos_r - window || j < keep) && j >= lo_r;
                         if (!vis) a[i] = 0xff800000u;
                         mx = fmaxf(mx, __uint_as_float(a[i]));
                     }
@@ -498,11 +507,11 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
                 const int j = jt * KN + u * 32 + lane;
-                page[u] = bt_row[j >= lo_min && j <= p_last ? pg.block(j) : 0];      // entry 0 exists; the range is checked again at use
+                page[u] = bt_row[(j >= lo_min || j < keep) && j <= p_last ? pg.block(j) : 0];      // entry 0 exists; the range is checked again at use
             }
         };
         int next_page[2];
-        ask_pages(jt_begin, next_page);
+        ask_pages(tile_of(jt_begin), next_page);
         for (int t = 0; t < n_tiles; ++t) {
             if (t >= STAGES) {
                 // the stage held tile t - 3: its keys are free when S(t - 3) is computed, its values when P V(t - 3) is done
@@ -512,7 +521,7 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
                 if (f < n_b) ok = mbar_wait(bar(b_free + 2 + (f & 1)), (f >> 1) & 1) && ok;
             }
             const unsigned tile_smem = bufs + st * K_BYTES;
-            const int jt = jt_begin + t;
+            const int jt = tile_of(jt_begin + t);
             // Lane L looks up where rows L and L + 32 of the tile lie (a null pointer: not to be read).  The copies
             // then go row by row, D / 8 neighbouring lanes taking the 16-byte pieces of one row, so that a
             // warp's instruction reads whole 128-byte lines; each row's address comes from the lane that
@@ -523,7 +532,7 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
             for (int u = 0; u < 2; ++u) {
                 const int j = jt * KN + u * 32 + lane;
                 where[u] = 0ull;
-                if (j >= lo_min && j <= p_last && next_page[u] >= 0)
+                if ((j >= lo_min || j < keep) && j <= p_last && next_page[u] >= 0)
                     where[u] = reinterpret_cast<unsigned long long>(pool + (((size_t)next_page[u] * Hkv + kvh) * pg.page_size + pg.row(j)) * D);
             }
             constexpr int LPR = D / 8, RPI = 32 / LPR;              // lanes a row, rows an instruction
@@ -541,7 +550,7 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
                 }
             }
             cp_async_commit();
-            if (t + 1 < n_tiles) ask_pages(jt + 1, next_page);
+            if (t + 1 < n_tiles) ask_pages(tile_of(jt_begin + t + 1), next_page);
             // tile t is on its way; tile t - 1 has to have landed.  It is announced only now, after the wait for
             // the stage above: the product that completes the next phase of that wait's barrier needs this
             // announcement, so the wait cannot fall a phase behind.
@@ -616,17 +625,18 @@ RB_EXPORT long long rb_attn_tc5_split_floats(int n_split, int total_rows, int Hq
 // tiles: [n_tiles, 2] = (segment, first row of a block of up to 256 query rows), the blocks with the
 // longest contexts first.  n_split > 1 splits the keys of every block over that many CTAs; ``scratch`` then
 // holds rb_attn_tc5_split_floats(...) floats and total_rows is the number of rows of q.
-// chunk, softcap, slopes, bias: the score options (0, 0, null, null: the plain kernel); a window and a chunk exclude each other.
+// chunk, softcap, slopes, bias, keep: the score options (0, 0, null, null, 0: the plain kernel); a window and a chunk exclude
+// each other, kept first positions go with a window.
 RB_EXPORT int rb_attn_prefill_tc5_mod(const void* q, int ld, const void* kpool, const void* vpool, const int* tiles,
                                       int n_tiles, const int* cu_q, const int* seg_pos0, const int* block_table,
                                       int bt_stride, int page_size, void* out, int Hq, int Hkv, float scale, int window,
                                       int n_split, void* scratch, int total_rows, int* status, const float* sink,
                                       int chunk, float softcap, const float* slopes, const float* bias, int bias_n,
-                                      cudaStream_t st) {
+                                      int keep, cudaStream_t st) {
     if (n_tiles <= 0) return 0;
     if (bias != nullptr && bias_n < 1) return (int)cudaErrorInvalidValue;
     if (n_tiles > 65535 || n_split < 1 || n_split > 64 || (n_split > 1 && scratch == nullptr)) return (int)cudaErrorInvalidValue;
-    if (window > 0 && chunk > 0) return (int)cudaErrorInvalidValue;
+    if ((window > 0 && chunk > 0) || keep < 0 || (keep > 0 && window <= 0)) return (int)cudaErrorInvalidValue;
     static PerDevice configured;
     const int rc = configured.once([](int) {
         cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc5_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
@@ -638,8 +648,8 @@ RB_EXPORT int rb_attn_prefill_tc5_mod(const void* q, int ld, const void* kpool, 
     float* part_ml = part_o ? part_o + (size_t)n_split * total_rows * Hq * D : nullptr;
     dim3 grid(Hq, n_tiles, n_split);
     ScoreMod sm;
-    sm.scale = scale; sm.softcap = softcap; sm.slopes = slopes; sm.chunk = chunk; sm.bias = bias; sm.bias_n = bias ? bias_n : 0;
-    if (chunk > 0 || softcap > 0.f || slopes != nullptr || bias != nullptr)
+    sm.scale = scale; sm.softcap = softcap; sm.slopes = slopes; sm.chunk = chunk; sm.bias = bias; sm.bias_n = bias ? bias_n : 0; sm.keep = keep;
+    if (chunk > 0 || softcap > 0.f || slopes != nullptr || bias != nullptr || keep > 0)
         attn_prefill_tc5_kernel<true><<<grid, THREADS, SMEM_BYTES, st>>>(
             (const bf16*)q, ld, (const bf16*)kpool, (const bf16*)vpool, tiles, cu_q, seg_pos0, block_table, bt_stride,
             page_size, (bf16*)out, Hq, Hkv, scale * LOG2E, window, part_o, part_ml, total_rows, status, sink, sm);
@@ -660,5 +670,5 @@ RB_EXPORT int rb_attn_prefill_tc5(const void* q, int ld, const void* kpool, cons
                                   int n_split, void* scratch, int total_rows, int* status, const float* sink,
                                   cudaStream_t st) {
     return rb_attn_prefill_tc5_mod(q, ld, kpool, vpool, tiles, n_tiles, cu_q, seg_pos0, block_table, bt_stride, page_size, out,
-                                   Hq, Hkv, scale, window, n_split, scratch, total_rows, status, sink, 0, 0.f, nullptr, nullptr, 0, st);
+                                   Hq, Hkv, scale, window, n_split, scratch, total_rows, status, sink, 0, 0.f, nullptr, nullptr, 0, 0, st);
 }

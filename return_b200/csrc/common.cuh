@@ -79,6 +79,14 @@ __device__ __forceinline__ float rb_activate(int op, float v, const void* bias, 
     return expf(-expf(v + (bias ? load_as_f32(bias, bias_dtype, c) : 0.f)));
 }
 
+// The gate of a gated unit is g sigmoid(a(g)): with a(g) = g that is silu, and with a(g) = 2 sqrt(2/pi) (g + 0.044715 g^3) the
+// tanh form of gelu, since 0.5 (1 + tanh(z)) = sigmoid(2 z).
+#define GATE_SILU 0
+#define GATE_GELU_TANH 1
+__device__ __forceinline__ float rb_gate_arg(int gate, float g) {
+    return gate == GATE_GELU_TANH ? 1.5957691216057308f * fmaf(0.044715f * g * g, g, g) : g;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -263,11 +263,11 @@ RB_EXPORT int rb_rmsnorm_rows(const void* x, const void* w, int w_dtype, float e
 }
 
 // ---------------------------------------------------------------- SwiGLU
-// out[t, i] = silu(gate) * up.  gu is [T, 2I].  block == 0: gate columns [0, I), up columns [I, 2I)
+// out[t, i] = silu(gate) * up, or with another gate (rb_gate_arg in common.cuh).  gu is [T, 2I].  block == 0: gate columns [0, I), up columns [I, 2I)
 // (the reference's concatenation, rollout/monkey_patch/qwen3.py:99-105).  block == 8: columns come in
 // blocks of 8 gate then 8 up (the layout that lets a matrix product's epilogue do this step).
 template <typename TA>
-__global__ void swiglu_kernel(const TA* __restrict__ gu, TA* __restrict__ out, int T, int I, int block) {
+__global__ void swiglu_kernel(const TA* __restrict__ gu, TA* __restrict__ out, int T, int I, int block, int gate) {
     const size_t total = (size_t)T * I;
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
          idx += (size_t)gridDim.x * blockDim.x) {
@@ -276,7 +276,7 @@ __global__ void swiglu_kernel(const TA* __restrict__ gu, TA* __restrict__ out, i
         const size_t ui = block ? gi + block : I + i;
         const float g = to_f32(gu[t * 2 * I + gi]);
         const float u = to_f32(gu[t * 2 * I + ui]);
-        out[idx] = from_f32<TA>(g / (1.0f + expf(-g)) * u);
+        out[idx] = from_f32<TA>(g / (1.0f + expf(-rb_gate_arg(gate, g))) * u);
     }
 }
 
@@ -284,7 +284,7 @@ __global__ void swiglu_kernel(const TA* __restrict__ gu, TA* __restrict__ out, i
 // The exponential and the division are the fast float32 forms (a few units in the last place, far
 // below the rounding to bfloat16 that follows): with the accurate ones the kernel is bound by
 // instruction issue, not by memory.
-__device__ __forceinline__ uint4 swiglu8(const uint4 gv, const uint4 uv) {
+__device__ __forceinline__ uint4 swiglu8(const uint4 gv, const uint4 uv, int gate) {
     const bf16* g = (const bf16*)&gv;
     const bf16* u = (const bf16*)&uv;
     uint4 ov;
@@ -292,12 +292,12 @@ __device__ __forceinline__ uint4 swiglu8(const uint4 gv, const uint4 uv) {
 #pragma unroll
     for (int k = 0; k < 8; ++k) {
         const float gf = __bfloat162float(g[k]);
-        o[k] = __float2bfloat16_rn(__fdividef(gf, 1.0f + __expf(-gf)) * __bfloat162float(u[k]));
+        o[k] = __float2bfloat16_rn(__fdividef(gf, 1.0f + __expf(-rb_gate_arg(gate, gf))) * __bfloat162float(u[k]));
     }
     return ov;
 }
 
-__global__ void swiglu_bf16x8_kernel(const bf16* __restrict__ gu, bf16* __restrict__ out, int T, int I, int block) {
+__global__ void swiglu_bf16x8_kernel(const bf16* __restrict__ gu, bf16* __restrict__ out, int T, int I, int block, int gate) {
     pdl_launch_dependents();
     pdl_wait();
     const int I8 = I >> 3;
@@ -312,85 +312,171 @@ __global__ void swiglu_bf16x8_kernel(const bf16* __restrict__ gu, bf16* __restri
         const uint4 uv = *(const uint4*)(gu + t * 2 * I + (block ? 2 * i + 8 : I + i));
         const uint4 gv2 = *(const uint4*)(gu + t2 * 2 * I + (block ? 2 * i2 : i2));
         const uint4 uv2 = *(const uint4*)(gu + t2 * 2 * I + (block ? 2 * i2 + 8 : I + i2));
-        *(uint4*)(out + t * I + i) = swiglu8(gv, uv);
-        if (two) *(uint4*)(out + t2 * I + i2) = swiglu8(gv2, uv2);
+        *(uint4*)(out + t * I + i) = swiglu8(gv, uv, gate);
+        if (two) *(uint4*)(out + t2 * I + i2) = swiglu8(gv2, uv2, gate);
     }
 }
 
-RB_EXPORT int rb_swiglu(const void* gu, void* out, int act_dtype, int T, int I, int block, cudaStream_t st) {
+RB_EXPORT int rb_swiglu(const void* gu, void* out, int act_dtype, int T, int I, int block, int gate, cudaStream_t st) {
     if (T <= 0) return 0;
+    if (gate < 0 || gate > GATE_GELU_TANH) return (int)cudaErrorInvalidValue;
     if (block != 0 && (block != 8 || I % 8)) return (int)cudaErrorInvalidValue;
     const int threads = 256;
     if (act_dtype == RB_BF16 && (I % 8) == 0 && ((uintptr_t)gu % 16) == 0 && ((uintptr_t)out % 16) == 0) {
         const size_t total = (size_t)T * (I >> 3);
         int blocks = (int)((total + threads - 1) / threads);
         if (blocks > 148 * 16) blocks = 148 * 16;
-        return rb_launch_pdl(swiglu_bf16x8_kernel, dim3(blocks), dim3(threads), 0, st, (const bf16*)gu, (bf16*)out, T, I, block);
+        return rb_launch_pdl(swiglu_bf16x8_kernel, dim3(blocks), dim3(threads), 0, st, (const bf16*)gu, (bf16*)out, T, I, block, gate);
     }
     const size_t total = (size_t)T * I;
     int blocks = (int)((total + threads - 1) / threads);
     if (blocks > 148 * 16) blocks = 148 * 16;
     if (act_dtype == RB_F32)
-        swiglu_kernel<float><<<blocks, threads, 0, st>>>((const float*)gu, (float*)out, T, I, block);
+        swiglu_kernel<float><<<blocks, threads, 0, st>>>((const float*)gu, (float*)out, T, I, block, gate);
     else
-        swiglu_kernel<bf16><<<blocks, threads, 0, st>>>((const bf16*)gu, (bf16*)out, T, I, block);
+        swiglu_kernel<bf16><<<blocks, threads, 0, st>>>((const bf16*)gu, (bf16*)out, T, I, block, gate);
     return rb_launch_status();
 }
 
 
+// ---------------------------------------------------------------- VEC neighbouring elements at a time
+// 4 where rows are multiples of 4 (16-byte loads and stores of float32), else 1.
+template <int VEC> __device__ __forceinline__ void load_vec(const float* p, float (&v)[VEC]) {
+    if constexpr (VEC == 4) { const float4 q = *reinterpret_cast<const float4*>(p); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
+    else v[0] = *p;
+}
+template <int VEC> __device__ __forceinline__ void load_vec(const bf16* p, float (&v)[VEC]) {
+    if constexpr (VEC == 4) {
+        const uint2 q = *reinterpret_cast<const uint2*>(p);
+        const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
+        const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+        v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+    } else v[0] = to_f32(*p);
+}
+template <int VEC> __device__ __forceinline__ void store_vec(float* p, const float (&v)[VEC]) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else *p = v[0];
+}
+template <int VEC> __device__ __forceinline__ void store_vec(bf16* p, const float (&v)[VEC]) {
+    if constexpr (VEC == 4) {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+        uint2 q;
+        q.x = *reinterpret_cast<const unsigned*>(&lo);
+        q.y = *reinterpret_cast<const unsigned*>(&hi);
+        *reinterpret_cast<uint2*>(p) = q;
+    } else *p = __float2bfloat16_rn(v[0]);
+}
+
 // ---------------------------------------------------------------- a sublayer's output normed before it joins the stream
-// For layers that norm a sublayer's output as well as its input: stream[r] += rmsnorm(delta[r]) * (offset_post + w_post),
-// and, if asked, out[r] = rmsnorm(stream[r]) * (offset_next + w_next) for the sublayer that runs next: one kernel at
-// every joint of such a layer.  float32 arithmetic; the row stays in shared memory between the two sums.
-template <typename TA>
-__global__ void postnorm_add_norm_kernel(float* __restrict__ stream, const TA* __restrict__ delta, const void* __restrict__ w_post,
-                                         int wp_dtype, float eps_post, float offset_post, const void* __restrict__ w_next,
-                                         int wn_dtype, float eps_next, float offset_next, TA* __restrict__ out, int H) {
-    extern __shared__ float smem[];
-    float* xrow = smem;          // H floats
-    float* scratch = smem + H;   // 33 floats
+// For layers that norm a sublayer's output: stream[r] += rmsnorm(delta[r]) * (offset_post + w_post), and, if asked, the rows
+// that the sublayer which runs next reads: out[r] = rmsnorm(stream[r]) * (offset_next + w_next), or, without w_next, the
+// stream itself in the activation type: one kernel at every joint of such a layer.  Without a delta nothing is added
+// (the rows for a model's first sublayer).  float32 arithmetic.  Which columns a thread sums depends on H alone.
+struct Joint {
+    const void* w_post;
+    int wp_dtype;
+    float eps_post, offset_post;
+    const void* w_next;
+    int wn_dtype;
+    float eps_next, offset_next;
+};
+
+// A row stays in the registers of its CTA: at most CH pieces of VEC columns a thread; everything is asked for before the
+// first sum.
+template <typename TA, int VEC, int CH>
+__global__ void __launch_bounds__(1024)
+postnorm_add_norm_kernel(float* __restrict__ stream, const TA* __restrict__ delta, const Joint J, TA* __restrict__ out, int H) {
+    __shared__ float scratch[33];
     pdl_launch_dependents();
     pdl_wait();
-    const int row = blockIdx.x;
-    float* s = stream + (size_t)row * H;
-    const TA* d = delta + (size_t)row * H;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        const float v = to_f32(d[i]);
-        xrow[i] = v;
-        ss += v * v;
+    float* s = stream + (size_t)blockIdx.x * H;
+    const TA* d = delta + (size_t)blockIdx.x * H;
+    float x[CH][VEC], y[CH][VEC];
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int i = (threadIdx.x + c * blockDim.x) * VEC;
+        if (i < H) {
+            load_vec<VEC>(s + i, x[c]);
+            if (delta != nullptr) load_vec<VEC>(d + i, y[c]);
+        }
     }
-    ss = block_sum(ss, scratch);
-    const float rstd_d = 1.0f / sqrtf(ss / (float)H + eps_post);
-    float ss2 = 0.f;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        const float x = s[i] + xrow[i] * rstd_d * (offset_post + load_as_f32(w_post, wp_dtype, i));
-        s[i] = x;
-        xrow[i] = x;
-        ss2 += x * x;
+    if (delta != nullptr) {
+        float ss = 0.f;
+#pragma unroll
+        for (int c = 0; c < CH; ++c)
+            if ((threadIdx.x + c * blockDim.x) * VEC < H) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) ss = fmaf(y[c][e], y[c][e], ss);
+            }
+        ss = block_sum(ss, scratch);
+        const float rstd = 1.0f / sqrtf(ss / (float)H + J.eps_post);
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+            const int i = (threadIdx.x + c * blockDim.x) * VEC;
+            if (i < H) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e)
+                    x[c][e] += y[c][e] * rstd * (J.offset_post + load_as_f32(J.w_post, J.wp_dtype, (size_t)(i + e)));
+                store_vec<VEC>(s + i, x[c]);
+            }
+        }
     }
     pdl_trigger_late();
     if (out == nullptr) return;
-    ss2 = block_sum(ss2, scratch);
-    const float rstd = 1.0f / sqrtf(ss2 / (float)H + eps_next);
-    TA* o = out + (size_t)row * H;
-    for (int i = threadIdx.x; i < H; i += blockDim.x)
-        o[i] = from_f32<TA>(xrow[i] * rstd * (offset_next + load_as_f32(w_next, wn_dtype, i)));
+    TA* o = out + (size_t)blockIdx.x * H;
+    float rstd = 1.0f;
+    if (J.w_next != nullptr) {
+        float ss = 0.f;
+#pragma unroll
+        for (int c = 0; c < CH; ++c)
+            if ((threadIdx.x + c * blockDim.x) * VEC < H) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) ss = fmaf(x[c][e], x[c][e], ss);
+            }
+        ss = block_sum(ss, scratch);
+        rstd = 1.0f / sqrtf(ss / (float)H + J.eps_next);
+    }
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int i = (threadIdx.x + c * blockDim.x) * VEC;
+        if (i < H) {
+            if (J.w_next != nullptr) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) x[c][e] *= rstd * (J.offset_next + load_as_f32(J.w_next, J.wn_dtype, (size_t)(i + e)));
+            }
+            store_vec<VEC>(o + i, x[c]);
+        }
+    }
+}
+
+template <typename TA>
+static int launch_postnorm(float* stream, const void* delta, const Joint& J, void* out, int n_rows, int H, cudaStream_t st) {
+    const bool vec = H % 4 == 0 && ((uintptr_t)stream % 16) == 0 && ((uintptr_t)delta % 16) == 0 && ((uintptr_t)out % 16) == 0;
+    const int pieces = vec ? H / 4 : H;
+    int threads = 64;
+    while (threads < 1024 && threads * 2 < pieces) threads <<= 1;
+    const int ch = (pieces + threads - 1) / threads;
+#define RB_JOINT(VEC_, CH_)                                                                                                     \
+    return rb_launch_pdl(postnorm_add_norm_kernel<TA, VEC_, CH_>, dim3(n_rows), dim3(threads), 0, st, stream, (const TA*)delta, J, \
+                         (TA*)out, H)
+    if (vec && ch <= 2) RB_JOINT(4, 2);
+    if (vec && ch <= 4) RB_JOINT(4, 4);
+    if (!vec && ch <= 4) RB_JOINT(1, 4);
+    if (!vec && ch <= 16) RB_JOINT(1, 16);
+#undef RB_JOINT
+    return (int)cudaErrorInvalidValue;                    // rows beyond 16,384 columns
 }
 
 RB_EXPORT int rb_postnorm_add_norm(float* stream, const void* delta, const void* w_post, int wp_dtype, float eps_post,
                                    float offset_post, const void* w_next, int wn_dtype, float eps_next, float offset_next,
                                    void* out, int act_dtype, int n_rows, int H, cudaStream_t st) {
-    if (n_rows <= 0) return 0;
-    const size_t smem = (size_t)(H + 33) * sizeof(float);
-    if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
-    int threads = 128;
-    while (threads < 1024 && threads * 8 < H) threads <<= 1;
-    if (act_dtype == RB_F32)
-        return rb_launch_pdl(postnorm_add_norm_kernel<float>, dim3(n_rows), dim3(threads), smem, st, stream, (const float*)delta,
-                             w_post, wp_dtype, eps_post, offset_post, w_next, wn_dtype, eps_next, offset_next, (float*)out, H);
-    return rb_launch_pdl(postnorm_add_norm_kernel<bf16>, dim3(n_rows), dim3(threads), smem, st, stream, (const bf16*)delta, w_post,
-                         wp_dtype, eps_post, offset_post, w_next, wn_dtype, eps_next, offset_next, (bf16*)out, H);
+    if (n_rows <= 0 || (delta == nullptr && out == nullptr)) return 0;
+    if (delta != nullptr && w_post == nullptr) return (int)cudaErrorInvalidValue;
+    Joint J;
+    J.w_post = w_post; J.wp_dtype = wp_dtype; J.eps_post = eps_post; J.offset_post = offset_post;
+    J.w_next = w_next; J.wn_dtype = wn_dtype; J.eps_next = eps_next; J.offset_next = offset_next;
+    if (act_dtype == RB_F32) return launch_postnorm<float>(stream, delta, J, out, n_rows, H, st);
+    return launch_postnorm<bf16>(stream, delta, J, out, n_rows, H, st);
 }
 
 // ---------------------------------------------------------------- soft cap of the logits
@@ -427,11 +513,38 @@ __global__ void activation_kernel(const TI* __restrict__ x, long long ldx, TO* _
     }
 }
 
+// bfloat16 rows of whole 16-byte pieces, without a bias: eight elements a thread and step.
+__global__ void activation_bf16x8_kernel(const bf16* __restrict__ x, long long ldx, bf16* __restrict__ out, long long ldo, int op,
+                                         int cols8, unsigned total) {
+    pdl_launch_dependents();
+    pdl_wait();
+    for (unsigned e = blockIdx.x * blockDim.x + threadIdx.x; e < total; e += gridDim.x * blockDim.x) {
+        const unsigned r = e / cols8, c = (e - r * cols8) * 8;
+        const uint4 raw = *reinterpret_cast<const uint4*>(x + (size_t)r * ldx + c);
+        const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+        uint4 v;
+        __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float2 f = __bfloat1622float2(p[j]);
+            o[j] = __floats2bfloat162_rn(rb_activate(op, f.x, nullptr, 0, 0), rb_activate(op, f.y, nullptr, 0, 0));
+        }
+        *reinterpret_cast<uint4*>(out + (size_t)r * ldo + c) = v;
+    }
+}
+
 RB_EXPORT int rb_activation(const void* x, long long ldx, int x_dtype, void* out, long long ldo, int out_dtype, int op,
                             const void* bias, int bias_dtype, int rows, int cols, cudaStream_t st) {
     if (rows <= 0 || cols <= 0) return 0;
     if (op < 0 || op > ACT_NEG_EXP_EXP) return (int)cudaErrorInvalidValue;
     const long long total = (long long)rows * cols;
+    if (x_dtype == RB_BF16 && out_dtype == RB_BF16 && bias == nullptr && cols % 8 == 0 && ldx % 8 == 0 && ldo % 8 == 0 &&
+        ((uintptr_t)x % 16) == 0 && ((uintptr_t)out % 16) == 0 && total / 8 < 0x7fffffffLL) {
+        const unsigned items = (unsigned)(total / 8);
+        const unsigned nblocks = (items + 255) / 256 < 148u * 16u ? (items + 255) / 256 : 148u * 16u;
+        return rb_launch_pdl(activation_bf16x8_kernel, dim3(nblocks), dim3(256), 0, st, (const bf16*)x, ldx, (bf16*)out, ldo, op,
+                             cols / 8, items);
+    }
     const int blocks = (int)((total + 255) / 256 < 8192 ? (total + 255) / 256 : 8192);
     if (x_dtype == RB_F32 && out_dtype == RB_F32)
         return rb_launch_pdl(activation_kernel<float, float>, dim3(blocks), dim3(256), 0, st, (const float*)x, ldx, (float*)out, ldo, op, bias, bias_dtype, rows, cols);
@@ -453,34 +566,6 @@ RB_EXPORT int rb_activation(const void* x, long long ldx, int x_dtype, void* out
 // of its columns in registers, S <= HYPER_MAX_STREAMS.  With `rows` the read kernel takes only the listed rows.
 #define HYPER_MAX_STREAMS 8
 
-// VEC columns a thread and step (4 when H is a multiple of 4: 16-byte loads and stores of the streams; else 1).  Which
-// columns a thread sums depends on H alone, so a row's sum of squares is added in one order whatever the step holds.
-template <int VEC> __device__ __forceinline__ void hyper_load(const float* p, float (&v)[VEC]) {
-    if constexpr (VEC == 4) { const float4 q = *reinterpret_cast<const float4*>(p); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
-    else v[0] = *p;
-}
-template <int VEC> __device__ __forceinline__ void hyper_load(const bf16* p, float (&v)[VEC]) {
-    if constexpr (VEC == 4) {
-        const uint2 q = *reinterpret_cast<const uint2*>(p);
-        const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
-        const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
-        v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
-    } else v[0] = to_f32(*p);
-}
-template <int VEC> __device__ __forceinline__ void hyper_store(float* p, const float (&v)[VEC]) {
-    if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-    else *p = v[0];
-}
-template <int VEC> __device__ __forceinline__ void hyper_store(bf16* p, const float (&v)[VEC]) {
-    if constexpr (VEC == 4) {
-        const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
-        uint2 q;
-        q.x = *reinterpret_cast<const unsigned*>(&lo);
-        q.y = *reinterpret_cast<const unsigned*>(&hi);
-        *reinterpret_cast<uint2*>(p) = q;
-    } else *p = __float2bfloat16_rn(v[0]);
-}
-
 // The normed rows from the sums a row left in shared memory.
 template <typename TA, int VEC>
 __device__ __forceinline__ void hyper_normed_rows(const float* u, float rstd, const void* w, int w_dtype, float offset,
@@ -489,10 +574,11 @@ __device__ __forceinline__ void hyper_normed_rows(const float* u, float rstd, co
         float o[VEC];
 #pragma unroll
         for (int e = 0; e < VEC; ++e) o[e] = u[i + e] * rstd * (offset + load_as_f32(w, w_dtype, (size_t)(i + e)));
-        hyper_store<VEC>(out_row + i, o);
+        store_vec<VEC>(out_row + i, o);
     }
 }
 
+// Which columns a thread sums depends on H alone, so a row's sum of squares is added in one order whatever the step holds.
 template <typename TA, int S, int VEC>
 __global__ void __launch_bounds__(256)
 hyper_read_norm_kernel(const float* __restrict__ streams, const float* __restrict__ a, const int* __restrict__ rows,
@@ -509,7 +595,7 @@ hyper_read_norm_kernel(const float* __restrict__ streams, const float* __restric
     for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {
         float old[S][VEC];
 #pragma unroll
-        for (int s = 0; s < S; ++s) hyper_load<VEC>(x + (size_t)s * H + i, old[s]);
+        for (int s = 0; s < S; ++s) load_vec<VEC>(x + (size_t)s * H + i, old[s]);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
             float u = 0.f;
@@ -547,8 +633,8 @@ hyper_write_kernel(float* __restrict__ streams, const TY* __restrict__ y, const 
     for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {
         float old[S][VEC], yv[VEC], u[VEC];
 #pragma unroll
-        for (int s = 0; s < S; ++s) hyper_load<VEC>(x + (size_t)s * H + i, old[s]);
-        hyper_load<VEC>(y + t * H + i, yv);
+        for (int s = 0; s < S; ++s) load_vec<VEC>(x + (size_t)s * H + i, old[s]);
+        load_vec<VEC>(y + t * H + i, yv);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) u[e] = 0.f;
 #pragma unroll
@@ -561,7 +647,7 @@ hyper_write_kernel(float* __restrict__ streams, const TY* __restrict__ y, const 
                 for (int s = 0; s < S; ++s) v[e] = fmaf(mix[s][r], old[s][e], v[e]);
                 u[e] = fmaf(an[r], v[e], u[e]);
             }
-            hyper_store<VEC>(x + (size_t)r * H + i, v);
+            store_vec<VEC>(x + (size_t)r * H + i, v);
         }
         if (out) {
 #pragma unroll

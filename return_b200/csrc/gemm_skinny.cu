@@ -56,7 +56,8 @@ struct SkinnyFused {
     float offset;
     float* ssq_out;           // residual form: [8, ssq_ld], this CTA writes column blockIdx.x; or null
     int ssq_ld;
-    int act;                  // plain form: 0, or 1 + the number of an activation (rb_activate) applied to every output
+    int act;                  // plain form: 0, or 1 + the number of an activation (rb_activate) applied to every output;
+                              // gated form: the number of its gate (rb_gate_arg)
     const void* act_bias;     // its bias per output column, or null
     int act_bias_dtype;
 };
@@ -67,7 +68,7 @@ struct Regs {                         // one buffer: U blocks of 32 k of the wei
 };
 
 // GATED: the 16 weight rows of a group are 8 gate rows followed by their 8 up rows (the feed-forward's
-// interleaved layout); the epilogue writes silu(gate) * up, 8 values per token, into out[M, N / 2].
+// interleaved layout); the epilogue writes silu(gate) * up (or another gate, F.act), 8 values per token, into out[M, N / 2].
 //
 // Persistent: a CTA walks groups of 16 weight rows (group = blockIdx.x, + gridDim.x, ...).  Each
 // warp owns one slice of K, cut into buffers of U blocks of 32; the buffers of all its groups form
@@ -164,7 +165,7 @@ gemm_skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TOut*
 #pragma unroll
                     for (int wi = 0; wi < SK_WARPS; ++wi) { gate += red[wi][j][m]; up += red[wi][8 + j][m]; }
                     if constexpr (FUSED != 0) { gate *= s_scale[m]; up *= s_scale[m]; }
-                    store_out<TOut>(out + (size_t)m * ldo + (n0 >> 1) + j, gate / (1.0f + expf(-gate)) * up);
+                    store_out<TOut>(out + (size_t)m * ldo + (n0 >> 1) + j, gate / (1.0f + expf(-rb_gate_arg(F.act, gate))) * up);
                 }
             }
         } else {
@@ -252,6 +253,7 @@ int launch(const bf16* x, const bf16* w, void* out, int out_f32, int gated, int 
     if (grid <= 0) return (int)cudaErrorInvalidDevice;
     SkinnyFused none = {};
     none.act = act; none.act_bias = act_bias; none.act_bias_dtype = act_bias_dtype;
+    if (gated) none.act = gated - 1;
     if (gated)
         return rb_launch_pdl(gemm_skinny_kernel<MT, bf16, true, 0>, dim3(grid), dim3(SK_WARPS * 32), 0, st, x, w, (bf16*)out, M, N, K, ldx, ldw, ldo, none);
     if (out_f32)
@@ -267,8 +269,8 @@ RB_EXPORT int rb_gemm_skinny_max_rows() { return 32; }
 // that its residual form writes per token.
 RB_EXPORT int rb_gemm_skinny_ctas(int N) { return grid_for(N); }
 
-// The fused forms, for up to 8 rows, bfloat16 out.  form 0: out[M, N] = rstd * acc (or silu(rstd gate) * (rstd up) into
-// out[M, N / 2] with gated = 1), rstd from ssq_in (null: 1).  form 1 (residual): v = stream[M, N] + rstd * acc goes to the
+// The fused forms, for up to 8 rows, bfloat16 out.  form 0: out[M, N] = rstd * acc (or the gated unit of the scaled sums into
+// out[M, N / 2], gated as in rb_gemm_skinny), rstd from ssq_in (null: 1).  form 1 (residual): v = stream[M, N] + rstd * acc goes to the
 // stream; out[M, N] = v * (offset + norm_w) if norm_w is given; ssq_out[m][cta] = this CTA's share of sum_n v^2.
 RB_EXPORT int rb_gemm_skinny_fused(const void* x, const void* w, void* out, int form, int gated, int M, int N, int K,
                                    int ldx, int ldw, int ldo, const float* ssq_in, int ssq_in_count, int norm_dim, float eps,
@@ -276,7 +278,7 @@ RB_EXPORT int rb_gemm_skinny_fused(const void* x, const void* w, void* out, int 
                                    int ssq_ld, cudaStream_t st) {
     if (M <= 0 || N <= 0) return 0;
     if (M > 8 || K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x % 16) || ((uintptr_t)w % 16)) return (int)cudaErrorInvalidValue;
-    if (gated && (N % 16 || form != 0)) return (int)cudaErrorInvalidValue;
+    if (gated && (N % 16 || form != 0 || gated < 0 || gated - 1 > GATE_GELU_TANH)) return (int)cudaErrorInvalidValue;
     if (form == 1 && (stream == nullptr || (norm_w != nullptr && out == nullptr))) return (int)cudaErrorInvalidValue;
     if (form == 0 && out == nullptr) return (int)cudaErrorInvalidValue;
     const int grid = grid_for(N);
@@ -290,19 +292,20 @@ RB_EXPORT int rb_gemm_skinny_fused(const void* x, const void* w, void* out, int 
     const bf16* wp = (const bf16*)w;
     if (form == 1)
         return rb_launch_pdl(gemm_skinny_kernel<1, bf16, false, 2>, dim3(grid), dim3(SK_WARPS * 32), 0, st, xp, wp, (bf16*)out, M, N, K, ldx, ldw, ldo, F);
+    if (gated) F.act = gated - 1;
     if (gated)
         return rb_launch_pdl(gemm_skinny_kernel<1, bf16, true, 1>, dim3(grid), dim3(SK_WARPS * 32), 0, st, xp, wp, (bf16*)out, M, N, K, ldx, ldw, ldo, F);
     return rb_launch_pdl(gemm_skinny_kernel<1, bf16, false, 1>, dim3(grid), dim3(SK_WARPS * 32), 0, st, xp, wp, (bf16*)out, M, N, K, ldx, ldw, ldo, F);
 }
 
 // gated = 1: w holds gate and up rows interleaved in blocks of 8 (N % 16 == 0) and out is
-// bfloat16 [M, N / 2] = silu(gate) * up.
+// bfloat16 [M, N / 2] = silu(gate) * up; 1 + the number of another gate (GATE_GELU_TANH): gate sigmoid(rb_gate_arg(gate)) * up.
 RB_EXPORT int rb_gemm_skinny(const void* x, const void* w, void* out, int out_f32, int gated, int M, int N, int K,
                              int ldx, int ldw, int ldo, cudaStream_t st) {
     if (M <= 0 || N <= 0) return 0;
     if (M > 32 || K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x % 16) || ((uintptr_t)w % 16))
         return (int)cudaErrorInvalidValue;
-    if (gated && (N % 16 || out_f32)) return (int)cudaErrorInvalidValue;
+    if (gated && (N % 16 || out_f32 || gated < 0 || gated - 1 > GATE_GELU_TANH)) return (int)cudaErrorInvalidValue;
     const bf16* xp = (const bf16*)x;
     const bf16* wp = (const bf16*)w;
     if (M <= 8) return launch<1>(xp, wp, out, out_f32, gated, M, N, K, ldx, ldw, ldo, st);

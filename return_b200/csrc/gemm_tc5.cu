@@ -203,7 +203,7 @@ constexpr int TC5_THREADS = 192;          // warp 0: TMA, warp 1: MMA, warps 2..
 template <int BN, int STAGES, int KPS, typename TOut, bool GATED>
 __global__ void __launch_bounds__(TC5_THREADS)
 tc5_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-                TOut* __restrict__ out, int M, int N, int K, int ldo, int* __restrict__ status) {
+                TOut* __restrict__ out, int M, int N, int K, int ldo, int* __restrict__ status, int gate_act) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     constexpr unsigned A_BYTES = BM * BK * 2, B_BYTES = BN * BK * 2, BLOCK_BYTES = A_BYTES + B_BYTES, STAGE_BYTES = KPS * BLOCK_BYTES;
@@ -303,7 +303,7 @@ tc5_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant
 #pragma unroll
                         for (int j = 0; j < 8; ++j) {
                             const float gate = __uint_as_float(r[b * 16 + j]), up = __uint_as_float(r[b * 16 + 8 + j]);
-                            g[b * 8 + j] = gate / (1.0f + __expf(-gate)) * up;
+                            g[b * 8 + j] = gate / (1.0f + __expf(-rb_gate_arg(gate_act, gate))) * up;
                         }
                     if (valid == 16 && sizeof(TOut) == 2 && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {
 #pragma unroll
@@ -418,7 +418,7 @@ __device__ __forceinline__ void tmem_dealloc_pair(unsigned taddr, unsigned cols)
 template <typename TOut, bool GATED>
 __global__ void __launch_bounds__(TC5_THREADS)
 tc5_gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-                     TOut* __restrict__ out, int M, int N, int K, int ldo, int* __restrict__ status) {
+                     TOut* __restrict__ out, int M, int N, int K, int ldo, int* __restrict__ status, int gate_act) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     __shared__ __align__(8) unsigned long long full_bar[PR_STAGES], empty_bar[PR_STAGES], acc_full[2], acc_empty[2];
@@ -525,7 +525,7 @@ tc5_gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
 #pragma unroll
                         for (int j = 0; j < 8; ++j) {
                             const float gate = __uint_as_float(r[b * 16 + j]), up = __uint_as_float(r[b * 16 + 8 + j]);
-                            g[b * 8 + j] = __fdividef(gate, 1.0f + __expf(-gate)) * up;
+                            g[b * 8 + j] = __fdividef(gate, 1.0f + __expf(-rb_gate_arg(gate_act, gate))) * up;
                         }
                     if (valid == 16 && sizeof(TOut) == 2 && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {
 #pragma unroll
@@ -561,7 +561,7 @@ tc5_gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
 // ------------------------------------------------------------------------------------ host side
 template <int BN, int STAGES, int KPS, typename TOut, bool GATED>
 int launch_tc5(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int ldw, int ldo, int* status,
-               cudaStream_t st) {
+               cudaStream_t st, int gate_act = GATE_SILU) {
     CUtensorMap mx, mw;
     if (!tma::make_map_bf16(&mx, x, M, K, ldx, BM) || !tma::make_map_bf16(&mw, w, N, K, ldw, BN)) return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)STAGES * KPS * (BM + BN) * BK * 2 + 1024;
@@ -575,12 +575,12 @@ int launch_tc5(const void* x, const void* w, void* out, int M, int N, int K, int
     if (num_sms <= 0) return (int)cudaErrorInvalidDevice;
     dim3 grid(tiles < num_sms ? tiles : num_sms);
     return rb_launch_pdl(tc5_gemm_kernel<BN, STAGES, KPS, TOut, GATED>, grid, dim3(TC5_THREADS), smem, st, mx, mw,
-                         (TOut*)out, M, N, K, ldo, status);
+                         (TOut*)out, M, N, K, ldo, status, gate_act);
 }
 
 template <typename TOut, bool GATED>
 int launch_pair(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int ldw, int ldo, int* status,
-                cudaStream_t st) {
+                cudaStream_t st, int gate_act = GATE_SILU) {
     CUtensorMap mx, mw;
     if (!tma::make_map_bf16(&mx, x, M, K, ldx, BM) || !tma::make_map_bf16(&mw, w, N, K, ldw, PR_HALF)) return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)PR_STAGES * PR_STAGE_BYTES + 1024;
@@ -628,20 +628,21 @@ int launch_pair(const void* x, const void* w, void* out, int M, int N, int K, in
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = RB_PDL_MODE == 3 ? 1 : 2;
-    return (int)cudaLaunchKernelEx(&cfg, tc5_gemm_pair_kernel<TOut, GATED>, mx, mw, (TOut*)out, M, N, K, ldo, status);
+    return (int)cudaLaunchKernelEx(&cfg, tc5_gemm_pair_kernel<TOut, GATED>, mx, mw, (TOut*)out, M, N, K, ldo, status, gate_act);
 }
 
 }  // namespace
 
-// out dtype: 0 bfloat16, 1 float32.  gated: SwiGLU epilogue over woven gate/up columns (out is [M, N/2]).
+// out dtype: 0 bfloat16, 1 float32.  gated: the gated unit over woven gate/up columns as the epilogue (out is [M, N/2]): 1 + the
+// number of its gate (GATE_SILU, GATE_GELU_TANH), or 0.
 // status: one int in device memory, set to 1 if a wait inside the kernel gave up (zero it beforehand).
 RB_EXPORT int rb_tc5_gemm(const void* x, const void* w, void* out, int out_f32, int gated, int M, int N, int K,
                           int ldx, int ldw, int ldo, int* status, cudaStream_t st) {
     if (M <= 0 || N <= 0) return 0;
     if (K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x % 16) || ((uintptr_t)w % 16)) return (int)cudaErrorInvalidValue;
     if (gated) {
-        if (out_f32 || N % 16) return (int)cudaErrorInvalidValue;
-        return launch_tc5<256, TC5_STAGES, TC5_KPS, bf16, true>(x, w, out, M, N, K, ldx, ldw, ldo, status, st);
+        if (out_f32 || N % 16 || gated < 0 || gated - 1 > GATE_GELU_TANH) return (int)cudaErrorInvalidValue;
+        return launch_tc5<256, TC5_STAGES, TC5_KPS, bf16, true>(x, w, out, M, N, K, ldx, ldw, ldo, status, st, gated - 1);
     }
     if (out_f32) return launch_tc5<256, TC5_STAGES, TC5_KPS, float, false>(x, w, out, M, N, K, ldx, ldw, ldo, status, st);
     return launch_tc5<256, TC5_STAGES, TC5_KPS, bf16, false>(x, w, out, M, N, K, ldx, ldw, ldo, status, st);
@@ -697,8 +698,8 @@ RB_EXPORT int rb_tc5_gemm_pair(const void* x, const void* w, void* out, int out_
     if (M <= 0 || N <= 0) return 0;
     if (K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x % 16) || ((uintptr_t)w % 16)) return (int)cudaErrorInvalidValue;
     if (gated) {
-        if (out_f32 || N % 16) return (int)cudaErrorInvalidValue;
-        return launch_pair<bf16, true>(x, w, out, M, N, K, ldx, ldw, ldo, status, st);
+        if (out_f32 || N % 16 || gated < 0 || gated - 1 > GATE_GELU_TANH) return (int)cudaErrorInvalidValue;
+        return launch_pair<bf16, true>(x, w, out, M, N, K, ldx, ldw, ldo, status, st, gated - 1);
     }
     if (out_f32) return launch_pair<float, false>(x, w, out, M, N, K, ldx, ldw, ldo, status, st);
     return launch_pair<bf16, false>(x, w, out, M, N, K, ldx, ldw, ldo, status, st);

@@ -114,13 +114,14 @@ RB_EXPORT int rb_moe_route(const float* z, int ldz, const float* bias, int* expe
 }
 
 // ---------------------------------------------------------------- a pair's product, weights streamed
-// out[i, n] = sum_k x[i / in_div, k] * W[expert_of[i]][n, k] for every pair i: the form for few pairs (decoded tokens)
+// out[i, n] = f(sum_k x[i / in_div, k] * W[expert_of[i]][n, k]) for every pair i, f the identity (act < 0) or an activation by
+// its number (rb_activate) on the float32 sum: the form for few pairs (decoded tokens)
 // and the float32 path.  One CTA takes one pair and a run of output rows; a warp an output row at a time, the lanes
 // striding k, so every sum has one order whatever else the step holds.  W: [E, N, K] contiguous.
 template <typename TA, typename TO>
 __global__ void __launch_bounds__(256)
 moe_pair_linear_kernel(const TA* __restrict__ x, int ldx, int in_div, const TA* __restrict__ W, const int* __restrict__ expert_of,
-                       TO* __restrict__ out, int ldo, int N, int K, int rows_per_cta) {
+                       TO* __restrict__ out, int ldo, int N, int K, int rows_per_cta, int act) {
     extern __shared__ float xs[];                         // K floats
     pdl_launch_dependents();
     pdl_wait();
@@ -137,7 +138,7 @@ moe_pair_linear_kernel(const TA* __restrict__ x, int ldx, int in_div, const TA* 
         float acc = 0.f;
         for (int k = lane; k < K; k += 32) acc = fmaf(xs[k], to_f32(wr[k]), acc);
         acc = warp_sum(acc);
-        if (lane == 0) out[(size_t)i * ldo + n] = from_f32<TO>(acc);
+        if (lane == 0) out[(size_t)i * ldo + n] = from_f32<TO>(act < 0 ? acc : rb_activate(act, acc, nullptr, 0, 0));
     }
 }
 
@@ -146,7 +147,7 @@ moe_pair_linear_kernel(const TA* __restrict__ x, int ldx, int in_div, const TA* 
 // float32.  Eight warps share 64 output rows; the sums keep one order (a lane's pieces in turn, then the butterfly).
 __global__ void __launch_bounds__(256)
 moe_pair_linear_vec_kernel(const bf16* __restrict__ x, int ldx, int in_div, const bf16* __restrict__ W,
-                           const int* __restrict__ expert_of, bf16* __restrict__ out, int ldo, int N, int K) {
+                           const int* __restrict__ expert_of, bf16* __restrict__ out, int ldo, int N, int K, int act) {
     extern __shared__ __align__(16) float xs[];           // K floats
     pdl_launch_dependents();
     pdl_wait();
@@ -192,27 +193,28 @@ moe_pair_linear_vec_kernel(const bf16* __restrict__ x, int ldx, int in_div, cons
         for (int j = 0; j < 4; ++j) {
             const float v = warp_sum(acc[j]);
             const int n = n_base + r0 + j;
-            if (lane == 0 && n < N) out[(size_t)i * ldo + n] = __float2bfloat16_rn(v);
+            if (lane == 0 && n < N) out[(size_t)i * ldo + n] = __float2bfloat16_rn(act < 0 ? v : rb_activate(act, v, nullptr, 0, 0));
         }
     }
     pdl_trigger_late();
 }
 
 RB_EXPORT int rb_moe_pair_linear(const void* x, int ldx, int in_div, const void* W, const int* expert_of, void* out, int ldo,
-                                 int act_dtype, int pairs, int N, int K, cudaStream_t st) {
+                                 int act_dtype, int pairs, int N, int K, int act, cudaStream_t st) {
     if (pairs <= 0 || N <= 0) return 0;
+    if (act > ACT_SILU) return (int)cudaErrorInvalidValue;
     const int rows_per_cta = 64;
     dim3 grid(pairs, (N + rows_per_cta - 1) / rows_per_cta);
     const size_t smem = (size_t)K * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     if (act_dtype == RB_BF16 && K % 8 == 0 && ldx % 8 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)W % 16) == 0)
         return rb_launch_pdl(moe_pair_linear_vec_kernel, grid, dim3(256), smem, st, (const bf16*)x, ldx, in_div, (const bf16*)W,
-                             expert_of, (bf16*)out, ldo, N, K);
+                             expert_of, (bf16*)out, ldo, N, K, act);
     if (act_dtype == RB_F32)
         return rb_launch_pdl(moe_pair_linear_kernel<float, float>, grid, dim3(256), smem, st, (const float*)x, ldx, in_div,
-                             (const float*)W, expert_of, (float*)out, ldo, N, K, rows_per_cta);
+                             (const float*)W, expert_of, (float*)out, ldo, N, K, rows_per_cta, act);
     return rb_launch_pdl(moe_pair_linear_kernel<bf16, bf16>, grid, dim3(256), smem, st, (const bf16*)x, ldx, in_div,
-                         (const bf16*)W, expert_of, (bf16*)out, ldo, N, K, rows_per_cta);
+                         (const bf16*)W, expert_of, (bf16*)out, ldo, N, K, rows_per_cta, act);
 }
 
 // ---------------------------------------------------------------- the gated unit with a capped gate
@@ -282,14 +284,16 @@ RB_EXPORT int rb_clamped_glu(const void* in, int ldi, void* out, int ldo, int ac
 }
 
 // ---------------------------------------------------------------- the weighted sum of a token's experts
-// out[t, :] = sum_k weight[t, k] * y[row_of ? row_of[t * top + k] : t * top + k, :]  (+ shared[t, :]), k ascending, float32
-// sums.  row_of: where a pair's row lies when the pairs were put in the order of their experts.  weight null: a plain sum.
+// out[t, :] = sum_k weight[t, k] * y[row_of ? row_of[t * top + k] : t * top + k, :]  (+ c shared[t, :]), k ascending, float32
+// sums; c = 1, or the logistic of shared_gate[t * gate_ld] (float32) if that is given.  row_of: where a pair's row lies when the pairs were put in the order of their experts.  weight null: a plain sum.
 template <typename TA>
 __global__ void moe_combine_kernel(const TA* __restrict__ y, const int* __restrict__ row_of, const float* __restrict__ weight,
-                                   const TA* __restrict__ shared, TA* __restrict__ out, int H, int top) {
+                                   const TA* __restrict__ shared, const float* __restrict__ shared_gate, int gate_ld,
+                                   TA* __restrict__ out, int H, int top) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
+    const float c = shared_gate ? 1.0f / (1.0f + expf(-shared_gate[(size_t)t * gate_ld])) : 1.0f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {
@@ -297,20 +301,59 @@ __global__ void moe_combine_kernel(const TA* __restrict__ y, const int* __restri
             const size_t row = row_of ? (size_t)row_of[pair] : (size_t)pair;
             acc = fmaf(weight ? weight[pair] : 1.f, to_f32(y[row * H + i]), acc);
         }
-        if (shared != nullptr) acc += to_f32(shared[(size_t)t * H + i]);
+        if (shared != nullptr) acc = fmaf(c, to_f32(shared[(size_t)t * H + i]), acc);
         out[(size_t)t * H + i] = from_f32<TA>(acc);
     }
 }
 
-RB_EXPORT int rb_moe_combine(const void* y, const int* row_of, const float* weight, const void* shared, void* out,
-                             int act_dtype, int T, int H, int top, cudaStream_t st) {
+// The bfloat16 form for rows of whole 16-byte pieces: eight columns a thread, the sums in the same order.
+__global__ void moe_combine_vec_kernel(const bf16* __restrict__ y, const int* __restrict__ row_of, const float* __restrict__ weight,
+                                       const bf16* __restrict__ shared, const float* __restrict__ shared_gate, int gate_ld,
+                                       bf16* __restrict__ out, int H, int top) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const float c = shared_gate ? 1.0f / (1.0f + expf(-shared_gate[(size_t)t * gate_ld])) : 1.0f;
+    for (int i = threadIdx.x * 8; i < H; i += blockDim.x * 8) {
+        float acc[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[j] = 0.f;
+        auto add = [&](const bf16* row, float f) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(row + i);
+            const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float2 v = __bfloat1622float2(p[j]);
+                acc[2 * j] = fmaf(f, v.x, acc[2 * j]);
+                acc[2 * j + 1] = fmaf(f, v.y, acc[2 * j + 1]);
+            }
+        };
+#pragma unroll 4
+        for (int k = 0; k < top; ++k) {
+            const int pair = t * top + k;
+            add(y + (row_of ? (size_t)row_of[pair] : (size_t)pair) * H, weight ? weight[pair] : 1.f);
+        }
+        if (shared != nullptr) add(shared + (size_t)t * H, c);
+        uint4 v;
+        __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[j] = __floats2bfloat162_rn(acc[2 * j], acc[2 * j + 1]);
+        *reinterpret_cast<uint4*>(out + (size_t)t * H + i) = v;
+    }
+}
+
+RB_EXPORT int rb_moe_combine(const void* y, const int* row_of, const float* weight, const void* shared, const float* shared_gate,
+                             int gate_ld, void* out, int act_dtype, int T, int H, int top, cudaStream_t st) {
     if (T <= 0) return 0;
+    if (act_dtype == RB_BF16 && H % 8 == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)shared % 16) == 0 && ((uintptr_t)out % 16) == 0)
+        return rb_launch_pdl(moe_combine_vec_kernel, dim3(T), dim3(H >= 2048 ? 256 : H >= 1024 ? 128 : 64), 0, st, (const bf16*)y,
+                             row_of, weight, (const bf16*)shared, shared_gate, gate_ld, (bf16*)out, H, top);
     const int threads = H >= 1024 ? 256 : 128;
     if (act_dtype == RB_F32)
         return rb_launch_pdl(moe_combine_kernel<float>, dim3(T), dim3(threads), 0, st, (const float*)y, row_of, weight,
-                             (const float*)shared, (float*)out, H, top);
+                             (const float*)shared, shared_gate, gate_ld, (float*)out, H, top);
     return rb_launch_pdl(moe_combine_kernel<bf16>, dim3(T), dim3(threads), 0, st, (const bf16*)y, row_of, weight,
-                         (const bf16*)shared, (bf16*)out, H, top);
+                         (const bf16*)shared, shared_gate, gate_ld, (bf16*)out, H, top);
 }
 
 // ---------------------------------------------------------------- the pairs in the order of their experts
@@ -354,7 +397,7 @@ RB_EXPORT int rb_moe_sort(const int* expert_of, int pairs, int E, int* offsets, 
 }
 
 // ---------------------------------------------------------------- the experts' products on the tensor cores
-// C[place, n] = sum_k A[row(place), k] * W[e][n, k] for every place of expert e's run, bfloat16 in, float32
+// C[place, n] = f(sum_k A[row(place), k] * W[e][n, k]) (f as for the pairs' products above) for every place of expert e's run, bfloat16 in, float32
 // accumulation (mma.sync m16n8k16), bfloat16 out.  row(place) = pair_at[place] / in_div when pair_at is given (the
 // first product reads the tokens' rows where they lie), else the place itself (the second reads what the first left).
 // A CTA owns a tile of 64 places of one expert x 128 output columns; it finds its expert by walking the offsets,
@@ -386,7 +429,7 @@ __device__ __forceinline__ void gg_mma(float (&c)[4], const unsigned (&a)[4], un
 __global__ void __launch_bounds__(256)
 moe_grouped_gemm_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__ pair_at, int in_div,
                         const bf16* __restrict__ W, const int* __restrict__ offsets, int E, bf16* __restrict__ C, int ldc,
-                        int N, int K) {
+                        int N, int K, int act) {
     __shared__ __align__(16) bf16 sA[GG_STAGES][GG_BM * GG_LD];
     __shared__ __align__(16) bf16 sB[GG_STAGES][GG_BN * GG_LD];
     __shared__ int s_tile[3];                             // expert, first place of the tile, places in it
@@ -473,19 +516,22 @@ moe_grouped_gemm_kernel(const bf16* __restrict__ A, int lda, const int* __restri
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int n = n0 + wn + j * 8 + 2 * t4;
-                if (n < N) crow[n] = __float2bfloat16_rn(acc[i][j][half * 2]);
-                if (n + 1 < N) crow[n + 1] = __float2bfloat16_rn(acc[i][j][half * 2 + 1]);
+                float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
+                if (act >= 0) { v0 = rb_activate(act, v0, nullptr, 0, 0); v1 = rb_activate(act, v1, nullptr, 0, 0); }
+                if (n < N) crow[n] = __float2bfloat16_rn(v0);
+                if (n + 1 < N) crow[n + 1] = __float2bfloat16_rn(v1);
             }
         }
 }
 
 RB_EXPORT int rb_moe_grouped_gemm(const void* A, int lda, const int* pair_at, int in_div, const void* W, const int* offsets,
-                                  int E, void* C, int ldc, int places, int N, int K, cudaStream_t st) {
+                                  int E, void* C, int ldc, int places, int N, int K, int act, cudaStream_t st) {
     if (places <= 0 || N <= 0) return 0;
+    if (act > ACT_SILU) return (int)cudaErrorInvalidValue;
     if (K % 8 || lda % 8 || ((uintptr_t)A % 16) || ((uintptr_t)W % 16)) return (int)cudaErrorInvalidValue;
     dim3 grid((places + GG_BM - 1) / GG_BM + E, (N + GG_BN - 1) / GG_BN);
     return rb_launch_pdl(moe_grouped_gemm_kernel, grid, dim3(256), 0, st, (const bf16*)A, lda, pair_at, in_div, (const bf16*)W,
-                         offsets, E, (bf16*)C, ldc, N, K);
+                         offsets, E, (bf16*)C, ldc, N, K, act);
 }
 
 // ---------------------------------------------------------------- the tokens' rows in the order of the places

@@ -76,7 +76,7 @@ __device__ __forceinline__ void store_chunk(bf16* dst, const unsigned (&r)[32], 
 __global__ void __launch_bounds__(THREADS)
 moe_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                const int* __restrict__ offsets, int E, bf16* __restrict__ out, int N, int K, int ldo,
-               int* __restrict__ status) {
+               int* __restrict__ status, int act) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     constexpr unsigned A_BYTES = BM * BK * 2, B_BYTES = BN * BK * 2, STAGE_BYTES = A_BYTES + B_BYTES;
@@ -170,6 +170,10 @@ moe_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 tmem_ld32(tacc + ((unsigned)(q * 32) << 16) + buf * BN + c0, r);
                 tmem_ld_wait();
                 if (r_local >= t.rows || t.n0 + c0 >= N) continue;
+                if (act >= 0) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(rb_activate(act, __uint_as_float(r[j]), nullptr, 0, 0));
+                }
                 store_chunk(out + (size_t)(t.m0 + r_local) * ldo + t.n0 + c0, r, min(32, N - t.n0 - c0));
             }
             fence_before_sync();
@@ -186,10 +190,11 @@ moe_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 }  // namespace
 
 // A [places, K] (the pairs' rows in the order of their experts), W [E, N, K] contiguous, offsets int32 [E + 1] on the
-// device, out [places, N] bfloat16.  status: one int in device memory, set to 1 if a wait inside the kernel gave up.
+// device, out [places, N] bfloat16; act: -1, or the number of an activation (rb_activate) on the float32 sums.  status: one int in device memory, set to 1 if a wait inside the kernel gave up.
 RB_EXPORT int rb_moe_tc5_gemm(const void* A, int lda, const void* W, const int* offsets, int E, void* out, int ldo, int places,
-                              int N, int K, int* status, cudaStream_t st) {
+                              int N, int K, int act, int* status, cudaStream_t st) {
     if (places <= 0 || N <= 0) return 0;
+    if (act > ACT_SILU) return (int)cudaErrorInvalidValue;
     if (E > MAX_EXPERTS || K % 8 || lda % 8 || ((uintptr_t)A % 16) || ((uintptr_t)W % 16)) return (int)cudaErrorInvalidValue;
     if ((long long)E * N > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
     CUtensorMap ma, mw;
@@ -204,5 +209,5 @@ RB_EXPORT int rb_moe_tc5_gemm(const void* A, int lda, const void* W, const int* 
     const int num_sms = rb_num_sms();
     if (num_sms <= 0) return (int)cudaErrorInvalidDevice;
     dim3 grid((unsigned)(worst < num_sms ? worst : num_sms));
-    return rb_launch_pdl(moe_tc5_kernel, grid, dim3(THREADS), smem, st, ma, mw, offsets, E, (bf16*)out, N, K, ldo, status);
+    return rb_launch_pdl(moe_tc5_kernel, grid, dim3(THREADS), smem, st, ma, mw, offsets, E, (bf16*)out, N, K, ldo, status, act);
 }

@@ -12,6 +12,10 @@
 // its position, so the key is rotated once, before the write.  Norm and rotation are float32,
 // with one rounding at the store.
 //
+// Options.  `norm_n`: how many elements of a head the norm's mean runs over, where heads are padded with zeros to D (0: D).
+// `ValueMix`: the values that are cached are blended with those of an earlier layer of the same token,
+// v <- (1 - share) v + share v_first, in float32 before the store.
+//
 // Cache layout of one layer: [num_pages, Hkv, P, D]; the page of a token is
 // block_table[segment][pos / P], its row in the page pos % P.
 #include "common.cuh"
@@ -31,6 +35,15 @@ template <> struct Pair<bf16> {
     }
 };
 
+// The value blend.  first: [T, ld] row-major, kv head g's values from column g * head_stride, n of them (what lies behind is
+// zero in both); share: one number, of type share_dtype.
+struct ValueMix {
+    const void* first;         // null: values are cached as they are
+    int ld, head_stride, n;
+    const void* share;
+    int share_dtype;
+};
+
 // One warp per token and HPW neighbouring heads; a lane holds the element pairs (i, i+1) of the first
 // rotary half and their partners (i + R/2, i + R/2 + 1) in registers, so a head is read once; head sizes
 // up to 256.  The loads of all of a warp's heads go out before the first is used: a head is only 256
@@ -45,7 +58,7 @@ __global__ void qk_norm_rope_write_kernel(
         const int* __restrict__ pos, const int* __restrict__ tok_seg,
         const int* __restrict__ block_table, int bt_stride, int page_size,
         TA* __restrict__ kpool, TA* __restrict__ vpool,
-        int Hq, int Hkv, int D, int write_kv) {
+        int Hq, int Hkv, int D, int write_kv, int norm_n, const ValueMix vm) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -106,6 +119,22 @@ __global__ void qk_norm_rope_write_kernel(
         if (hh >= Hq + Hkv) {                       // v head: copy
             if (slot_base < 0) continue;
             TA* dst = vpool + slot_base + (long long)(hh - Hq - Hkv) * page_size * D;
+            if (vm.first != nullptr) {
+                const TA* vf = (const TA*)vm.first + (size_t)t * vm.ld + (size_t)(hh - Hq - Hkv) * vm.head_stride;
+                const float share = load_as_f32(vm.share, vm.share_dtype, 0), own = 1.0f - share;
+#pragma unroll
+                for (int j = 0; j < ROPE_MAX_J; ++j) {
+                    const int i = 2 * lane + 64 * j;
+                    if (i < D) {
+                        const float f0 = i < vm.n ? to_f32(vf[i]) : 0.f, f1 = i + 1 < vm.n ? to_f32(vf[i + 1]) : 0.f;
+                        a[u][j] = make_float2(own * a[u][j].x + share * f0, own * a[u][j].y + share * f1);
+                    }
+                    if (i + 128 < D) {
+                        const float f0 = i + 128 < vm.n ? to_f32(vf[i + 128]) : 0.f, f1 = i + 129 < vm.n ? to_f32(vf[i + 129]) : 0.f;
+                        b[u][j] = make_float2(own * b[u][j].x + share * f0, own * b[u][j].y + share * f1);
+                    }
+                }
+            }
 #pragma unroll
             for (int j = 0; j < ROPE_MAX_J; ++j) {
                 const int i = 2 * lane + 64 * j;
@@ -134,7 +163,7 @@ __global__ void qk_norm_rope_write_kernel(
         float rstd = 1.f;
         if (w) {
             ss = warp_sum(ss);
-            rstd = 1.0f / sqrtf(ss / (float)D + eps);
+            rstd = 1.0f / sqrtf(ss / (float)norm_n + eps);
         }
 #pragma unroll
         for (int j = 0; j < ROPE_MAX_J; ++j) {
@@ -158,10 +187,11 @@ __global__ void qk_norm_rope_write_kernel(
     }
 }
 
-// The same for many tokens of bfloat16 with head sizes 64, 128 or 256 rotated over their whole width, in
-// 16-byte pieces: LPH = D / 16 lanes share a head, each holding 8 neighbouring elements of the first half and
-// their partners in the second, so a warp works on 32 / LPH heads at once, twice over (ROUNDS), and a head is
-// two 16-byte loads and two 16-byte stores a lane.  A warp takes one (token, group of heads) item.
+// The same for many tokens of bfloat16 with head sizes 32, 64, 128 or 256 and a rotary width that is a multiple of 16, in
+// 16-byte pieces: LPH = D / 16 lanes share a head.  The first rot / 16 of them hold piece c of the first rotary half and
+// its partner in the second; each of the others holds two neighbouring pieces of what is not rotated (their cosine is one).
+// So a warp works on 32 / LPH heads at once, twice over (ROUNDS), and a head is two 16-byte loads and two 16-byte
+// stores a lane.  A warp takes one (token, group of heads) item.
 constexpr int ROPE_VEC_ROUNDS = 2;
 
 __device__ __forceinline__ void unpack8(const uint4& v, float (&f)[8]) {
@@ -186,12 +216,12 @@ __global__ void __launch_bounds__(128)
 qk_norm_rope_write_vec_kernel(
         bf16* __restrict__ qkv, int ld,
         const void* __restrict__ qw, const void* __restrict__ kw, int w_dtype, float eps, float offset,
-        const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+        const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot_dim,
         const int* __restrict__ pos, const int* __restrict__ tok_seg,
         const int* __restrict__ block_table, int bt_stride, int page_size,
         bf16* __restrict__ kpool, bf16* __restrict__ vpool,
-        int T, int Hq, int Hkv, int write_kv, int groups_per_token) {
-    constexpr int D = LPH * 16, HALF = D / 2, HEADS_AT_ONCE = 32 / LPH, HEADS_PER_WARP = HEADS_AT_ONCE * ROPE_VEC_ROUNDS;
+        int T, int Hq, int Hkv, int write_kv, int groups_per_token, int norm_n, const ValueMix vm) {
+    constexpr int D = LPH * 16, HEADS_AT_ONCE = 32 / LPH, HEADS_PER_WARP = HEADS_AT_ONCE * ROPE_VEC_ROUNDS;
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -199,6 +229,9 @@ qk_norm_rope_write_vec_kernel(
     const int t = (int)(item / groups_per_token), hg = (int)(item % groups_per_token);
     if (t >= T) return;
     const int sub = lane % LPH, hsel = lane / LPH;
+    const int half = rot_dim >> 1;
+    const bool turns = 8 * sub < half;                        // this lane's two pieces are rotated against each other
+    const int i1 = turns ? 8 * sub : rot_dim + 16 * (sub - (half >> 3)), i2 = turns ? i1 + half : i1 + 8;
     const int n_heads = write_kv ? Hq + 2 * Hkv : Hq + Hkv;
     const int p = pos[t];
     long long slot_base = -1;     // element offset of (page, kv head 0, row) in a pool
@@ -212,15 +245,17 @@ qk_norm_rope_write_vec_kernel(
     for (int r = 0; r < ROPE_VEC_ROUNDS; ++r) {
         const int hh = hg * HEADS_PER_WARP + r * HEADS_AT_ONCE + hsel;
         if (hh < n_heads) {
-            const bf16* x = row + (size_t)hh * D + 8 * sub;
-            a[r] = *reinterpret_cast<const uint4*>(x);
-            b[r] = *reinterpret_cast<const uint4*>(x + HALF);
+            const bf16* x = row + (size_t)hh * D;
+            a[r] = *reinterpret_cast<const uint4*>(x + i1);
+            b[r] = *reinterpret_cast<const uint4*>(x + i2);
         }
     }
     float c[8], sn[8];
-    {
-        const float4* cp = reinterpret_cast<const float4*>(cos_t + (size_t)p * HALF + 8 * sub);
-        const float4* sp = reinterpret_cast<const float4*>(sin_t + (size_t)p * HALF + 8 * sub);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) { c[i] = 1.f; sn[i] = 0.f; }
+    if (turns) {
+        const float4* cp = reinterpret_cast<const float4*>(cos_t + (size_t)p * half + 8 * sub);
+        const float4* sp = reinterpret_cast<const float4*>(sin_t + (size_t)p * half + 8 * sub);
         const float4 c0 = cp[0], c1 = cp[1], s0 = sp[0], s1 = sp[1];
         c[0] = c0.x; c[1] = c0.y; c[2] = c0.z; c[3] = c0.w; c[4] = c1.x; c[5] = c1.y; c[6] = c1.z; c[7] = c1.w;
         sn[0] = s0.x; sn[1] = s0.y; sn[2] = s0.z; sn[3] = s0.w; sn[4] = s1.x; sn[5] = s1.y; sn[6] = s1.z; sn[7] = s1.w;
@@ -244,9 +279,28 @@ qk_norm_rope_write_vec_kernel(
         if (!live) continue;
         if (is_v) {
             if (slot_base < 0) continue;
-            bf16* dst = vpool + slot_base + (long long)(hh - Hq - Hkv) * page_size * D + 8 * sub;
-            *reinterpret_cast<uint4*>(dst) = a[r];
-            *reinterpret_cast<uint4*>(dst + HALF) = b[r];
+            bf16* dst = vpool + slot_base + (long long)(hh - Hq - Hkv) * page_size * D;
+            if (vm.first != nullptr) {
+                const bf16* vf = (const bf16*)vm.first + (size_t)t * vm.ld + (size_t)(hh - Hq - Hkv) * vm.head_stride;
+                const float share = load_as_f32(vm.share, vm.share_dtype, 0), own = 1.0f - share;
+                float f1[8], f2[8];
+                if (i1 + 8 <= vm.n) unpack8(*reinterpret_cast<const uint4*>(vf + i1), f1);
+                else {
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) f1[i] = i1 + i < vm.n ? __bfloat162float(vf[i1 + i]) : 0.f;
+                }
+                if (i2 + 8 <= vm.n) unpack8(*reinterpret_cast<const uint4*>(vf + i2), f2);
+                else {
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) f2[i] = i2 + i < vm.n ? __bfloat162float(vf[i2 + i]) : 0.f;
+                }
+#pragma unroll
+                for (int i = 0; i < 8; ++i) { x1[i] = own * x1[i] + share * f1[i]; x2[i] = own * x2[i] + share * f2[i]; }
+                a[r] = pack8(x1);
+                b[r] = pack8(x2);
+            }
+            *reinterpret_cast<uint4*>(dst + i1) = a[r];
+            *reinterpret_cast<uint4*>(dst + i2) = b[r];
             continue;
         }
         const void* w = is_k ? kw : qw;
@@ -256,11 +310,11 @@ qk_norm_rope_write_vec_kernel(
             dst = kpool + slot_base + (long long)(hh - Hq) * page_size * D;
         }
         if (w) {
-            const float rstd = 1.0f / sqrtf(ss / (float)D + eps);
+            const float rstd = 1.0f / sqrtf(ss / (float)norm_n + eps);
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
-                x1[i] = x1[i] * rstd * (offset + load_as_f32(w, w_dtype, 8 * sub + i));        // (x * rstd) * w, as the other form
-                x2[i] = x2[i] * rstd * (offset + load_as_f32(w, w_dtype, HALF + 8 * sub + i));
+                x1[i] = x1[i] * rstd * (offset + load_as_f32(w, w_dtype, i1 + i));        // (x * rstd) * w, as the other form
+                x2[i] = x2[i] * rstd * (offset + load_as_f32(w, w_dtype, i2 + i));
             }
         }
         float o1[8], o2[8];
@@ -269,48 +323,59 @@ qk_norm_rope_write_vec_kernel(
             o1[i] = x1[i] * c[i] - x2[i] * sn[i];
             o2[i] = x2[i] * c[i] + x1[i] * sn[i];
         }
-        *reinterpret_cast<uint4*>(dst + 8 * sub) = pack8(o1);
-        *reinterpret_cast<uint4*>(dst + HALF + 8 * sub) = pack8(o2);
+        *reinterpret_cast<uint4*>(dst + i1) = pack8(o1);
+        *reinterpret_cast<uint4*>(dst + i2) = pack8(o2);
     }
 }
 
 template <int LPH>
 static int launch_rope_vec(void* qkv, int ld, const void* qw, const void* kw, int w_dtype, float eps, float offset,
-                           const float* cos_t, const float* sin_t, const int* pos, const int* tok_seg,
+                           const float* cos_t, const float* sin_t, int rot_dim, const int* pos, const int* tok_seg,
                            const int* block_table, int bt_stride, int page_size, void* kpool, void* vpool,
-                           int T, int Hq, int Hkv, int write_kv, cudaStream_t st) {
+                           int T, int Hq, int Hkv, int write_kv, int norm_n, const ValueMix& vm, cudaStream_t st) {
     const int heads = write_kv ? Hq + 2 * Hkv : Hq + Hkv;
     const int per_warp = (32 / LPH) * ROPE_VEC_ROUNDS;
     const int groups = (heads + per_warp - 1) / per_warp;
     const long long items = (long long)T * groups;
     const dim3 grid((unsigned)((items + 3) / 4));
     return rb_launch_pdl(qk_norm_rope_write_vec_kernel<LPH>, grid, dim3(128), 0, st,
-        (bf16*)qkv, ld, qw, kw, w_dtype, eps, offset, cos_t, sin_t, pos, tok_seg, block_table, bt_stride, page_size,
-        (bf16*)kpool, (bf16*)vpool, T, Hq, Hkv, write_kv, groups);
+        (bf16*)qkv, ld, qw, kw, w_dtype, eps, offset, cos_t, sin_t, rot_dim, pos, tok_seg, block_table, bt_stride,
+        page_size, (bf16*)kpool, (bf16*)vpool, T, Hq, Hkv, write_kv, groups, norm_n, vm);
 }
 
+// norm_n: elements of a head that the norm's mean runs over (0: D).  v_first (null: no blend) [T, v_first_ld] with kv head
+// g's values from column g * v_first_head_stride, v_first_n of them, in the activation dtype; v_share: one number.
 RB_EXPORT int rb_qk_norm_rope_write(
         void* qkv, int ld, const void* qw, const void* kw, int w_dtype, float eps, float offset,
         const float* cos_t, const float* sin_t, int rot_dim,
         const int* pos, const int* tok_seg, const int* block_table, int bt_stride, int page_size,
-        void* kpool, void* vpool, int act_dtype, int T, int Hq, int Hkv, int D, int write_kv,
+        void* kpool, void* vpool, int act_dtype, int T, int Hq, int Hkv, int D, int write_kv, int norm_n,
+        const void* v_first, int v_first_ld, int v_first_head_stride, int v_first_n, const void* v_share, int v_share_dtype,
         cudaStream_t st) {
     if (T <= 0) return 0;
     // pairs of neighbours: the rotary half must be even, and a lane holds at most ROPE_MAX_J pairs of pairs
     if (rot_dim > D || (rot_dim & 3) || (D & 1) || rot_dim > 128 * ROPE_MAX_J) return (int)cudaErrorInvalidValue;
+    if (norm_n < 0 || norm_n > D || (v_first != nullptr && v_share == nullptr)) return (int)cudaErrorInvalidValue;
+    if (norm_n == 0) norm_n = D;
+    ValueMix vm;
+    vm.first = v_first; vm.ld = v_first_ld; vm.head_stride = v_first_head_stride; vm.n = v_first_n;
+    vm.share = v_share; vm.share_dtype = v_share_dtype;
     const int threads = 128;
     const int heads = write_kv ? Hq + 2 * Hkv : Hq + Hkv;
     // many tokens: four heads a warp, so that enough bytes are in flight; few tokens: one head a warp, so that
     // the few warps there are spread over the SMs
-    const bool aligned = ld % 8 == 0 && ((uintptr_t)qkv % 16) == 0 && ((uintptr_t)kpool % 16) == 0 && ((uintptr_t)vpool % 16) == 0;
-    if ((long long)T * heads >= 8192 && act_dtype != RB_F32 && rot_dim == D && aligned && (D == 64 || D == 128 || D == 256)) {
-        // many tokens of bfloat16 with a whole-head rotation: 16-byte pieces
-        if (D == 64) return launch_rope_vec<4>(qkv, ld, qw, kw, w_dtype, eps, offset, cos_t, sin_t, pos, tok_seg, block_table,
-                                               bt_stride, page_size, kpool, vpool, T, Hq, Hkv, write_kv, st);
-        if (D == 128) return launch_rope_vec<8>(qkv, ld, qw, kw, w_dtype, eps, offset, cos_t, sin_t, pos, tok_seg, block_table,
-                                                bt_stride, page_size, kpool, vpool, T, Hq, Hkv, write_kv, st);
-        return launch_rope_vec<16>(qkv, ld, qw, kw, w_dtype, eps, offset, cos_t, sin_t, pos, tok_seg, block_table,
-                                   bt_stride, page_size, kpool, vpool, T, Hq, Hkv, write_kv, st);
+    const bool aligned = ld % 8 == 0 && ((uintptr_t)qkv % 16) == 0 && ((uintptr_t)kpool % 16) == 0 && ((uintptr_t)vpool % 16) == 0 &&
+                         (v_first == nullptr || (v_first_ld % 8 == 0 && v_first_head_stride % 8 == 0 && ((uintptr_t)v_first % 16) == 0));
+    if ((long long)T * heads >= 8192 && act_dtype != RB_F32 && rot_dim % 16 == 0 && aligned) {
+        // many tokens of bfloat16: 16-byte pieces
+#define RB_ROPE_VEC(LPH_)                                                                                                       \
+        return launch_rope_vec<LPH_>(qkv, ld, qw, kw, w_dtype, eps, offset, cos_t, sin_t, rot_dim, pos, tok_seg, block_table,   \
+                                     bt_stride, page_size, kpool, vpool, T, Hq, Hkv, write_kv, norm_n, vm, st)
+        if (D == 32) RB_ROPE_VEC(2);
+        if (D == 64) RB_ROPE_VEC(4);
+        if (D == 128) RB_ROPE_VEC(8);
+        if (D == 256) RB_ROPE_VEC(16);
+#undef RB_ROPE_VEC
     }
     if ((long long)T * heads >= 8192) {
         constexpr int HPW = 4;
@@ -318,17 +383,17 @@ RB_EXPORT int rb_qk_norm_rope_write(
         if (act_dtype == RB_F32)
             return rb_launch_pdl(qk_norm_rope_write_kernel<float, HPW>, grid, dim3(threads), 0, st,
                 (float*)qkv, ld, qw, kw, w_dtype, eps, offset, cos_t, sin_t, rot_dim, pos, tok_seg,
-                block_table, bt_stride, page_size, (float*)kpool, (float*)vpool, Hq, Hkv, D, write_kv);
+                block_table, bt_stride, page_size, (float*)kpool, (float*)vpool, Hq, Hkv, D, write_kv, norm_n, vm);
         return rb_launch_pdl(qk_norm_rope_write_kernel<bf16, HPW>, grid, dim3(threads), 0, st,
                 (bf16*)qkv, ld, qw, kw, w_dtype, eps, offset, cos_t, sin_t, rot_dim, pos, tok_seg,
-                block_table, bt_stride, page_size, (bf16*)kpool, (bf16*)vpool, Hq, Hkv, D, write_kv);
+                block_table, bt_stride, page_size, (bf16*)kpool, (bf16*)vpool, Hq, Hkv, D, write_kv, norm_n, vm);
     }
     const dim3 grid(T, (heads + 3) / 4);
     if (act_dtype == RB_F32)
         return rb_launch_pdl(qk_norm_rope_write_kernel<float, 1>, grid, dim3(threads), 0, st,
             (float*)qkv, ld, qw, kw, w_dtype, eps, offset, cos_t, sin_t, rot_dim, pos, tok_seg,
-            block_table, bt_stride, page_size, (float*)kpool, (float*)vpool, Hq, Hkv, D, write_kv);
+            block_table, bt_stride, page_size, (float*)kpool, (float*)vpool, Hq, Hkv, D, write_kv, norm_n, vm);
     return rb_launch_pdl(qk_norm_rope_write_kernel<bf16, 1>, grid, dim3(threads), 0, st,
             (bf16*)qkv, ld, qw, kw, w_dtype, eps, offset, cos_t, sin_t, rot_dim, pos, tok_seg,
-            block_table, bt_stride, page_size, (bf16*)kpool, (bf16*)vpool, Hq, Hkv, D, write_kv);
+            block_table, bt_stride, page_size, (bf16*)kpool, (bf16*)vpool, Hq, Hkv, D, write_kv, norm_n, vm);
 }

@@ -88,7 +88,7 @@ def core() -> ctypes.CDLL:
         lib.rb_rmsnorm_rows.argtypes = [P, P, I, F, F, P, I, I, I, P]
         lib.rb_rmsnorm_rows_ld.argtypes = [P, I, P, I, F, F, P, I, I, I, I, P]
         lib.rb_rmsnorm_rows_ld.restype = c_int
-        lib.rb_swiglu.argtypes = [P, P, I, I, I, I, P]
+        lib.rb_swiglu.argtypes = [P, P, I, I, I, I, I, P]
         lib.rb_gemm_f32.argtypes = [P, P, P, I, I, I, I, I, I, P]
         lib.rb_gemm_skinny.argtypes = [P, P, P, I, I, I, I, I, I, I, I, P]
         lib.rb_gemm_skinny.restype = c_int
@@ -98,9 +98,9 @@ def core() -> ctypes.CDLL:
         lib.rb_gemm_skinny_fused.restype = c_int
         lib.rb_gemm_skinny_ctas.argtypes = [I]
         lib.rb_gemm_skinny_ctas.restype = c_int
-        lib.rb_qk_norm_rope_write.argtypes = [P, I, P, P, I, F, F, P, P, I, P, P, P, I, I, P, P, I, I, I, I, I, I, P]
+        lib.rb_qk_norm_rope_write.argtypes = [P, I, P, P, I, F, F, P, P, I, P, P, P, I, I, P, P, I, I, I, I, I, I, I, P, I, I, I, P, I, P]
         lib.rb_attention_simt.argtypes = [P, I, P, P, P, P, P, I, I, P, I, I, I, I, I, F, I, P]
-        lib.rb_attention_simt_mod.argtypes = [P, I, P, P, P, P, P, I, I, P, I, I, I, I, I, F, I, I, F, P, P, P, I, P]
+        lib.rb_attention_simt_mod.argtypes = [P, I, P, P, P, P, P, I, I, P, I, I, I, I, I, F, I, I, F, P, P, P, I, I, P]
         lib.rb_attn_prep.argtypes = [P, I, I, I, I, P, P, P, I, P, P, I, F, P, P, I, P, P, P, I, I, P, P, P, I, I, I, I, I, I, I, I, P]
         lib.rb_attn_gate.argtypes = [P, P, I, I, I, I, I, I, I, I, P]
         lib.rb_embedding_pair.argtypes = [P, P, I, P, P, P, P, P, P, P, I, I, I, F, I, L, L, P]
@@ -265,28 +265,36 @@ def rmsnorm_columns(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torc
                                      out.stride(0), dtype_code(x.dtype), T, N, _stream()), "rmsnorm_columns")
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleave: int = 0) -> None:
-    """out = silu(gate) * up.  ``interleave`` 0: gate_up[t] = [gate | up]; 8: blocks of 8 gate then 8 up."""
+GATES = {"silu": 0, "gelu_tanh": 1}
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleave: int = 0, act: str = "silu") -> None:
+    """out = act(gate) * up, ``act`` one of ``GATES``.  ``interleave`` 0: gate_up[t] = [gate | up]; 8: blocks of 8 gate then
+    8 up."""
     T, I2 = gate_up.shape
     assert out.shape == (T, I2 // 2) and gate_up.is_contiguous() and out.is_contiguous()
     assert out.dtype == gate_up.dtype and interleave in (0, 8)
-    _check(core().rb_swiglu(_ptr(gate_up), _ptr(out), dtype_code(out.dtype), T, I2 // 2, interleave, _stream()), "swiglu")
+    _check(core().rb_swiglu(_ptr(gate_up), _ptr(out), dtype_code(out.dtype), T, I2 // 2, interleave, GATES[act], _stream()), "swiglu")
 
 
-def postnorm_add_norm(stream: torch.Tensor, delta: torch.Tensor, post, nxt=None, out: Optional[torch.Tensor] = None) -> None:
+def postnorm_add_norm(stream: torch.Tensor, delta: Optional[torch.Tensor], post, nxt=None, out: Optional[torch.Tensor] = None) -> None:
     """stream (float32) += rmsnorm(delta) * (offset + w) with ``post`` = (w, eps, offset); with ``nxt`` = (w, eps, offset)
     and ``out``, also out = rmsnorm(stream) * (offset + w): the joint between two sublayers of a layer that norms a
-    sublayer's output as well as its input."""
+    sublayer's output.  ``out`` without ``nxt``: out = stream in out's type, for a layer whose sublayers read the stream
+    itself.  ``delta`` (and ``post``) None: nothing is added."""
     T, H = stream.shape
-    assert stream.dtype == torch.float32 and stream.is_contiguous() and delta.shape == stream.shape and delta.is_contiguous()
-    wp, eps_p, off_p = post
-    assert wp.numel() == H
+    assert stream.dtype == torch.float32 and stream.is_contiguous() and (delta is not None or out is not None)
+    wp, eps_p, off_p = post if delta is not None else (None, 0.0, 0.0)
+    if delta is not None:
+        assert delta.shape == stream.shape and delta.is_contiguous() and wp.numel() == H
     wn, eps_n, off_n = nxt if nxt is not None else (None, 0.0, 0.0)
     if out is not None:
-        assert wn is not None and wn.numel() == H and out.shape == stream.shape and out.is_contiguous() and out.dtype == delta.dtype
-    _check(core().rb_postnorm_add_norm(_ptr(stream), _ptr(delta), _ptr(wp), dtype_code(wp.dtype), eps_p, off_p, _ptr(wn),
-                                       dtype_code(wn.dtype) if wn is not None else F32, eps_n, off_n, _ptr(out),
-                                       dtype_code(delta.dtype), T, H, _stream()), "postnorm_add_norm")
+        assert out.shape == stream.shape and out.is_contiguous() and (delta is None or out.dtype == delta.dtype)
+        assert wn is None or wn.numel() == H
+    _check(core().rb_postnorm_add_norm(_ptr(stream), _ptr(delta), _ptr(wp), dtype_code(wp.dtype) if wp is not None else F32, eps_p,
+                                       off_p, _ptr(wn), dtype_code(wn.dtype) if wn is not None else F32, eps_n, off_n, _ptr(out),
+                                       dtype_code((delta if delta is not None else out).dtype), T, H, _stream()),
+           "postnorm_add_norm")
 
 
 def softcap(x: torch.Tensor, cap: float) -> None:
@@ -313,25 +321,31 @@ SKINNY_MAX_ROWS = 8             # what the engine gives it: beyond 8 rows the li
                                 # 16 rows and 106 at 32, for N = 24576, K = 4096)
 
 
+def _gated_code(gated: bool, act: str = "silu") -> int:
+    """What the products with a gated epilogue take: 0, or 1 + the number of the gate."""
+    return 1 + GATES[act] if gated else 0
+
+
 def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gated: bool = False, act: Optional[str] = None,
                 bias: Optional[torch.Tensor] = None) -> None:
     """out[M, N] = x[M, K] @ w[N, K]^T for M <= 32 in bfloat16: the weight-streaming kernel of decode steps
     (the engine uses it up to 8 rows).
-    ``gated``: w holds gate and up rows interleaved in blocks of 8; out[M, N/2] = silu(gate) * up.
-    ``act``: one of ``ACTIVATIONS`` applied to the float32 sums before they are stored (``bias``: its bias per column)."""
+    ``gated``: w holds gate and up rows interleaved in blocks of 8; out[M, N/2] = silu(gate) * up, or with ``act`` another of
+    ``GATES``.  ``act`` without ``gated``: one of ``ACTIVATIONS`` applied to the float32 sums before they are stored (``bias``: its
+    bias per column)."""
     M, K = x.shape
     N = w.shape[0]
     assert x.dtype == w.dtype == torch.bfloat16 and out.dtype in (torch.bfloat16, torch.float32)
     assert w.shape[1] == K and out.shape == (M, N // 2 if gated else N) and M <= SKINNY_KERNEL_MAX_ROWS
     assert x.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1
-    if act is not None:
-        assert not gated and (bias is None or (act == "neg_exp_exp" and bias.numel() == N and bias.is_contiguous()))
+    if act is not None and not gated:
+        assert (bias is None or (act == "neg_exp_exp" and bias.numel() == N and bias.is_contiguous()))
         _check(core().rb_gemm_skinny_act(_ptr(x), _ptr(w), _ptr(out), 1 if out.dtype == torch.float32 else 0,
                                          ACTIVATIONS[act], _ptr(bias), dtype_code(bias.dtype) if bias is not None else F32,
                                          M, N, K, x.stride(0), w.stride(0), out.stride(0), _stream()), "gemm_skinny_act")
         return
     _check(core().rb_gemm_skinny(_ptr(x), _ptr(w), _ptr(out), 1 if out.dtype == torch.float32 else 0,
-                                 1 if gated else 0, M, N, K, x.stride(0), w.stride(0), out.stride(0), _stream()),
+                                 _gated_code(gated, act or "silu"), M, N, K, x.stride(0), w.stride(0), out.stride(0), _stream()),
            "gemm_skinny")
 
 
@@ -410,23 +424,23 @@ def pair_ok(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> bool:
             and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def gated_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, interleave: int, ctx=None) -> None:
-    """out[T, I] = silu(x @ gate^T) * (x @ up^T) for the fused weight ``w`` [2I, K] of a gated
+def gated_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, interleave: int, ctx=None, act: str = "silu") -> None:
+    """out[T, I] = act(x @ gate^T) * (x @ up^T), ``act`` one of ``GATES``, for the fused weight ``w`` [2I, K] of a gated
     feed-forward.  With the interleaved layout the product's epilogue does the gating where an own kernel
     is the fastest: for few rows (weight streaming) and for many (tcgen05, pairs of CTAs); otherwise a product
     into a [T, 2I] buffer (from ``ctx``, a parts.base.LayerContext, if given) is followed by the SwiGLU kernel."""
     if interleave == 8 and skinny_ok(x, w):
-        gemm_skinny(x, w, out, gated=True)
+        gemm_skinny(x, w, out, gated=True, act=act)
         return
     if interleave == 8 and x.shape[0] >= PAIR_MIN_ROWS and pair_ok(x, w, out):
-        gemm_tc5(x, w, out, gated=True, pair=True)
+        gemm_tc5(x, w, out, gated=True, pair=True, act=act)
         return
     if ctx is not None:
         gu = ctx.buffer("gated_linear.gate_up", (x.shape[0], w.shape[0]), x.dtype, x.device)
     else:
         gu = torch.empty((x.shape[0], w.shape[0]), dtype=x.dtype, device=x.device)
     linear(x, w, gu)
-    swiglu(gu, out, interleave)
+    swiglu(gu, out, interleave, act)
 
 
 _tc5 = None
@@ -491,9 +505,9 @@ def check_status(device) -> None:
 
 
 def gemm_tc5(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gated: bool = False, simple_bn: int = 0,
-             pair: bool = False) -> None:
-    """out[M, N] = x[M, K] @ w[N, K]^T on the tcgen05 tensor cores (TMA-fed).  ``gated``: SwiGLU epilogue over
-    woven gate/up rows of w, out [M, N/2].  ``simple_bn``: run the one-stage twin with that tile width.
+             pair: bool = False, act: str = "silu") -> None:
+    """out[M, N] = x[M, K] @ w[N, K]^T on the tcgen05 tensor cores (TMA-fed).  ``gated``: the gated unit (its gate: ``act``,
+    one of ``GATES``) over woven gate/up rows of w as the epilogue, out [M, N/2].  ``simple_bn``: run the one-stage twin with that tile width.
     ``pair``: 256 x 256 tiles by pairs of CTAs (two-SM MMAs)."""
     M, K = x.shape
     N = w.shape[0]
@@ -507,7 +521,7 @@ def gemm_tc5(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gated: bool = 
                                           w.stride(0), out.stride(0), _ptr(status), _stream())
     else:
         fn = tc5_lib().rb_tc5_gemm_pair if pair else tc5_lib().rb_tc5_gemm
-        rc = fn(_ptr(x), _ptr(w), _ptr(out), f32, 1 if gated else 0, M, N, K, x.stride(0),
+        rc = fn(_ptr(x), _ptr(w), _ptr(out), f32, _gated_code(gated, act), M, N, K, x.stride(0),
                 w.stride(0), out.stride(0), _ptr(status), _stream())
     _tc5_launched.add(x.device)
     _check(rc, "gemm_tc5")
@@ -582,9 +596,12 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: Optional[st
 
 def qk_norm_rope_write(qkv, q_weight, k_weight, eps, cos, sin, rot_dim, pos, tok_seg, block_table,
                        page_size, k_pool, v_pool, num_heads, num_kv_heads, head_dim, write_kv=True,
-                       offset=0.0) -> None:
+                       offset=0.0, norm_size=None, blend=None) -> None:
     """In place on qkv [T, (Hq+2Hkv)*D]: q heads normed and rotated; k heads normed, rotated and
-    written to ``k_pool``; v heads written to ``v_pool``.  Pools: [pages, Hkv, P, D]."""
+    written to ``k_pool``; v heads written to ``v_pool``.  Pools: [pages, Hkv, P, D].  ``norm_size``: the elements of a
+    head that the norm's mean runs over, where heads are padded with zeros (None: all).  ``blend`` = (first, head_stride, n,
+    share): what is cached of a value v is (1 - share) v + share first, ``first`` [T, ...] the values of an earlier layer
+    (kv head g from column g * head_stride, n of them; what lies behind is zero in both), ``share`` one number."""
     T = qkv.shape[0]
     assert qkv.stride(1) == 1
     assert pos.dtype == tok_seg.dtype == block_table.dtype == torch.int32
@@ -602,7 +619,16 @@ def qk_norm_rope_write(qkv, q_weight, k_weight, eps, cos, sin, rot_dim, pos, tok
         _ptr(qkv), qkv.stride(0), _ptr(q_weight), _ptr(k_weight), wd, eps, offset, _ptr(cos), _ptr(sin),
         rot_dim, _ptr(pos), _ptr(tok_seg), _ptr(block_table), block_table.stride(0), page_size,
         _ptr(k_pool), _ptr(v_pool), dtype_code(qkv.dtype), T, num_heads, num_kv_heads, head_dim,
-        1 if write_kv else 0, _stream()), "qk_norm_rope_write")
+        1 if write_kv else 0, int(norm_size or 0), *_blend_args(blend, qkv), _stream()), "qk_norm_rope_write")
+
+
+def _blend_args(blend, qkv):
+    """(first, its row length, head stride, values a head, share, share's type) for the kernels that cache values."""
+    if blend is None:
+        return None, 0, 0, 0, None, F32
+    first, head_stride, n, share = blend
+    assert first.dtype == qkv.dtype and first.stride(1) == 1 and first.shape[0] == qkv.shape[0] and share.numel() == 1
+    return _ptr(first), first.stride(0), head_stride, n, _ptr(share), dtype_code(share.dtype)
 
 
 def attention_simt(qkv, k_pool, v_pool, pos, tok_seg, block_table, page_size, out, num_heads,
@@ -633,10 +659,11 @@ def attention_lib(head_dim: int) -> ctypes.CDLL:
         P, I, F = c_void_p, c_int, c_float
         lib.rb_attn_prefill.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, I, I, F, I, P, P]
         lib.rb_attn_decode.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, P, I, I, F, I, I, P, P]
-        lib.rb_attn_decode_fused.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, P, I, I, F, I, I, P, P, I, F, F, P, P, I, I, P]
+        lib.rb_attn_decode_fused.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, P, I, I, F, I, I, P, P, I, F, F, P, P, I, I,
+                                             I, P, I, I, I, P, I, P, I, F, P, P, I, I, P]
         lib.rb_attn_decode_fused.restype = c_int
-        lib.rb_attn_prefill_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, I, I, F, I, P, I, F, P, P, I, P]
-        lib.rb_attn_decode_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, P, I, I, F, I, I, P, I, F, P, P, I, P]
+        lib.rb_attn_prefill_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, I, I, F, I, P, I, F, P, P, I, I, P]
+        lib.rb_attn_decode_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, P, I, I, F, I, I, P, I, F, P, P, I, I, P]
         lib.rb_attn_prefill_mod.restype = lib.rb_attn_decode_mod.restype = c_int
         lib.rb_attn_decode_scratch_floats.argtypes = [I, I, I]
         lib.rb_attn_decode_scratch_floats.restype = ctypes.c_longlong
@@ -679,7 +706,7 @@ def attention_tc5_lib(head_dim: int) -> ctypes.CDLL:
         lib = build.load(f"return_attn_tc5_d{head_dim}", ["attention_tc5.cu"], _attn_tc5_defines(head_dim))
         P, I, F = c_void_p, c_int, c_float
         lib.rb_attn_prefill_tc5.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, I, I, F, I, I, P, I, P, P, P]
-        lib.rb_attn_prefill_tc5_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, I, I, F, I, I, P, I, P, P, I, F, P, P, I, P]
+        lib.rb_attn_prefill_tc5_mod.argtypes = [P, I, P, P, P, I, P, P, P, I, I, P, I, I, F, I, I, P, I, P, P, I, F, P, P, I, I, P]
         lib.rb_attn_prefill_tc5_mod.restype = c_int
         lib.rb_attn_tc5_split_floats.argtypes = [I, I, I]
         lib.rb_attn_tc5_split_floats.restype = ctypes.c_longlong
@@ -705,12 +732,12 @@ def _bias_args(bias, num_heads):
 
 def attention_prefill_tc5(qkv, k_pool, v_pool, tiles, cu_q, seg_pos0, block_table, page_size, out, num_heads,
                           num_kv_heads, head_dim, scale, window=0, num_splits=1, held=None, sink=None,
-                          chunk=0, softcap=0.0, slopes=None, bias=None) -> None:
+                          chunk=0, softcap=0.0, slopes=None, bias=None, keep=0) -> None:
     """tcgen05 attention for the listed (segment, first row) blocks of up to TC5_TILE_ROWS query rows
     (the blocks with the longest contexts should come first: they take longest).  ``num_splits`` > 1 splits
     every block's keys over that many CTAs and merges them in a second launch; ``held``: the step's map of
-    work buffers, so that the layers share the buffer of the partial results.  ``chunk``, ``softcap``, ``slopes``, ``bias``:
-    the score options of ``paged_attention``."""
+    work buffers, so that the layers share the buffer of the partial results.  ``chunk``, ``softcap``, ``slopes``, ``bias``,
+    ``keep``: the score options of ``paged_attention``."""
     assert qkv.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.is_contiguous()
     assert tiles.dtype == torch.int32 and tiles.is_contiguous()
     lib = attention_tc5_lib(head_dim)
@@ -729,7 +756,8 @@ def attention_prefill_tc5(qkv, k_pool, v_pool, tiles, cu_q, seg_pos0, block_tabl
                                        block_table.stride(0), page_size, _ptr(out), num_heads, num_kv_heads, scale,
                                        int(window or 0), num_splits, _ptr(scratch), T, _ptr(tc5_status(qkv.device)),
                                        _sink_ptr(sink, num_heads), int(chunk or 0), float(softcap or 0.0),
-                                       _sink_ptr(slopes, num_heads), *_bias_args(bias, num_heads), _stream()), "attention_prefill_tc5", 2 if num_splits > 1 else 1)
+                                       _sink_ptr(slopes, num_heads), *_bias_args(bias, num_heads), int(keep or 0), _stream()),
+           "attention_prefill_tc5", 2 if num_splits > 1 else 1)
 
 
 PREFILL_SPLIT_MIN_KEYS = 512       # a CTA of a split block keeps at least this many keys
@@ -777,9 +805,9 @@ def decode_splits(n_ctas_base: int, max_kv_len: int, ctas_per_sm: int = 2) -> in
 
 def attention_prefill_mma(qkv, k_pool, v_pool, tiles, cu_q, seg_pos0, block_table, page_size, out, num_heads,
                           num_kv_heads, head_dim, scale, window=0, sink=None, chunk=0, softcap=0.0, slopes=None,
-                          bias=None) -> None:
+                          bias=None, keep=0) -> None:
     """Tensor-core attention for the listed (segment, first row) tiles of up to 64 query rows.  ``chunk``, ``softcap``,
-    ``slopes``, ``bias``: the score options of ``paged_attention``."""
+    ``slopes``, ``bias``, ``keep``: the score options of ``paged_attention``."""
     assert qkv.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.is_contiguous()
     assert tiles.dtype == torch.int32 and tiles.is_contiguous()
     lib = attention_lib(head_dim)
@@ -787,7 +815,7 @@ def attention_prefill_mma(qkv, k_pool, v_pool, tiles, cu_q, seg_pos0, block_tabl
                                    _ptr(cu_q), _ptr(seg_pos0), _ptr(block_table), block_table.stride(0), page_size,
                                    _ptr(out), num_heads, num_kv_heads, scale, int(window or 0), _sink_ptr(sink, num_heads),
                                    int(chunk or 0), float(softcap or 0.0), _sink_ptr(slopes, num_heads), *_bias_args(bias, num_heads),
-                                   _stream()), "attention_prefill")
+                                   int(keep or 0), _stream()), "attention_prefill")
 
 
 def _split_scratch(lib, n, num_heads, num_splits, device, held=None):
@@ -805,9 +833,9 @@ def _split_scratch(lib, n, num_heads, num_splits, device, held=None):
 
 def attention_decode_mma(qkv, k_pool, v_pool, decode_segs, cu_q, seg_kv_len, block_table, page_size, out,
                          num_heads, num_kv_heads, head_dim, scale, window=0, num_splits=1, held=None, sink=None,
-                         chunk=0, softcap=0.0, slopes=None, bias=None) -> None:
+                         chunk=0, softcap=0.0, slopes=None, bias=None, keep=0) -> None:
     """Tensor-core attention for segments of one token, the keys split ``num_splits`` ways.  ``chunk``, ``softcap``,
-    ``slopes``, ``bias``: the score options of ``paged_attention``."""
+    ``slopes``, ``bias``, ``keep``: the score options of ``paged_attention``."""
     assert qkv.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.is_contiguous()
     lib = attention_lib(head_dim)
     n = decode_segs.shape[0]
@@ -816,7 +844,8 @@ def attention_decode_mma(qkv, k_pool, v_pool, decode_segs, cu_q, seg_kv_len, blo
                                   _ptr(cu_q), _ptr(seg_kv_len), _ptr(block_table), block_table.stride(0), page_size,
                                   _ptr(scratch), _ptr(out), num_heads, num_kv_heads, scale, int(window or 0),
                                   num_splits, _sink_ptr(sink, num_heads), int(chunk or 0), float(softcap or 0.0),
-                                  _sink_ptr(slopes, num_heads), *_bias_args(bias, num_heads), _stream()), "attention_decode", 2 if num_splits > 1 else 1)
+                                  _sink_ptr(slopes, num_heads), *_bias_args(bias, num_heads), int(keep or 0), _stream()),
+           "attention_decode", 2 if num_splits > 1 else 1)
 
 
 def _decode_split_count(batch, num_heads, num_kv_heads, window) -> int:
@@ -841,6 +870,11 @@ def _decode_split_count_now(batch, num_heads, num_kv_heads, window) -> int:
         longest = min(longest, int(window))
     fixed = getattr(batch, "variant", {}).get(decode_splits_key(num_heads, num_kv_heads, window))
     return fixed or decode_splits(base, longest)
+
+
+def keys_seen(window, keep=0):
+    """How many keys a query can see at most: the window and the kept first positions, or None (all)."""
+    return int(window) + int(keep or 0) if window else None
 
 
 def decode_splits_key(num_heads, num_kv_heads, window):
@@ -872,13 +906,14 @@ def decode_only(batch, dtype, num_heads, num_kv_heads, window=None) -> bool:
 
 def attention_decode_fused(qkv, q_weight, k_weight, eps, offset, cos, sin, rot_dim, k_pool, v_pool, batch,
                            block_table, page_size, out, num_heads, num_kv_heads, head_dim, scale, window=None,
-                           write_kv=True) -> None:
-    """A step of single tokens: per-head q/k norm, rotation, cache write and split-KV attention in one kernel
-    (plus the merge of the splits).  ``qkv`` holds the raw projections and is left as it is."""
+                           write_kv=True, norm_size=None, blend=None, sink=None, softcap=None, keep=0) -> None:
+    """A step of single tokens: per-head q/k norm, rotation, blend of the values, cache write and split-KV attention in one
+    kernel (plus the merge of the splits).  ``qkv`` holds the raw projections and is left as it is.  ``norm_size``,
+    ``blend``: as in ``qk_norm_rope_write``; ``sink``, ``softcap``, ``keep``: as in ``paged_attention``."""
     assert qkv.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.is_contiguous()
     lib = attention_lib(head_dim)
     n = batch.decode_segs.shape[0]
-    splits = _decode_split_count(batch, num_heads, num_kv_heads, window)
+    splits = _decode_split_count(batch, num_heads, num_kv_heads, keys_seen(window, keep))
     scratch = _split_scratch(lib, n, num_heads, splits, qkv.device, getattr(batch, "scratch", None))
     if rot_dim:
         assert cos.dtype == torch.float32 and sin.dtype == torch.float32 and cos.shape[1] * 2 == rot_dim
@@ -890,24 +925,29 @@ def attention_decode_fused(qkv, q_weight, k_weight, eps, offset, cos, sin, rot_d
                                     _ptr(batch.cu_q), _ptr(batch.seg_kv_len), _ptr(block_table), block_table.stride(0),
                                     page_size, _ptr(scratch), _ptr(out), num_heads, num_kv_heads, scale,
                                     int(window or 0), splits, _ptr(q_weight), _ptr(k_weight), wd, eps, offset,
-                                    _ptr(cos), _ptr(sin), rot_dim, 1 if write_kv else 0, _stream()),
+                                    _ptr(cos), _ptr(sin), rot_dim, 1 if write_kv else 0, int(norm_size or 0),
+                                    *_blend_args(blend, qkv), _sink_ptr(sink, num_heads), 0, float(softcap or 0.0), None,
+                                    None, 0, int(keep or 0), _stream()),
            "attention_decode_fused", 2 if splits > 1 else 1)
 
 
 def paged_attention(qkv, k_pool, v_pool, batch, block_table, page_size, out, num_heads, num_kv_heads,
-                    head_dim, scale, window=None, sink=None, chunk=None, softcap=None, slopes=None, bias=None) -> None:
+                    head_dim, scale, window=None, sink=None, chunk=None, softcap=None, slopes=None, bias=None,
+                    keep=0) -> None:
     """Attention of every token of the step over its request's cached keys (its own included).
 
     float32: the CUDA-core kernel, whose result does not depend on how the work was cut.
     bfloat16: the tensor-core kernels, one for prompt portions and one (split over the keys) for
     single decoded tokens.
 
-    Options of the score: ``window`` (the last n keys) or ``chunk`` (the keys of the query's own block of n positions,
+    Options of the score: ``window`` (the last n keys, and with ``keep`` also the sequence's first ``keep`` keys) or ``chunk`` (the keys of the query's own block of n positions,
     blocks counted from position 0), never both; ``sink`` (float32 [heads]: exp(sink) joins the softmax's denominator);
     ``softcap`` (a scaled score s becomes cap * tanh(s / cap)); ``slopes`` (float32 [heads]: slopes[h] * (i - j) is taken
     off the score of key j for query i); ``bias`` (float32 [heads, n]: bias[h, min(i - j, n - 1)] is added to it)."""
     if window and chunk:
         raise KernelError("a window and a chunk exclude each other")
+    if keep and not window:
+        raise KernelError("kept first positions go with a window")
     if qkv.dtype == torch.float32:
         T = qkv.shape[0]
         assert out.is_contiguous() and out.dtype == qkv.dtype and k_pool.dtype == qkv.dtype
@@ -915,26 +955,26 @@ def paged_attention(qkv, k_pool, v_pool, batch, block_table, page_size, out, num
             _ptr(qkv), qkv.stride(0), _ptr(k_pool), _ptr(v_pool), _ptr(batch.pos), _ptr(batch.tok_seg), _ptr(block_table),
             block_table.stride(0), page_size, _ptr(out), dtype_code(qkv.dtype), T, num_heads, num_kv_heads, head_dim, scale,
             int(window or 0), int(chunk or 0), float(softcap or 0.0), _sink_ptr(slopes, num_heads),
-            _sink_ptr(sink, num_heads), *_bias_args(bias, num_heads), _stream()), "attention_simt")
+            _sink_ptr(sink, num_heads), *_bias_args(bias, num_heads), int(keep or 0), _stream()), "attention_simt")
         return
     host = batch.host
-    bound = window or chunk                       # either bounds the keys a query can see
+    bound = keys_seen(window, keep) or chunk      # either bounds the keys a query can see
     if host.num_multi:
         if head_dim in TC5_ATTENTION_HEAD_DIMS:
             attention_prefill_tc5(qkv, k_pool, v_pool, batch.tiles[TILES_TC5], batch.cu_q, batch.seg_pos0, block_table,
                                   page_size, out, num_heads, num_kv_heads, head_dim, scale, window or 0,
                                   _prefill_split_count(batch, num_heads, bound), getattr(batch, "scratch", None), sink,
-                                  chunk, softcap, slopes, bias)
+                                  chunk, softcap, slopes, bias, keep)
         else:
             attention_prefill_mma(qkv, k_pool, v_pool, batch.tiles[TILES_MMA], batch.cu_q, batch.seg_pos0, block_table,
                                   page_size, out, num_heads, num_kv_heads, head_dim, scale, window or 0, sink,
-                                  chunk, softcap, slopes, bias)
+                                  chunk, softcap, slopes, bias, keep)
     n_dec = host.decode_segs.shape[0]
     if n_dec:
         attention_decode_mma(qkv, k_pool, v_pool, batch.decode_segs, batch.cu_q, batch.seg_kv_len, block_table,
                              page_size, out, num_heads, num_kv_heads, head_dim, scale, window or 0,
                              _decode_split_count(batch, num_heads, num_kv_heads, bound), getattr(batch, "scratch", None), sink,
-                             chunk, softcap, slopes, bias)
+                             chunk, softcap, slopes, bias, keep)
 
 
 def attention_prepare(proj, q_off: int, k_off: int, v_off: int, biases, norms, eps: float, tables, batch, kv, q_out,
@@ -1598,11 +1638,11 @@ def moe_lib() -> ctypes.CDLL:
         lib = build.load("return_moe", _MOE_SOURCES, {"RB_PDL_MODE": PDL_MODE})
         P, I, F = c_void_p, c_int, c_float
         lib.rb_moe_route.argtypes = [P, I, P, P, P, I, I, I, I, I, F, I, I, F, I, P]
-        lib.rb_moe_pair_linear.argtypes = [P, I, I, P, P, P, I, I, I, I, I, P]
+        lib.rb_moe_pair_linear.argtypes = [P, I, I, P, P, P, I, I, I, I, I, I, P]
         lib.rb_clamped_glu.argtypes = [P, I, P, I, I, I, I, F, F, F, P, P, P]
-        lib.rb_moe_combine.argtypes = [P, P, P, P, P, I, I, I, I, P]
+        lib.rb_moe_combine.argtypes = [P, P, P, P, P, I, P, I, I, I, I, P]
         lib.rb_moe_sort.argtypes = [P, I, I, P, P, P, P]
-        lib.rb_moe_grouped_gemm.argtypes = [P, I, P, I, P, P, I, P, I, I, I, I, P]
+        lib.rb_moe_grouped_gemm.argtypes = [P, I, P, I, P, P, I, P, I, I, I, I, I, P]
         lib.rb_moe_gather_rows.argtypes = [P, ctypes.c_longlong, P, I, P, I, I, P]
         for name in ("rb_moe_route", "rb_moe_pair_linear", "rb_clamped_glu", "rb_moe_combine", "rb_moe_sort",
                      "rb_moe_grouped_gemm", "rb_moe_gather_rows"):
@@ -1629,14 +1669,19 @@ def moe_route(logits, expert_of, weight, top: int, groups: int = 1, keep: int = 
                                   keep, tiny, {"softmax": 0, "sigmoid": 1}[score], group_top, scale, 1 if renorm else 0, _stream()), "moe_route")
 
 
-def moe_pair_linear(x, in_div: int, w, expert_of, out) -> None:
-    """out[i] = x[i // in_div] @ w[expert_of[i]]^T for every (token, chosen expert) pair i; w [E, N, K]."""
+def _act_code(act: Optional[str]) -> int:
+    return -1 if act is None else ACTIVATIONS[act]
+
+
+def moe_pair_linear(x, in_div: int, w, expert_of, out, act: Optional[str] = None) -> None:
+    """out[i] = x[i // in_div] @ w[expert_of[i]]^T for every (token, chosen expert) pair i; w [E, N, K].  ``act``: one of
+    ``ACTIVATIONS`` (without a bias) on the float32 sums."""
     E, N, K = w.shape
     pairs = expert_of.numel()
     assert x.dtype == w.dtype == out.dtype and x.stride(1) == 1 and w.is_contiguous() and out.stride(1) == 1
     assert x.shape[1] == K and out.shape == (pairs, N) and x.shape[0] * in_div == pairs
     _check(moe_lib().rb_moe_pair_linear(_ptr(x), x.stride(0), in_div, _ptr(w), _ptr(expert_of), _ptr(out), out.stride(0),
-                                        dtype_code(x.dtype), pairs, N, K, _stream()), "moe_pair_linear")
+                                        dtype_code(x.dtype), pairs, N, K, _act_code(act), _stream()), "moe_pair_linear")
 
 
 def clamped_glu(gate_up, out, limit: float, alpha: float, shift: float = 1.0, weight=None, pair_at=None) -> None:
@@ -1652,9 +1697,9 @@ def clamped_glu(gate_up, out, limit: float, alpha: float, shift: float = 1.0, we
            "clamped_glu")
 
 
-def moe_combine(y, weight, shared, out, row_of=None, top=None) -> None:
-    """out[t] = sum_k weight[t, k] * y[row of pair t * top + k] (+ shared[t]); sums in float32 in the order of k.  ``weight``
-    None (with ``top``): a plain sum."""
+def moe_combine(y, weight, shared, out, row_of=None, top=None, shared_gate=None) -> None:
+    """out[t] = sum_k weight[t, k] * y[row of pair t * top + k] (+ c shared[t]); sums in float32 in the order of k; c = 1, or
+    the logistic of ``shared_gate``[t] (float32 [T], any stride).  ``weight`` None (with ``top``): a plain sum."""
     T, H = out.shape
     if weight is not None:
         assert weight.shape[0] == T and weight.dtype == torch.float32 and weight.is_contiguous()
@@ -1662,8 +1707,11 @@ def moe_combine(y, weight, shared, out, row_of=None, top=None) -> None:
     assert y.shape == (T * top, H) and y.is_contiguous() and out.is_contiguous() and out.dtype == y.dtype
     if shared is not None:
         assert shared.shape == out.shape and shared.is_contiguous() and shared.dtype == y.dtype
-    _check(moe_lib().rb_moe_combine(_ptr(y), _ptr(row_of), _ptr(weight), _ptr(shared), _ptr(out), dtype_code(y.dtype), T, H, top,
-                                    _stream()), "moe_combine")
+    if shared_gate is not None:
+        assert shared is not None and shared_gate.dtype == torch.float32 and shared_gate.shape == (T,)
+    _check(moe_lib().rb_moe_combine(_ptr(y), _ptr(row_of), _ptr(weight), _ptr(shared), _ptr(shared_gate),
+                                    shared_gate.stride(0) if shared_gate is not None else 0, _ptr(out), dtype_code(y.dtype), T, H,
+                                    top, _stream()), "moe_combine")
 
 
 def moe_sort(expert_of, num_experts: int, offsets, pair_at, place_of) -> None:
@@ -1676,15 +1724,15 @@ def moe_sort(expert_of, num_experts: int, offsets, pair_at, place_of) -> None:
            "moe_sort")
 
 
-def moe_grouped_gemm(x, pair_at, in_div: int, w, offsets, out) -> None:
+def moe_grouped_gemm(x, pair_at, in_div: int, w, offsets, out, act: Optional[str] = None) -> None:
     """out[place] = x[row(place)] @ w[expert of the place]^T on the tensor cores, bfloat16: row(place) = pair_at[place] //
-    in_div, or the place itself with pair_at None.  w [E, N, K]; offsets int32 [E + 1]."""
+    in_div, or the place itself with pair_at None.  w [E, N, K]; offsets int32 [E + 1].  ``act``: as in ``moe_pair_linear``."""
     E, N, K = w.shape
     places = out.shape[0]
     assert x.dtype == w.dtype == out.dtype == torch.bfloat16 and x.stride(1) == 1 and w.is_contiguous() and out.stride(1) == 1
     assert x.shape[1] == K and out.shape[1] == N
     _check(moe_lib().rb_moe_grouped_gemm(_ptr(x), x.stride(0), _ptr(pair_at), in_div, _ptr(w), _ptr(offsets), E, _ptr(out),
-                                         out.stride(0), places, N, K, _stream()), "moe_grouped_gemm")
+                                         out.stride(0), places, N, K, _act_code(act), _stream()), "moe_grouped_gemm")
 
 
 _moe_tc5 = None
@@ -1697,7 +1745,7 @@ def moe_tc5_lib() -> ctypes.CDLL:
     if _moe_tc5 is None:
         lib = build.load("return_moe_tc5", _MOE_TC5_SOURCES, {"RB_PDL_MODE": PDL_MODE})
         P, I = c_void_p, c_int
-        lib.rb_moe_tc5_gemm.argtypes = [P, I, P, P, I, P, I, I, I, I, P, P]
+        lib.rb_moe_tc5_gemm.argtypes = [P, I, P, P, I, P, I, I, I, I, I, P, P]
         lib.rb_moe_tc5_gemm.restype = c_int
         _moe_tc5 = lib
     return _moe_tc5
@@ -1712,15 +1760,16 @@ def moe_gather_rows(x, pair_at, in_div: int, out) -> None:
                                         _stream()), "moe_gather_rows")
 
 
-def moe_tc5_gemm(x_sorted, w, offsets, out) -> None:
-    """out[place] = x_sorted[place] @ w[expert of the place]^T on tcgen05 (TMA-fed), bfloat16; w [E, N, K]."""
+def moe_tc5_gemm(x_sorted, w, offsets, out, act: Optional[str] = None) -> None:
+    """out[place] = x_sorted[place] @ w[expert of the place]^T on tcgen05 (TMA-fed), bfloat16; w [E, N, K].  ``act``: as in
+    ``moe_pair_linear``."""
     E, N, K = w.shape
     places = out.shape[0]
     assert x_sorted.dtype == w.dtype == out.dtype == torch.bfloat16 and x_sorted.stride(1) == 1 and w.is_contiguous()
     assert x_sorted.shape == (places, K) and out.shape[1] == N and out.stride(1) == 1
     _tc5_launched.add(x_sorted.device)
     _check(moe_tc5_lib().rb_moe_tc5_gemm(_ptr(x_sorted), x_sorted.stride(0), _ptr(w), _ptr(offsets), E, _ptr(out), out.stride(0),
-                                         places, N, K, _ptr(tc5_status(x_sorted.device)), _stream()), "moe_tc5_gemm")
+                                         places, N, K, _act_code(act), _ptr(tc5_status(x_sorted.device)), _stream()), "moe_tc5_gemm")
 
 
 # From this many (token, expert) pairs on, a step's experts run as tiles on the tensor cores over the pairs sorted by
@@ -1731,14 +1780,18 @@ MOE_GROUPED_MIN_PAIRS = 64
 MOE_TC5_MIN_PAIRS = 1024
 
 
-def moe_experts(x, gate_up, down, expert_of, weight, shared, out, limit: float, alpha: float, ctx=None,
-                shift: float = 1.0, weigh_input: bool = False) -> None:
-    """out[t] = sum_k weight[t, k] * expert_{expert_of[t, k]}(x[t]) (+ shared[t]), or with ``weigh_input`` the sum of
-    expert(weight[t, k] * x[t]); gate_up [E, 2F, H], down [E, H, F];
-    an expert is down(g sigmoid(alpha g) (u + shift)) with the gate capped at ``limit`` and the up part clamped to it."""
-    E, F2, H = gate_up.shape
+def moe_experts(x, up, down, expert_of, weight, shared, out, limit: float = float("inf"), alpha: float = 1.0, ctx=None,
+                shift: float = 1.0, weigh_input: bool = False, act: Optional[str] = None, shared_gate=None) -> None:
+    """out[t] = sum_k weight[t, k] * expert_{expert_of[t, k]}(x[t]) (+ c shared[t]), or with ``weigh_input`` the sum of
+    expert(weight[t, k] * x[t]); c as in ``moe_combine``.  Gated experts: ``up`` [E, 2F, H] (gate rows, then up rows), down
+    [E, H, F]; an expert is down(g sigmoid(alpha g) (u + shift)) with the gate capped at ``limit`` and the up part clamped to
+    it.  ``act`` (one of ``ACTIVATIONS``): experts without a gate, ``up`` [E, F, H], an expert is down(act(up)); the activation
+    is applied in the first product's epilogue."""
+    E, FU, H = up.shape
+    F = down.shape[2]
     T, top = expert_of.shape
     pairs = T * top
+    assert FU == (F if act is not None else 2 * F) and not (act is not None and weigh_input)
 
     def buf(name, shape, dtype=None):
         if ctx is not None:
@@ -1746,10 +1799,10 @@ def moe_experts(x, gate_up, down, expert_of, weight, shared, out, limit: float, 
         return torch.empty(shape, dtype=dtype or x.dtype, device=x.device)
 
     w_in, w_out = (weight, None) if weigh_input else (None, weight)
-    gu = buf("moe.pair_gate_up", (pairs, F2))
-    act = buf("moe.pair_act", (pairs, F2 // 2))
+    hidden = buf("moe.pair_act", (pairs, F))
+    gu = buf("moe.pair_gate_up", (pairs, FU)) if act is None else hidden
     y = buf("moe.pair_y", (pairs, H))
-    if (x.dtype == torch.bfloat16 and pairs >= MOE_GROUPED_MIN_PAIRS and H % 8 == 0 and F2 % 16 == 0 and x.stride(0) % 8 == 0
+    if (x.dtype == torch.bfloat16 and pairs >= MOE_GROUPED_MIN_PAIRS and H % 8 == 0 and F % 8 == 0 and x.stride(0) % 8 == 0
             and x.data_ptr() % 16 == 0):
         offsets = buf("moe.offsets", (E + 1,), torch.int32)
         pair_at = buf("moe.pair_at", (pairs,), torch.int32)
@@ -1758,19 +1811,22 @@ def moe_experts(x, gate_up, down, expert_of, weight, shared, out, limit: float, 
         if pairs >= MOE_TC5_MIN_PAIRS and E <= 1024:
             rows = buf("moe.pair_rows", (pairs, H))
             moe_gather_rows(x, pair_at, top, rows)
-            moe_tc5_gemm(rows, gate_up, offsets, gu)
-            clamped_glu(gu, act, limit, alpha, shift, w_in, pair_at)
-            moe_tc5_gemm(act, down, offsets, y)
+            moe_tc5_gemm(rows, up, offsets, gu, act)
+            if act is None:
+                clamped_glu(gu, hidden, limit, alpha, shift, w_in, pair_at)
+            moe_tc5_gemm(hidden, down, offsets, y)
         else:
-            moe_grouped_gemm(x, pair_at, top, gate_up, offsets, gu)
-            clamped_glu(gu, act, limit, alpha, shift, w_in, pair_at)
-            moe_grouped_gemm(act, None, 1, down, offsets, y)
-        moe_combine(y, w_out, shared, out, row_of=place_of, top=top)
+            moe_grouped_gemm(x, pair_at, top, up, offsets, gu, act)
+            if act is None:
+                clamped_glu(gu, hidden, limit, alpha, shift, w_in, pair_at)
+            moe_grouped_gemm(hidden, None, 1, down, offsets, y)
+        moe_combine(y, w_out, shared, out, row_of=place_of, top=top, shared_gate=shared_gate)
         return
-    moe_pair_linear(x, top, gate_up, expert_of, gu)
-    clamped_glu(gu, act, limit, alpha, shift, w_in)
-    moe_pair_linear(act, 1, down, expert_of, y)
-    moe_combine(y, w_out, shared, out, top=top)
+    moe_pair_linear(x, top, up, expert_of, gu, act)
+    if act is None:
+        clamped_glu(gu, hidden, limit, alpha, shift, w_in)
+    moe_pair_linear(hidden, 1, down, expert_of, y)
+    moe_combine(y, w_out, shared, out, top=top, shared_gate=shared_gate)
 
 
 # ------------------------------------------------------------------------------- sampling

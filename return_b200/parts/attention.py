@@ -4,7 +4,8 @@ Projections q, k, v as one fused product (the reference runs three, :29-31; the 
 their row-wise concatenation), per-head RMSNorm of q and k before the rotation (:29-30),
 rotation and cache write in one kernel (for a step of single tokens: inside the attention kernel),
 attention over the block table, output projection
-(:55-56).  Sizes, window, norm and position encoding come from the specification.
+(:55-56).  Sizes, window, norm and position encoding come from the specification, as do the options that the reference's
+model has no use for: first keys kept beside a window, capped scores, a sink, values blended with an earlier layer's.
 """
 from __future__ import annotations
 
@@ -26,22 +27,33 @@ class PagedAttention(Mixer):
             raise ValueError(f"head_dim={spec.head_dim}: the attention kernels take multiples of 16 from 16 to 256")
         if spec.window is not None and spec.window <= 0:
             raise ValueError("window must be positive")
+        if spec.keep_first < 0 or (spec.keep_first and spec.window is None):
+            raise ValueError("keep_first: not negative, and only beside a window")
+        if spec.softcap is not None and not spec.softcap > 0:
+            raise ValueError("softcap must be positive")
+        if spec.value_mix not in (None, "source", "blend"):
+            raise ValueError(f"value_mix={spec.value_mix!r}; known: None, 'source', 'blend'")
         self.q_norm = NORMS.build(spec.qk_norm, env) if spec.qk_norm is not None else None
         self.k_norm = NORMS.build(spec.qk_norm, env) if spec.qk_norm is not None else None
-        if spec.qk_norm is not None and (spec.qk_norm.kind != "rmsnorm" or spec.qk_norm.size != spec.head_dim):
-            raise ValueError("the fused q/k norm is an RMSNorm over head_dim")
+        if spec.qk_norm is not None and (spec.qk_norm.kind != "rmsnorm" or spec.qk_norm.size != (spec.key_dim or spec.head_dim)):
+            raise ValueError("the fused q/k norm is an RMSNorm over a head's elements (its key_dim, or head_dim)")
         self.position = POSITION_ENCODINGS.build(spec.position, env) if spec.position is not None else None
         self.q_size = spec.num_heads * spec.head_dim
         self.kv_size = spec.num_kv_heads * spec.head_dim
+        self._sink = None
 
     # ------------------------------------------------------------------ parameters and cache
     def params(self):
         s = self.spec
         p = {"qkv": ParamSpec((self.q_size + 2 * self.kv_size, s.hidden_size)),
              "o": ParamSpec((s.hidden_size, self.q_size))}
-        if self.q_norm is not None:
-            p["q_norm.weight"] = self.q_norm.params()["weight"]
-            p["k_norm.weight"] = self.k_norm.params()["weight"]
+        if self.q_norm is not None:           # as long as the padded heads are
+            weight = ParamSpec((s.head_dim,), role="vector", init=self.q_norm.params()["weight"].init)
+            p["q_norm.weight"] = p["k_norm.weight"] = weight
+        if s.sink:
+            p["sink"] = ParamSpec((s.num_heads,), role="vector", init="normal:0.5")
+        if s.value_mix == "blend":
+            p["value_share"] = ParamSpec((1,), role="vector", init="uniform01")
         return p
 
     def bind(self, tensors):
@@ -50,9 +62,13 @@ class PagedAttention(Mixer):
         if self.q_norm is not None:
             self.q_norm.bind({"weight": tensors["q_norm.weight"]})
             self.k_norm.bind({"weight": tensors["k_norm.weight"]})
+        if self.spec.sink:
+            self._sink = tensors["sink"].float().contiguous()
+        if self.spec.value_mix == "blend":
+            self.value_share = tensors["value_share"].float().contiguous()
 
     def cache_need(self):
-        return KVCacheNeed(self.spec.num_kv_heads, self.spec.head_dim, self.spec.window)
+        return KVCacheNeed(self.spec.num_kv_heads, self.spec.head_dim, self.spec.window, self.spec.keep_first)
 
     def batch_tilings(self):
         """The row blocks of the tensor-core kernel for prompt portions that this head size runs on."""
@@ -68,13 +84,19 @@ class PagedAttention(Mixer):
         if self.env.act_dtype != torch.bfloat16:
             return {}
         s = self.spec
-        return {ops.decode_splits_key(s.num_heads, s.num_kv_heads, s.window):
-                ops.decode_splits_for(n_tokens, longest_context, s.num_heads, s.num_kv_heads, s.window)}
+        seen = ops.keys_seen(s.window, s.keep_first)
+        return {ops.decode_splits_key(s.num_heads, s.num_kv_heads, seen):
+                ops.decode_splits_for(n_tokens, longest_context, s.num_heads, s.num_kv_heads, seen)}
 
     # ------------------------------------------------------------------ one step
+    @property
+    def _qkv_name(self):
+        """A layer whose values later layers read keeps its projections in a buffer of its own until the step is over."""
+        return "attention.qkv_source" if self.spec.value_mix == "source" else "attention.qkv"
+
     def forward(self, x, ctx):
         T = x.shape[0]
-        qkv = ctx.buffer("attention.qkv", (T, self.q_size + 2 * self.kv_size), x.dtype, x.device)
+        qkv = ctx.buffer(self._qkv_name, (T, self.q_size + 2 * self.kv_size), x.dtype, x.device)
         ops.linear(x, self.p_qkv, qkv)
         o = self.core(qkv, ctx)
         y = ctx.buffer("attention.y", (T, self.spec.hidden_size), x.dtype, x.device)
@@ -85,15 +107,18 @@ class PagedAttention(Mixer):
     # products in kernels of its own choosing (fused with the norms around them).
     def in_projection(self):
         """(weight [q + 2 kv, hidden], name of the buffer its output goes to)."""
-        return self.p_qkv, "attention.qkv"
+        return self.p_qkv, self._qkv_name
 
     def out_projection(self):
         return self.p_o
 
     def core(self, qkv, ctx):
         """From the projections [T, q + 2 kv] to the attention output [T, q]: per-head norm, position encoding,
-        cache write, attention over the block table."""
+        blend of the values, cache write, attention over the block table."""
         s, b, kv = self.spec, ctx.batch, ctx.kv
+        blend = self._blend(qkv, b)
+        norm_size = s.qk_norm.size if s.qk_norm is not None else None
+        seen = ops.keys_seen(s.window, s.keep_first)
         T = qkv.shape[0]
         qw = self.q_norm.p_weight if self.q_norm is not None else None
         kw = self.k_norm.p_weight if self.k_norm is not None else None
@@ -101,32 +126,51 @@ class PagedAttention(Mixer):
         offset = s.qk_norm.offset if s.qk_norm is not None else 0.0
         tables = self.position.rotary_tables() if self.position is not None else None
         o = ctx.buffer("attention.o", (T, self.q_size), qkv.dtype, qkv.device)
-        if (tables is not None or self.position is None) and ops.decode_only(b, qkv.dtype, s.num_heads, s.num_kv_heads, s.window):
+        if (tables is not None or self.position is None) and ops.decode_only(b, qkv.dtype, s.num_heads, s.num_kv_heads, seen):
             # single decoded tokens only: norm, rotation, cache write and attention are one kernel
             cos, sin, rot = tables if tables is not None else (None, None, 0)
             ops.attention_decode_fused(qkv, qw, kw, eps, offset, cos, sin, rot, kv.k, kv.v, b, kv.block_table,
                                        kv.page_size, o, s.num_heads, s.num_kv_heads, s.head_dim, s.scale, s.window,
-                                       write_kv=ctx.write_cache)
+                                       write_kv=ctx.write_cache, norm_size=norm_size, blend=blend, sink=self._sink,
+                                       softcap=s.softcap, keep=s.keep_first)
             return o
         if tables is not None or self.position is None:
             cos, sin, rot = tables if tables is not None else (None, None, 0)
             ops.qk_norm_rope_write(qkv, qw, kw, eps, cos, sin, rot, b.pos, b.tok_seg, kv.block_table,
                                    kv.page_size, kv.k, kv.v, s.num_heads, s.num_kv_heads, s.head_dim,
-                                   write_kv=ctx.write_cache, offset=offset)
+                                   write_kv=ctx.write_cache, offset=offset, norm_size=norm_size, blend=blend)
         else:
             # an encoding that is not a rotation of pairs: norm, then the encoding's own in-place
             # step on q and k, then the cache write
             ops.qk_norm_rope_write(qkv, qw, kw, eps, None, None, 0, b.pos, b.tok_seg, kv.block_table,
                                    kv.page_size, kv.k, kv.v, s.num_heads, s.num_kv_heads, s.head_dim,
-                                   write_kv=False, offset=offset)
+                                   write_kv=False, offset=offset, norm_size=norm_size)
             self.position.apply(qkv, b, s.num_heads, s.num_kv_heads, s.head_dim)
             if ctx.write_cache:
                 ops.qk_norm_rope_write(qkv, None, None, 0.0, None, None, 0, b.pos, b.tok_seg, kv.block_table,
                                        kv.page_size, kv.k, kv.v, s.num_heads, s.num_kv_heads, s.head_dim,
-                                       write_kv=True)
+                                       write_kv=True, blend=blend)
         ops.paged_attention(qkv, kv.k, kv.v, b, kv.block_table, kv.page_size, o, s.num_heads,
-                            s.num_kv_heads, s.head_dim, s.scale, s.window)
+                            s.num_kv_heads, s.head_dim, s.scale, s.window, self._sink, None, s.softcap, keep=s.keep_first)
         return o
+
+    def _blend(self, qkv, batch):
+        """What the cache write blends the step's values with (``ops.qk_norm_rope_write``), or None.  A "source" layer leaves
+        its raw values, columns of its projections, under ``attention.source_values`` in the step's scratch."""
+        s = self.spec
+        if s.value_mix is None:
+            return None
+        held = getattr(batch, "scratch", None)
+        if held is None:
+            raise ValueError("layers that share values within a step need the step's map of buffers")
+        if s.value_mix == "source":
+            held["attention.source_values"] = (qkv[:, self.q_size + self.kv_size:], s.num_kv_heads, s.head_dim,
+                                               s.value_dim or s.head_dim)
+            return None
+        first, heads, stride, n = held["attention.source_values"]
+        if heads != s.num_kv_heads or n != (s.value_dim or s.head_dim):
+            raise ValueError("values are blended head by head: both layers have as many key/value heads of the same value size")
+        return first, stride, n, self.value_share
 
 
 def distance_rows(rows: int, reach: float):

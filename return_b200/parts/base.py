@@ -41,10 +41,11 @@ class ParamSpec:
 
 @dataclass(frozen=True)
 class KVCacheNeed:
-    """The mixer wants paged keys and values: all of them, or a window."""
+    """The mixer wants paged keys and values: all of them, or a window and the sequence's first ``keep_first``."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)

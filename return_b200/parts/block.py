@@ -83,7 +83,7 @@ class PreNormBlock(Block):
             mixer, ff = self.mixer, self.feed_forward
             n2 = self.feed_forward_norm
             norms_ok = self.first_norm() is not None and getattr(n2.spec, "kind", None) == "rmsnorm" and hasattr(n2, "p_weight")
-            if norms_ok and hasattr(mixer, "in_projection") and hasattr(mixer, "core") and hasattr(ff, "gated_projections"):
+            if norms_ok and hasattr(mixer, "in_projection") and hasattr(mixer, "core") and hasattr(ff, "gated_projections") and getattr(ff, "gate", "silu") == "silu":
                 (w_in, in_name), w_out = mixer.in_projection(), mixer.out_projection()
                 gate_up, down, interleave = ff.gated_projections()
                 weights = (w_in, w_out, gate_up, down)
@@ -402,6 +402,81 @@ class SandwichBlock(Block):
         else:
             ops.postnorm_add_norm(stream, last[0], last[1])
         return None
+
+
+@BLOCKS.register("postnorm")
+class PostNormBlock(Block):
+    """x += norm_a(mixer(x)); x += norm_b(feed_forward(x)) (``PostNormBlockSpec``).
+
+    One kernel sits behind every sublayer: it norms the sublayer's output, adds it to the float32 stream and leaves the
+    stream in the activation type for the sublayer that runs next (csrc/elementwise.cu, ``postnorm_add_norm`` without a
+    second norm), also across the border to the next block of this kind (``postnorm.rows`` in the step's scratch).  In
+    float32 the sublayers read the stream as it lies.  The block owes the stream nothing when it returns."""
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.mixer = MIXERS.build(spec.mixer, env)
+        self.feed_forward = FEED_FORWARDS.build(spec.feed_forward, env) if spec.feed_forward is not None else None
+        self._children = {"mixer": self.mixer, "mixer_post_norm": NORMS.build(spec.mixer_post_norm, env)}
+        if self.feed_forward is not None:
+            self._children.update({"feed_forward": self.feed_forward,
+                                   "feed_forward_post_norm": NORMS.build(spec.feed_forward_post_norm, env)})
+        if any(getattr(part.spec, "kind", None) != "rmsnorm" for name, part in self._children.items() if name.endswith("norm")):
+            raise ValueError("the norms of a post-norm block are RMSNorms")
+
+    @property
+    def graph_safe(self):
+        return all(part.graph_safe for part in self._children.values())
+
+    def params(self):
+        return {f"{child}.{name}": p for child, part in self._children.items() for name, p in part.params().items()}
+
+    def bind(self, tensors):
+        for child, part in self._children.items():
+            prefix = child + "."
+            part.bind({k[len(prefix):]: v for k, v in tensors.items() if k.startswith(prefix)})
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def batch_tilings(self):
+        out = {}
+        for part in self._children.values():
+            out.update(part.batch_tilings())
+        return out
+
+    def graph_variant(self, n_tokens, longest_context):
+        out = {}
+        for part in self._children.values():
+            out.update(part.graph_variant(n_tokens, longest_context))
+        return out
+
+    def forward(self, stream, delta, ctx):
+        dt = self.env.act_dtype
+        if delta is not None:
+            ops.add_dual_norm(stream, (delta,), None, None, 0.0, 0.0, None, None)    # what the block before still owes
+        held = getattr(ctx.batch, "scratch", None)
+        pre = held.pop("postnorm.rows", None) if held is not None else None
+        rows = stream if dt == torch.float32 else ctx.buffer("postnorm.rows", tuple(stream.shape), dt, stream.device)
+        ready = delta is None and pre == ctx.position
+        if rows is not stream and not ready:
+            ops.postnorm_add_norm(stream, None, None, None, rows)
+        copy = rows if rows is not stream else None               # where a joint leaves the new stream for the next sublayer
+        nxt = ctx.next_block
+        ahead = copy is not None and held is not None and isinstance(nxt, PostNormBlock)
+        y = self.mixer.forward(rows, ctx)
+        if self.feed_forward is not None:
+            ops.postnorm_add_norm(stream, y, self._triple("mixer_post_norm"), None, copy)
+            y = self.feed_forward.forward(rows, ctx)
+        last = "feed_forward_post_norm" if self.feed_forward is not None else "mixer_post_norm"
+        ops.postnorm_add_norm(stream, y, self._triple(last), None, copy if ahead else None)
+        if ahead:
+            held["postnorm.rows"] = ctx.position + 1              # the rows' buffer holds the input of the run with this position
+        return None
+
+    def _triple(self, name):
+        n = self._children[name]
+        return n.p_weight, n.spec.eps, n.spec.offset
 
 
 @BLOCKS.register("hyper")

@@ -1,4 +1,4 @@
-"""Dense SwiGLU feed-forward (rollout/monkey_patch/qwen3.py:20-22,99-105)."""
+"""Dense gated feed-forward, SwiGLU unless its specification names another gate (rollout/monkey_patch/qwen3.py:20-22,99-105)."""
 from __future__ import annotations
 
 import torch
@@ -9,7 +9,7 @@ from .base import FEED_FORWARDS, FeedForward, ParamSpec, work_buffer
 
 @FEED_FORWARDS.register("swiglu")
 class SwiGLU(FeedForward):
-    """y = down( silu(g) * u ) with [g, u] = x @ gate_up^T.  The reference concatenates gate rows
+    """y = down( act(g) * u ) with [g, u] = x @ gate_up^T, act silu unless the specification says otherwise.  The reference concatenates gate rows
     and up rows; ``spec.interleave`` may instead ask for blocks of 8 gate rows and 8 up rows, so that
     the product's epilogue applies the gate when a step has few rows."""
 
@@ -17,6 +17,9 @@ class SwiGLU(FeedForward):
         super().__init__(spec, env)
         if spec.interleave not in (0, 8) or (spec.interleave and spec.intermediate_size % spec.interleave):
             raise ValueError("interleave is 0, or 8 with intermediate_size a multiple of 8")
+        self.gate = getattr(spec, "activation", "silu")
+        if self.gate not in ops.GATES:
+            raise ValueError(f"activation={self.gate!r}; known: {sorted(ops.GATES)}")
 
     def params(self):
         s = self.spec
@@ -32,7 +35,7 @@ class SwiGLU(FeedForward):
         s = self.spec
         T = x.shape[0]
         act = work_buffer(ctx, "mlp.act", (T, s.intermediate_size), x.dtype, x.device)
-        ops.gated_linear(x, self.p_gate_up, act, s.interleave, ctx)
+        ops.gated_linear(x, self.p_gate_up, act, s.interleave, ctx, self.gate)
         y = work_buffer(ctx, "mlp.y", (T, s.hidden_size), x.dtype, x.device)
         ops.linear(act, self.p_down, y)
         return y

@@ -126,6 +126,16 @@ class AttentionSpec:
     # elements meet zero columns of the output projection), so one cache layout and one set of kernels serve them.
     key_dim: Optional[int] = None
     value_dim: Optional[int] = None
+    # Options of the score, each off unless given.  ``keep_first`` n: beside the window a query sees the sequence's first n
+    # keys.  ``softcap``: a scaled score s becomes cap tanh(s / cap).  ``sink``: a learned number per head whose exponential
+    # joins the softmax's denominator.
+    keep_first: int = 0
+    softcap: Optional[float] = None
+    sink: bool = False
+    # ``value_mix`` "source": the layer's values serve the later layers of a step; "blend": the values that are cached are
+    # (1 - share) v + share v_source with one learned number, ``v_source`` those of the layer before it in the schedule that
+    # says "source" (as many key/value heads, values of the same size)
+    value_mix: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -332,13 +342,14 @@ class ParallelBlockSpec:
 
 @dataclass(frozen=True)
 class SwiGLUSpec:
-    """down( silu(gate(x)) * up(x) ), dense.  ``interleave``: row layout of the fused gate_up weight:
+    """down( act(gate(x)) * up(x) ), dense; ``activation``: "silu" or "gelu_tanh".  ``interleave``: row layout of the fused gate_up weight:
     0 = all gate rows then all up rows; 8 = blocks of 8 gate rows then their 8 up rows, which lets
     the product's epilogue apply the gate (needs intermediate_size % 8 == 0)."""
     hidden_size: int
     intermediate_size: int
     interleave: int = 0
     kind: str = "swiglu"
+    activation: str = "silu"
 
 
 @dataclass(frozen=True)
@@ -369,8 +380,9 @@ class MoESpec:
     form that many equal groups of neighbours and only those of the ``keep_groups`` groups with the largest best score
     can be chosen; the chosen scores divided by their sum (+ ``renorm_tiny``) weigh the experts' outputs (with
     ``renorm_tiny`` = 0 that is the softmax over the chosen logits alone).  ``router_bias``: a bias per expert is added to
-    the logits.  ``expert`` is a ``ClampedGLUSpec`` or a ``SwiGLUSpec`` with rows not woven.  ``shared``: a feed-forward
-    that runs for every token and is added, or None.  ``score`` "sigmoid": every expert's score is the logistic of its own
+    the logits.  ``expert`` is a ``ClampedGLUSpec``, a ``SwiGLUSpec`` (silu) with rows not woven, or a ``DenseMLPSpec`` (no
+    gate).  ``shared``: a feed-forward that runs for every token and is added, or None; ``shared_gate``: what it gives is
+    first multiplied by the logistic of one projected number per token (its row stands behind the router's).  ``score`` "sigmoid": every expert's score is the logistic of its own
     logit instead of a softmax over all.  ``group_top`` 2: a group is ranked by the sum of its two largest scores instead of
     its largest.  ``weight_scale``: a factor on the weights after they were divided by their sum.  ``renormalize`` False: the
     chosen scores are the weights as they are.  ``weigh_input`` True: a weight multiplies its expert's input instead of its
@@ -390,6 +402,7 @@ class MoESpec:
     weight_scale: float = 1.0
     renormalize: bool = True
     weigh_input: bool = False
+    shared_gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -408,6 +421,17 @@ class SandwichBlockSpec:
     layer_scale: bool = False
     token_shift: bool = False
     kind: str = "sandwich"
+
+
+@dataclass(frozen=True)
+class PostNormBlockSpec:
+    """x += norm_a(mixer(x)); x += norm_b(feed_forward(x)): the sublayers read the stream itself, their outputs are normed
+    before they join it.  ``feed_forward`` None: the layer has none (and no norm for it).  The norms are RMSNorms."""
+    mixer: Any
+    feed_forward: Any
+    mixer_post_norm: Any
+    feed_forward_post_norm: Any = None
+    kind: str = "postnorm"
 
 
 @dataclass(frozen=True)
