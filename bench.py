@@ -92,10 +92,10 @@ def main():
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--only", default="all", choices=["all", "decode", "prefill"],
                     help="a reduced run for profiling: only the decode steps, or only the prefill")
-    ap.add_argument("--design", default=None, choices=["pisatar", "gonozen", "nozizen", "duvadra", "losorax"],
+    ap.add_argument("--design", default=None, choices=["pisatar", "gonozen", "nozizen", "duvadra", "losorax", "sizudra"],
                     help="instead of the default workload: prefill and decode throughput of this design beside the Qwen3 "
                          "decoder (nozizen: beside the Pisatar decoder; duvadra: beside the Nozizen decoder; losorax: beside the "
-                         "Duvadra decoder) at equal layer sizes (--sizes), random weights, one JSON line")
+                         "Duvadra decoder; sizudra: beside the Gonozen decoder too) at equal layer sizes (--sizes), random weights, one JSON line")
     ap.add_argument("--sizes", default="1k,2k", help="with --design: names of return_b200.benchmark.DESIGN_SIZES")
     ap.add_argument("--kernels", action="store_true",
                     help="with --impl reference: time the reference's Triton kernels alone, one JSON line each")
@@ -122,8 +122,10 @@ def main():
         clocks = ClockSampler()
         clocks.start()
         compare = {"gonozen": benchmark.compare_gonozen, "nozizen": benchmark.compare_nozizen,
-                   "duvadra": benchmark.compare_duvadra, "losorax": benchmark.compare_losorax}.get(args.design, benchmark.compare_designs)
-        beside = {"nozizen": "Pisatar", "duvadra": "Nozizen", "losorax": "Duvadra"}.get(args.design, "Qwen3") + " at equal width, feed-forward, layers and heads"
+                   "duvadra": benchmark.compare_duvadra, "losorax": benchmark.compare_losorax,
+                   "sizudra": benchmark.compare_sizudra}.get(args.design, benchmark.compare_designs)
+        beside = {"nozizen": "Pisatar", "duvadra": "Nozizen", "losorax": "Duvadra",
+                  "sizudra": "Qwen3 and Gonozen"}.get(args.design, "Qwen3") + " at equal width, feed-forward, layers and heads"
         rows = [compare(size, PROMPT_LEN, args.batch, K, W, hbm_gbs, bf16_tflops) for size in args.sizes.split(",")]
         print(json.dumps({"design": args.design, "beside": beside,
                           "dtype": "bf16", "data": "synthetic: random weights, uniform random token ids", "steps": K,

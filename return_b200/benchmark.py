@@ -996,3 +996,97 @@ def compare_losorax(size: str, tokens: int, batch: int, steps: int, warmup: int,
         del r["prefill_kernels"], r["decode_kernels"]
     return {"size": size, "width": W, "ff": ff, "heads": H, "kv_heads": G, "layers": L, "tokens": tokens, "batch": batch,
             "bias_rows": 32, "bias_max": 1024, "losorax": new, "duvadra": old, "kernels": kernels}
+
+
+def sizudra_raw_config(width: int, ff: int, heads: int, kv_heads: int, layers: int, vocab: int, window: int = 1024,
+                       keep_first: int = 16) -> dict:
+    """A Sizudra configuration with the attention heads of a Qwen3 model of this width (128 elements, half of them rotated,
+    values blended with the first layer's): every other layer sees all keys, the others a window of 1,024 and the first 16,
+    scores capped at 30 and a sink; of every four feed-forwards two are dense, two are 32 experts of half of the dense
+    size each, four of them a token (two matrices instead of a gated unit's three, so a token's experts do a third more
+    than the dense one's work), beside a shared one of the same size."""
+    dense = {"kind": "dense", "ff": ff}
+    experts = {"kind": "moe", "router": {"experts": 32, "top": 4}, "expert": {"ff": ff // 2}, "shared": {"ff": ff // 2}}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "v_mix": True,
+           "rot": {"base": 1e6, "dims": 64}}
+    windowed = dict(att, mask={"size": window, "keep_first": keep_first}, softcap=30.0)
+    return {"architecture": "Sizudra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}},
+            "layers": [{"type": "attention_2" if i % 2 else "attention", "mixer": windowed if i % 2 else att,
+                        "mlp": experts if i % 4 in (1, 2) else dense} for i in range(layers)]}
+
+
+def compare_sizudra(size: str, tokens: int, batch: int, steps: int, warmup: int, hbm_gbs: float, bf16_tflops: float):
+    """The Sizudra design beside its two nearest at equal width, feed-forward, layer count and heads: the Qwen3 decoder (the
+    same attention without the options, dense gated units) and the Gonozen decoder (experts with a shared one, norms behind
+    the sublayers, a window and a sink).  Throughput of all three, and how far the kernels of each mechanism are from their
+    rooflines beside the like kernels of the others.  Rooflines: attention over decoded tokens against the copy bandwidth
+    (the keys and values a query sees read once), over a prompt against the tensor peak (the causal half, or the window's
+    band and the kept keys), layers with and without score options apart; the kernel that norms, rotates, blends and caches
+    (projections read, queries and pages written) and the joints of two sublayers (float32 stream read and written, the
+    sublayer's output read, the next one's input written) against the copy bandwidth; the experts' products of a prompt
+    against the tensor peak and of decoded tokens against the copy bandwidth (each reached expert read once); the gated
+    product of a prompt against the tensor peak."""
+    from .config.gonozen_config import GonozenConfig
+    from .config.model_config import Qwen3Config
+    from .config.sizudra_config import SizudraConfig
+    sz = DESIGN_SIZES[size]
+    W, ff, H, G, L, V = sz["width"], sz["ff"], sz["heads"], sz["kv_heads"], sz["layers"], sz["vocab"]
+    raw, gon_raw = sizudra_raw_config(W, ff, H, G, L, V), gonozen_raw_config(W, ff, H, L, V)
+    new = measure_design(SizudraConfig(raw), tokens, batch, steps, warmup)
+    qwen = measure_design(Qwen3Config.from_dict(dict(vocab_size=V, hidden_size=W, intermediate_size=ff, num_hidden_layers=L,
+                                                     num_attention_heads=H, num_key_value_heads=G, head_dim=128,
+                                                     rope_theta=1e6, rms_norm_eps=1e-6, tie_word_embeddings=False,
+                                                     max_position_embeddings=32768)), tokens, batch, steps, warmup)
+    gon = measure_design(GonozenConfig(gon_raw), tokens, batch, steps, warmup)
+    D, E, top, F, FG = 128, 32, 4, ff // 2, ff // 4
+    window, keep = raw["layers"][1]["mixer"]["mask"]["size"], raw["layers"][1]["mixer"]["mask"]["keep_first"]
+    n_win = sum(1 for layer in raw["layers"] if layer["type"] == "attention_2")
+    n_full = L - n_win
+    n_moe = sum(1 for layer in raw["layers"] if layer["mlp"]["kind"] == "moe")
+    seen = min(tokens, window + keep)
+    band = tokens * tokens / 2 if window >= tokens else tokens * window - window * window / 2 + keep * (tokens - window)
+    distinct = E * (1.0 - (1.0 - 1.0 / E) ** (batch * top))
+    frac = lambda work, ms, peak: round(work / (ms * 1e-3) / peak, 4) if ms > 0 else None
+    hbm, peak = hbm_gbs * 1e9, bf16_tflops * 1e12
+    row = lambda times, names, work, roof, key: {"ms": round(_kernel_ms(times, *names), 4), key: frac(work, _kernel_ms(times, *names), roof)}
+    k_new, k_q, k_g = new["prefill_kernels"], qwen["prefill_kernels"], gon["prefill_kernels"]
+    d_new, d_q, d_g = new["decode_kernels"], qwen["decode_kernels"], gon["decode_kernels"]
+    moe_pf, moe_dec = ("moe_grouped_gemm", "moe_tc5"), ("moe_pair_linear", "moe_grouped_gemm")
+    kv_bytes = 2.0 * 2 * G * D * batch
+    rows_bytes = 2.0 * D * 2 * (H + 2 * G) * tokens                   # a layer's projections read, queries and pages written
+    joint_bytes = 2.0 * L * tokens * W * (2 * 4 + 2 + 2)
+    kernels = {
+        "decode_attention_full_sizudra": row(d_new, ("attn_decode_kernel<true, false>",), kv_bytes * tokens * n_full, hbm, "of_hbm"),
+        "decode_attention_windowed_sizudra": row(d_new, ("attn_decode_kernel<true, true>",), kv_bytes * seen * n_win, hbm, "of_hbm"),
+        "decode_attention_qwen3": row(d_q, ("attn_decode_kernel",), kv_bytes * tokens * L, hbm, "of_hbm"),
+        "decode_combine_sizudra": row(d_new, ("attn_combine",), 0.0, hbm, "of_hbm"),
+        "decode_combine_qwen3": row(d_q, ("attn_combine",), 0.0, hbm, "of_hbm"),
+        "prefill_attention_full_sizudra": row(k_new, ("attn_prefill_tc5_kernel<false>",), 4.0 * tokens * tokens / 2 * H * D * n_full, peak, "of_bf16_peak"),
+        "prefill_attention_windowed_sizudra": row(k_new, ("attn_prefill_tc5_kernel<true>",), 4.0 * band * H * D * n_win, peak, "of_bf16_peak"),
+        "prefill_attention_qwen3": row(k_q, ("attn_prefill_tc5",), 4.0 * tokens * tokens / 2 * H * D * L, peak, "of_bf16_peak"),
+        "prefill_rows_sizudra": row(k_new, ("qk_norm_rope_write",), rows_bytes * L + 2.0 * D * G * tokens * (L - 1), hbm, "of_hbm"),
+        "prefill_rows_qwen3": row(k_q, ("qk_norm_rope_write",), rows_bytes * L, hbm, "of_hbm"),
+        "prefill_joint_sizudra": row(k_new, ("postnorm_add_norm",), joint_bytes, hbm, "of_hbm"),
+        "prefill_joint_gonozen": row(k_g, ("postnorm_add_norm",), joint_bytes, hbm, "of_hbm"),
+        "prefill_add_norm_qwen3": row(k_q, ("add_rmsnorm",), joint_bytes, hbm, "of_hbm"),
+        "prefill_gated_product_sizudra": row(k_new, ("tc5_gemm_pair",), (L - n_moe) * 4.0 * tokens * ff * W, peak, "of_bf16_peak"),
+        "prefill_gated_product_qwen3": row(k_q, ("tc5_gemm_pair",), L * 4.0 * tokens * ff * W, peak, "of_bf16_peak"),
+        "prefill_experts_sizudra": row(k_new, moe_pf, n_moe * 2.0 * tokens * top * 2 * F * W, peak, "of_bf16_peak"),
+        "prefill_experts_gonozen": row(k_g, moe_pf, L * 2.0 * tokens * top * 3 * FG * W, peak, "of_bf16_peak"),
+        "decode_experts_sizudra": row(d_new, moe_dec, n_moe * 2.0 * distinct * 2 * F * W, hbm, "of_hbm"),
+        "decode_experts_gonozen": row(d_g, moe_dec, L * 2.0 * distinct * 3 * FG * W, hbm, "of_hbm"),
+        # what combines the experts' outputs with the shared one's: the pairs' rows and the shared row read, one written
+        "prefill_combine_sizudra": row(k_new, ("moe_combine",), n_moe * 2.0 * tokens * (top + 2) * W, hbm, "of_hbm"),
+        "prefill_combine_gonozen": row(k_g, ("moe_combine",), L * 2.0 * tokens * (top + 2) * W, hbm, "of_hbm"),
+    }
+    for name, names in (("joints", ("postnorm_add_norm", "add_rmsnorm")), ("weight_streaming", ("gemm_skinny",)),
+                        ("expert_helpers", ("moe_combine", "moe_route", "moe_sort", "moe_gather", "clamped_glu", "activation"))):
+        for model, pf, dec in (("sizudra", k_new, d_new), ("qwen3", k_q, d_q), ("gonozen", k_g, d_g)):
+            kernels[f"decode_{name}_{model}"] = {"ms": round(_kernel_ms(dec, *names), 4)}
+            if name == "expert_helpers":
+                kernels[f"prefill_{name}_{model}"] = {"ms": round(_kernel_ms(pf, *names), 4)}
+    for r in (new, qwen, gon):
+        del r["prefill_kernels"], r["decode_kernels"]
+    return {"size": size, "width": W, "ff": ff, "heads": H, "kv_heads": G, "layers": L, "tokens": tokens, "batch": batch,
+            "window": window, "keep_first": keep, "sizudra": new, "qwen3": qwen, "gonozen": gon, "kernels": kernels}

@@ -108,11 +108,28 @@ struct ScoreMod {
     int bias_n;
     int keep;                  // with a window: the first `keep` positions stay visible (0: none)
 };
-// `brow`: the head's row of the bias table for a distance that may lie within it, or null: then `blast` (its last entry,
-// or zero without a table) is added.
-__device__ __forceinline__ float mod_score(float dot, const ScoreMod& sm, float slope, int dist, const float* brow, float blast) {
-    float v = dot * sm.scale;
-    if (sm.softcap > 0.f) v = sm.softcap * fast_tanh(v / sm.softcap);
+// Caps N scores (dot products) of a thread: v <- the scaled score through the cap, in natural units.  Where all of a warp's are
+// well below the cap the tanh is a polynomial (tanh_poly in common.cuh), else fast_tanh.
+template <int N>
+__device__ __forceinline__ void cap_scores(float (&v)[N], const ScoreMod& sm) {
+    const float k = sm.scale / sm.softcap;
+    float top = 0.f;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        v[i] *= k;
+        top = fmaxf(top, fabsf(v[i]));
+    }
+    if (!__any_sync(0xffffffffu, !(top <= TANH_POLY_MAX))) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = sm.softcap * tanh_poly(v[i]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = sm.softcap * fast_tanh(v[i]);
+    }
+}
+// What comes after the cap: the distance's penalty and bias, and the units of log2.  `brow`: the head's row of the bias table
+// for a distance that may lie within it, or null: then `blast` (its last entry, or zero without a table) is added.
+__device__ __forceinline__ float mod_score(float v, const ScoreMod& sm, float slope, int dist, const float* brow, float blast) {
     v = fmaf(-slope, (float)dist, v);
     v += brow != nullptr ? __ldg(brow + min(max(dist, 0), sm.bias_n - 1)) : blast;
     return v * LOG2E;
@@ -284,6 +301,14 @@ attn_prefill_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__
             // scale, mask, running maximum
             const float* brow = (MOD && p0 + wrow - (j_base + PF_N - 1) < sm.bias_n - 1) ? bias_row : nullptr;
             float mx0 = -INFINITY, mx1 = -INFINITY;
+            if (MOD) {
+                if (sm.softcap > 0.f) {
+                    cap_scores(reinterpret_cast<float(&)[PF_N / 2]>(s), sm);
+                } else {
+#pragma unroll
+                    for (int nt = 0; nt < PF_N / 8; ++nt) { s[nt][0] *= sm.scale; s[nt][1] *= sm.scale; s[nt][2] *= sm.scale; s[nt][3] *= sm.scale; }
+                }
+            }
 #pragma unroll
             for (int nt = 0; nt < PF_N / 8; ++nt) {
 #pragma unroll
@@ -570,12 +595,12 @@ attn_decode_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__ 
                     const bf16* vs = tok + (size_t)(Hq + Hkv + kvh) * D;
                     if (fr.v_first != nullptr) {
                         const bf16* vf = fr.v_first + (size_t)tok_row * fr.v_first_ld + (size_t)kvh * fr.v_first_head_stride;
-                        const float share = load_as_f32(fr.v_share, fr.v_share_dtype, 0), own = 1.0f - share;
+                        const float share = load_as_f32(fr.v_share, fr.v_share_dtype, 0);
                         for (int i = 2 * lane; i < D; i += 64) {
                             const float2 v = ld_pair(vs + i);
                             const float f0 = i < fr.v_first_n ? __bfloat162float(vf[i]) : 0.f;
                             const float f1 = i + 1 < fr.v_first_n ? __bfloat162float(vf[i + 1]) : 0.f;
-                            st_pair(fr.vpool + slot + i, make_float2(own * v.x + share * f0, own * v.y + share * f1));
+                            st_pair(fr.vpool + slot + i, make_float2(rb_blend(v.x, f0, share), rb_blend(v.y, f1, share)));
                         }
                     } else {
                         for (int ch = lane; ch < CHUNKS; ch += 32)
@@ -649,20 +674,46 @@ attn_decode_kernel(const bf16* __restrict__ q, int ld, const bf16* __restrict__ 
         }
         float mx0 = -INFINITY, mx1 = -INFINITY;
         if (MOD) {
-            const float sl0 = (sm.slopes && g < rows_valid) ? sm.slopes[h0 + g] : 0.f;
-            const float sl1 = (sm.slopes && g + 8 < rows_valid) ? sm.slopes[h0 + g + 8] : 0.f;
-            const bool near = hi - (j_base + DC_N - 1) < sm.bias_n - 1;           // the tile holds distances within the table
-            const float* br0 = near ? bias0 : nullptr;
-            const float* br1 = near ? bias1 : nullptr;
+            // the scores in units of log2; rows 8 to 15 of the tile only if they are query heads
+            const bool upper = rows_valid > 8;
+            float v0[4] = {s[0][0] + s2[0][0], s[0][1] + s2[0][1], s[1][0] + s2[1][0], s[1][1] + s2[1][1]};       // row g
+            float v1[4] = {s[0][2] + s2[0][2], s[0][3] + s2[0][3], s[1][2] + s2[1][2], s[1][3] + s2[1][3]};       // row g + 8
+            if (sm.softcap > 0.f) {
+                cap_scores(v0, sm);
+                if (upper) cap_scores(v1, sm);
+            }
+            const float unit = sm.softcap > 0.f ? LOG2E : scale_log2;
+            if (sm.slopes != nullptr || sm.bias != nullptr) {
+                const float natural = sm.softcap > 0.f ? 1.f : sm.scale;
+                const float sl0 = (sm.slopes && g < rows_valid) ? sm.slopes[h0 + g] : 0.f;
+                const float sl1 = (sm.slopes && g + 8 < rows_valid) ? sm.slopes[h0 + g + 8] : 0.f;
+                const bool near = hi - (j_base + DC_N - 1) < sm.bias_n - 1;           // the tile holds distances within the table
+                const float* br0 = near ? bias0 : nullptr;
+                const float* br1 = near ? bias1 : nullptr;
 #pragma unroll
-            for (int nt = 0; nt < 2; ++nt) {
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int j = j_base + nt * 8 + 2 * t4 + (e & 1);
-                    const float v = ((j >= lo || j < keep) && j <= hi) ? mod_score(s[nt][e] + s2[nt][e], sm, (e & 2) ? sl1 : sl0, hi - j, (e & 2) ? br1 : br0, (e & 2) ? last1 : last0) : -INFINITY;
-                    s[nt][e] = v;
-                    if (e & 2) mx1 = fmaxf(mx1, v); else mx0 = fmaxf(mx0, v);
+                for (int i = 0; i < 4; ++i) {
+                    const int dist = hi - (j_base + (i >> 1) * 8 + 2 * t4 + (i & 1));
+                    v0[i] = mod_score(natural * v0[i], sm, sl0, dist, br0, last0);
+                    v1[i] = mod_score(natural * v1[i], sm, sl1, dist, br1, last1);
                 }
+            } else {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) { v0[i] *= unit; v1[i] *= unit; }
+            }
+            const bool whole = (j_base >= lo || j_base + DC_N <= keep) && j_base + DC_N - 1 <= hi;      // every key of the tile is visible
+            if (!whole) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int j = j_base + (i >> 1) * 8 + 2 * t4 + (i & 1);
+                    if (!((j >= lo || j < keep) && j <= hi)) v0[i] = v1[i] = -INFINITY;
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                s[i >> 1][i & 1] = v0[i];
+                s[i >> 1][2 + (i & 1)] = v1[i];
+                mx0 = fmaxf(mx0, v0[i]);
+                mx1 = fmaxf(mx1, v1[i]);
             }
         } else if (j_base >= lo && j_base + DC_N - 1 <= hi) {            // every key of the tile is visible
 #pragma unroll

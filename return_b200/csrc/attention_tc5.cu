@@ -40,7 +40,9 @@
 // with the distance, slopes[h] * (i - j), taken off before the softmax, and a bias per head and distance added to the
 // score, bias[h, min(i - j, bias_n - 1)]: only key tiles within the table's reach look it up (neighbouring rows read
 // neighbouring entries), behind it the last entry is a constant.  A row's thread does that to its 64 scores
-// of a key tile right after it has read them from tensor memory; everything else is the plain kernel.  With a window it can
+// of a key tile right after it has read them from tensor memory; everything else is the plain kernel.  A capped score needs a
+// tanh: where all of a warp's scores of a tile are well below the cap it is a polynomial, two scores an instruction
+// (tanh_poly in common.cuh); else the hardware's 2^x and reciprocal, which take as long as the softmax's own three times over.  With a window it can
 // also keep the first `keep` positions visible for every later query: the key tiles are then walked in two runs, the tiles
 // of the kept positions that lie before the window's first tile, then the window's.
 // A step with too few such CTAs to fill the GPU (a short portion of a long prompt) splits the keys of every
@@ -109,6 +111,11 @@ __device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigne
 __device__ __forceinline__ unsigned long long add2(unsigned long long a, unsigned long long b) {
     unsigned long long d;
     asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b) {
+    unsigned long long d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
     return d;
 }
 __device__ __forceinline__ float max3(float a, float b, float c) {
@@ -237,9 +244,14 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
         const bool full_tile = m_rows >= (qt + 1) * QM;
         const int lo_r = chunk > 0 ? (pos_r / chunk) * chunk : 0;               // the first key of this row's own block
         const float slope = (MOD && sm.slopes) ? sm.slopes[h] : 0.f;
-        const float scale_eff = MOD ? 1.f : scale_log2;                        // the MOD rows hold finished exponents
+        // The softmax's 2^x takes scale_eff * a[i] - m.  Without a penalty or bias a[i] is the raw product, or the tanh of the
+        // capped score; with one it is the finished exponent.
+        const bool capped = MOD && sm.softcap > 0.f;
+        const bool finished = MOD && (sm.slopes != nullptr || sm.bias != nullptr);
         const float cap_l = MOD ? sm.softcap * LOG2E : 0.f, slope_l = slope * LOG2E;
-        const float k_tanh = (MOD && sm.softcap > 0.f) ? sm.scale / sm.softcap * (2.0f * LOG2E) : 0.f;
+        const float scale_eff = finished ? 1.f : capped ? cap_l : scale_log2;
+        const float k_cap = capped ? sm.scale / sm.softcap : 0.f;              // a raw product times this is the tanh's argument
+        const float raw_max = capped ? TANH_POLY_MAX / k_cap : 0.f;            // up to this product the polynomial holds
         const float* bias_row = (MOD && sm.bias) ? sm.bias + (size_t)h * sm.bias_n : nullptr;
         const float bias_last_l = (MOD && sm.bias) ? bias_row[sm.bias_n - 1] * LOG2E : 0.f;
         unsigned char* myQ = sQ + qt * Q_BYTES;
@@ -272,40 +284,62 @@ attn_prefill_tc5_kernel(const bf16* __restrict__ q, int ld, const bf16* __restri
             tmem_ld_wait();
             float mx = -INFINITY;
             if (MOD) {
-                // the finished exponent of key j = j_base + i, in units of log2:
-                //   cap L tanh(s scale / cap) - slope L (pos - j)  =  cap L - 2 cap L / (e^(2 s scale / cap) + 1) + slope L i - slope L (pos - j_base)
-                // with L = log2(e): one product, 2^x, one sum, a reciprocal and two fused products a score
-                const bool near = sm.bias != nullptr && p0_t - (j_base + KN - 1) < sm.bias_n - 1;   // the tile holds distances within the table
-                const float c0 = cap_l - slope_l * (float)(pos_r - j_base) + (near ? 0.f : bias_last_l);
-                if (sm.softcap > 0.f) {
+                if (capped) {
+                    float top = 0.f;
 #pragma unroll
-                    for (int i = 0; i < 64; ++i) {
-                        float e;
-                        asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(__uint_as_float(a[i]) * k_tanh));
-                        float rc;
-                        asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(rc) : "f"(e + 1.f));
-                        a[i] = __float_as_uint(fmaf(-2.f * cap_l, rc, fmaf(slope_l, (float)i, c0)));
+                    for (int i = 0; i < 64; i += 2) top = fmaxf(top, fmaxf(fabsf(__uint_as_float(a[i])), fabsf(__uint_as_float(a[i + 1]))));
+                    if (!__any_sync(0xffffffffu, !(top <= raw_max))) {
+                        const unsigned long long k2 = pack2(k_cap, k_cap);
+#pragma unroll
+                        for (int i = 0; i < 64; i += 2) {
+                            const unsigned long long x = mul2(pack2(__uint_as_float(a[i]), __uint_as_float(a[i + 1])), k2), u = mul2(x, x);
+                            unsigned long long t = fma2(u, pack2(TANH_P4, TANH_P4), pack2(TANH_P3, TANH_P3));
+                            t = fma2(u, t, pack2(TANH_P2, TANH_P2));
+                            t = fma2(u, t, pack2(TANH_P1, TANH_P1));
+                            t = mul2(x, fma2(u, t, pack2(TANH_P0, TANH_P0)));
+                            float t0, t1;
+                            unpack2(t, t0, t1);
+                            a[i] = __float_as_uint(t0);
+                            a[i + 1] = __float_as_uint(t1);
+                        }
+                    } else {
+                        // tanh(x) = 1 - 2 / (e^(2 x) + 1)
+#pragma unroll
+                        for (int i = 0; i < 64; ++i) {
+                            float e, rc;
+                            asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(__uint_as_float(a[i]) * (k_cap * 2.0f * LOG2E)));
+                            asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(rc) : "f"(e + 1.f));
+                            a[i] = __float_as_uint(fmaf(-2.f, rc, 1.f));
+                        }
                     }
-                } else {
-#pragma unroll
-                    for (int i = 0; i < 64; ++i)
-                        a[i] = __float_as_uint(fmaf(__uint_as_float(a[i]), sm.scale * LOG2E, fmaf(slope_l, (float)i, c0)));
                 }
-                if (near) {
-                    const int d0 = pos_r - j_base;
+                if (finished) {
+                    // the exponent of key j = j_base + i, in units of log2: the (capped) score - slope (pos - j) + bias(pos - j)
+                    const bool near = sm.bias != nullptr && p0_t - (j_base + KN - 1) < sm.bias_n - 1;   // the tile holds distances within the table
+                    const float c0 = (near ? 0.f : bias_last_l) - slope_l * (float)(pos_r - j_base);
+                    const float unit = capped ? cap_l : scale_log2;
 #pragma unroll
                     for (int i = 0; i < 64; ++i)
-                        a[i] = __float_as_uint(fmaf(__ldg(bias_row + min(max(d0 - i, 0), sm.bias_n - 1)), LOG2E, __uint_as_float(a[i])));
+                        a[i] = __float_as_uint(fmaf(__uint_as_float(a[i]), unit, fmaf(slope_l, (float)i, c0)));
+                    if (near) {
+                        const int d0 = pos_r - j_base;
+#pragma unroll
+                        for (int i = 0; i < 64; ++i)
+                            a[i] = __float_as_uint(fmaf(__ldg(bias_row + min(max(d0 - i, 0), sm.bias_n - 1)), LOG2E, __uint_as_float(a[i])));
+                    }
                 }
                 if (all_visible) {
 #pragma unroll
                     for (int i = 0; i < 64; i += 2) mx = max3(mx, __uint_as_float(a[i]), __uint_as_float(a[i + 1]));
                 } else {
+                    // which of the tile's keys this row sees, as bits: not behind the row, and in the window (or the block) or kept
+                    auto below = [](int n) { return n <= 0 ? 0ull : n >= 64 ? ~0ull : (1ull << n) - 1ull; };      // keys before n
+                    const int lo_i = max(window > 0 ? pos_r - window + 1 : 0, lo_r) - j_base;
+                    const unsigned long long vis = row_valid ? below(pos_r + 1 - j_base) & (~below(lo_i) | below(keep - j_base)) : 0ull;
+                    const unsigned vis_lo = (unsigned)vis, vis_hi = (unsigned)(vis >> 32);
 #pragma unroll
                     for (int i = 0; i < 64; ++i) {
-                        const int j = j_base + i;
-                        const bool vis = row_valid && j <= pos_r && (window <= 0 || j > pos_r - window || j < keep) && j >= lo_r;
-                        if (!vis) a[i] = 0xff800000u;
+                        if (!((i < 32 ? vis_lo : vis_hi) & (1u << (i & 31)))) a[i] = 0xff800000u;
                         mx = fmaxf(mx, __uint_as_float(a[i]));
                     }
                 }

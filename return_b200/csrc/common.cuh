@@ -87,6 +87,23 @@ __device__ __forceinline__ float rb_gate_arg(int gate, float g) {
     return gate == GATE_GELU_TANH ? 1.5957691216057308f * fmaf(0.044715f * g * g, g, g) : g;
 }
 
+// A value blended with another layer's, with one order of rounding wherever it is worked out.
+__device__ __forceinline__ float rb_blend(float v, float first, float share) { return fmaf(share, first, (1.0f - share) * v); }
+
+// tanh(x) = x P(x^2) for |x| <= TANH_POLY_MAX: a polynomial fitted to tanh(x) / x for the smallest largest absolute error of
+// tanh (least squares reweighted by the error, 9e-8; 1.5e-7 with float32 arithmetic).  No special-function unit is involved,
+// which is what counts where every score of an attention is capped.
+#define TANH_POLY_MAX 0.7f
+#define TANH_P0 0.99999851f
+#define TANH_P1 -0.333269745f
+#define TANH_P2 0.132574588f
+#define TANH_P3 -0.0501953885f
+#define TANH_P4 0.0131943217f
+__device__ __forceinline__ float tanh_poly(float x) {
+    const float u = x * x;
+    return x * fmaf(fmaf(fmaf(fmaf(TANH_P4, u, TANH_P3), u, TANH_P2), u, TANH_P1), u, TANH_P0);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

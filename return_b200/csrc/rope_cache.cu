@@ -121,17 +121,17 @@ __global__ void qk_norm_rope_write_kernel(
             TA* dst = vpool + slot_base + (long long)(hh - Hq - Hkv) * page_size * D;
             if (vm.first != nullptr) {
                 const TA* vf = (const TA*)vm.first + (size_t)t * vm.ld + (size_t)(hh - Hq - Hkv) * vm.head_stride;
-                const float share = load_as_f32(vm.share, vm.share_dtype, 0), own = 1.0f - share;
+                const float share = load_as_f32(vm.share, vm.share_dtype, 0);
 #pragma unroll
                 for (int j = 0; j < ROPE_MAX_J; ++j) {
                     const int i = 2 * lane + 64 * j;
                     if (i < D) {
                         const float f0 = i < vm.n ? to_f32(vf[i]) : 0.f, f1 = i + 1 < vm.n ? to_f32(vf[i + 1]) : 0.f;
-                        a[u][j] = make_float2(own * a[u][j].x + share * f0, own * a[u][j].y + share * f1);
+                        a[u][j] = make_float2(rb_blend(a[u][j].x, f0, share), rb_blend(a[u][j].y, f1, share));
                     }
                     if (i + 128 < D) {
                         const float f0 = i + 128 < vm.n ? to_f32(vf[i + 128]) : 0.f, f1 = i + 129 < vm.n ? to_f32(vf[i + 129]) : 0.f;
-                        b[u][j] = make_float2(own * b[u][j].x + share * f0, own * b[u][j].y + share * f1);
+                        b[u][j] = make_float2(rb_blend(b[u][j].x, f0, share), rb_blend(b[u][j].y, f1, share));
                     }
                 }
             }
@@ -282,7 +282,7 @@ qk_norm_rope_write_vec_kernel(
             bf16* dst = vpool + slot_base + (long long)(hh - Hq - Hkv) * page_size * D;
             if (vm.first != nullptr) {
                 const bf16* vf = (const bf16*)vm.first + (size_t)t * vm.ld + (size_t)(hh - Hq - Hkv) * vm.head_stride;
-                const float share = load_as_f32(vm.share, vm.share_dtype, 0), own = 1.0f - share;
+                const float share = load_as_f32(vm.share, vm.share_dtype, 0);
                 float f1[8], f2[8];
                 if (i1 + 8 <= vm.n) unpack8(*reinterpret_cast<const uint4*>(vf + i1), f1);
                 else {
@@ -295,7 +295,7 @@ qk_norm_rope_write_vec_kernel(
                     for (int i = 0; i < 8; ++i) f2[i] = i2 + i < vm.n ? __bfloat162float(vf[i2 + i]) : 0.f;
                 }
 #pragma unroll
-                for (int i = 0; i < 8; ++i) { x1[i] = own * x1[i] + share * f1[i]; x2[i] = own * x2[i] + share * f2[i]; }
+                for (int i = 0; i < 8; ++i) { x1[i] = rb_blend(x1[i], f1[i], share); x2[i] = rb_blend(x2[i], f2[i], share); }
                 a[r] = pack8(x1);
                 b[r] = pack8(x2);
             }

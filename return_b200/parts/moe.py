@@ -91,6 +91,8 @@ class MixtureOfExperts(FeedForward):
     def bind(self, tensors):
         s, e = self.spec, self.spec.expert
         self.p_router = tensors["router"]
+        if self.p_router.dtype == torch.bfloat16 and self.p_router.shape[0] % 8:      # whole 16-byte pieces: other logits, unread
+            self.p_router = torch.nn.functional.pad(self.p_router, (0, 0, 0, -self.p_router.shape[0] % 8))
         self.router_bias = tensors["router_bias"].float().contiguous() if s.router_bias else None
         self.up = tensors[self.up_name].view(s.num_experts, self._up_rows(), s.hidden_size)
         self.down = tensors["experts.down"].view(s.num_experts, s.hidden_size, e.intermediate_size)
