@@ -211,28 +211,32 @@ def _copies_beyond_l2(nbytes: int, l2_bytes: int = 126 << 20) -> int:
 
 
 def kernel_attention_decode(batch=64, ctx=2048, heads=32, kv_heads=8, head_dim=128, page=16, splits=0,
-                            iters=10, warmup=3) -> Dict[str, float]:
-    """The split-KV decode attention kernel alone: device time and the bandwidth of the keys and values it reads."""
+                            iters=10, warmup=3, window=0, keep=0, softcap=0.0) -> Dict[str, float]:
+    """The split-KV decode attention kernel alone: device time and the bandwidth of the keys and values it reads.
+    ``window``, ``keep``, ``softcap``: the score options of ``ops.paged_attention`` (0: none)."""
     from .ext import ops
     dev = torch.device("cuda:0")
-    nbytes = 2 * batch * ctx * kv_heads * head_dim * 2
+    seen = min(ctx, window + keep) if window else ctx
+    nbytes = 2 * batch * seen * kv_heads * head_dim * 2
     group = heads // kv_heads
-    n = splits or ops.decode_splits(batch * kv_heads * ((group + 15) // 16), ctx)
+    n = splits or ops.decode_splits(batch * kv_heads * ((group + 15) // 16), seen)
     segs = torch.arange(batch, dtype=torch.int32, device=dev)
     fns = []
     for _ in range(_copies_beyond_l2(nbytes)):
         qkv, k_pool, v_pool, bt, cu_q, _, seg_kv_len = _paged_case(batch, ctx, 1, heads, kv_heads, head_dim, page, dev)
         out = torch.empty((batch, heads * head_dim), dtype=torch.bfloat16, device=dev)
         fns.append(lambda a=(qkv, k_pool, v_pool, cu_q, seg_kv_len, bt, out): ops.attention_decode_mma(
-            a[0], a[1], a[2], segs, a[3], a[4], a[5], page, a[6], heads, kv_heads, head_dim, head_dim ** -0.5, 0, n))
+            a[0], a[1], a[2], segs, a[3], a[4], a[5], page, a[6], heads, kv_heads, head_dim, head_dim ** -0.5, window, n,
+            softcap=softcap, keep=keep))
     ms = _time_kernels(fns, iters, warmup)
     return {"kernel": "attention_decode", "batch": batch, "ctx": ctx, "splits": n, "ms": ms,
             "GBps": nbytes / ms / 1e6}
 
 
 def kernel_attention_prefill(batch=1, ctx=2048, q_len=2048, heads=32, kv_heads=8, head_dim=128, page=16,
-                             iters=10, warmup=3, impl=0, splits=0) -> Dict[str, float]:
-    """The prefill attention kernel alone: device time and causal TFLOP/s.
+                             iters=10, warmup=3, impl=0, splits=0, window=0, keep=0, softcap=0.0) -> Dict[str, float]:
+    """The prefill attention kernel alone: device time and TFLOP/s over the visible keys.
+    ``window``, ``keep``, ``softcap``: the score options of ``ops.paged_attention`` (0: none).
     ``impl`` 0: the tcgen05 kernel (head sizes 64 and 128); 1: the mma.sync kernel.
     ``splits``: ways the tcgen05 kernel splits the keys (0: the engine's choice for this many CTAs)."""
     from .ext import ops
@@ -245,9 +249,12 @@ def kernel_attention_prefill(batch=1, ctx=2048, q_len=2048, heads=32, kv_heads=8
     splits = splits or ops.prefill_splits(int(tiles.shape[0]) * heads, ctx)
     more = {} if impl else {"num_splits": splits, "held": {}}
     fn = lambda: kernel(qkv, k_pool, v_pool, tiles, cu_q, seg_pos0, bt, page, out, heads,
-                        kv_heads, head_dim, head_dim ** -0.5, 0, **more)
+                        kv_heads, head_dim, head_dim ** -0.5, window, softcap=softcap, keep=keep, **more)
     ms = _time_kernels([fn], iters, warmup)
-    flops = 4.0 * batch * heads * head_dim * (q_len * (ctx - q_len) + q_len * q_len / 2.0)
+    pairs = q_len * (ctx - q_len) + q_len * q_len / 2.0
+    if window:
+        pairs = sum(min(p + 1, window + min(keep, max(0, p + 1 - window))) for p in range(ctx - q_len, ctx))
+    flops = 4.0 * batch * heads * head_dim * pairs
     return {"kernel": "attention_prefill_mma" if impl else "attention_prefill_tc5", "batch": batch, "ctx": ctx, "q_len": q_len, "splits": 1 if impl else splits,
             "ctas": int(tiles.shape[0]) * heads, "ms": ms, "TFLOPs": flops / ms / 1e9}
 
