@@ -656,7 +656,7 @@ def test_one_key_far_back_among_hundreds(tmp_path_factory, dtype, dim):
         assert (row_errors(got, want)[places] < 0.25 * gone).all()
 
 
-@pytest.mark.parametrize("dim,size,keep", [(16, 40, 6), (64, 64, 16), (64, 129, 70), (128, 33, 1), (16, 100, 130)])
+@pytest.mark.parametrize("dim,size,keep", [(16, 44, 5), (64, 64, 16), (64, 129, 70), (128, 33, 1), (16, 100, 130)])
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_keys_just_inside_and_outside_the_window_and_the_kept_first(tmp_path_factory, dtype, dim, size, keep):
     """Answering keys exactly at the window's last position and one before it, at the last kept position and one behind it, at
